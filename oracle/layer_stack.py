@@ -1,0 +1,156 @@
+"""Plain numpy (float64) restatement of the layer-stack designs: one function per mechanism, one token or one
+query at a time, no blocking, no cache tricks.  Test infrastructure only: nothing in `reimagined_b200/` imports
+this file, and it imports nothing from there.
+
+A model is a configuration dict plus a dict of named weight arrays; `Decoder` runs it token by token or in
+portions, with the recurrent states and the latent caches of one sequence.
+"""
+from __future__ import annotations
+
+from typing import Dict, List, Optional
+
+import numpy as np
+
+F = np.float64
+
+
+def sigmoid(z):
+    z = np.asarray(z, F)
+    e = np.exp(-np.abs(z))
+    return np.where(z >= 0, 1.0, e) / (1.0 + e)
+
+
+def silu(z):
+    return z * sigmoid(z)
+
+
+def linear(x, w, b=None):
+    """Rows of x times W^T; W is stored [out, in]."""
+    y = np.asarray(x, F) @ np.asarray(w, F).T
+    return y if b is None else y + np.asarray(b, F)
+
+
+def rms_norm(x, w, eps):
+    """x / sqrt(mean(x^2) + eps) over the last axis, times w (None: no weight)."""
+    x = np.asarray(x, F)
+    y = x / np.sqrt(np.mean(x * x, axis=-1, keepdims=True) + eps)
+    return y if w is None else y * np.asarray(w, F)
+
+
+def embed(table, tokens, scale):
+    return np.asarray(table, F)[np.asarray(tokens)] * scale
+
+
+def rotate_half(x, positions, base, dims):
+    """Rotary positions on the first `dims` entries of the last axis; entry i goes with entry i + dims/2.
+    x [T, ..., n], positions [T]."""
+    x = np.array(x, F)
+    half = dims // 2
+    freq = F(base) ** (-2.0 * np.arange(half) / dims)
+    ang = np.asarray(positions, F)[:, None] * freq[None, :]
+    ang = ang.reshape((len(positions),) + (1,) * (x.ndim - 2) + (half,))
+    u, v = x[..., :half].copy(), x[..., half:dims].copy()
+    x[..., :half] = u * np.cos(ang) - v * np.sin(ang)
+    x[..., half:dims] = v * np.cos(ang) + u * np.sin(ang)
+    return x
+
+
+def unit(k):
+    return k / np.sqrt(np.sum(k * k, axis=-1, keepdims=True) + 1e-6)
+
+
+def delta_decay(h, w1, w2, w0):
+    """Decay per channel, in (exp(-exp(-1/2)), 1)."""
+    z = linear(np.tanh(linear(h, w1)), w2) + np.asarray(w0, F)
+    return np.exp(-np.exp(-0.5) * sigmoid(z))
+
+
+def delta_step(S, r, k, v, w, a):
+    """One token of the generalized delta rule of one head: state [key, value] -> (new state, output)."""
+    u = unit(k)
+    S = w[:, None] * S - np.outer(a * u, u @ S) + np.outer(k, v)
+    return S, S.T @ r
+
+
+def general_delta(h, P, p, cfg, eps, states):
+    """Mixer: h [T, width]; states [heads, dim, dim] is updated in place."""
+    H, d = cfg["heads"], cfg["dim"]
+    T = len(h)
+    r, k, v = (linear(h, P[p + n]).reshape(T, H, d) for n in ("r", "k", "v"))
+    w = delta_decay(h, P[p + "w1"], P[p + "w2"], P[p + "w0"]).reshape(T, H, d)
+    a = sigmoid(linear(h, P[p + "a"], P[p + "a.b"])).reshape(T, H, d)
+    o = np.zeros((T, H, d))
+    for t in range(T):
+        for n in range(H):
+            states[n], o[t, n] = delta_step(states[n], r[t, n], k[t, n], v[t, n], w[t, n], a[t, n])
+    o = rms_norm(o, None, eps).reshape(T, H * d) * np.asarray(P[p + "norm"], F)
+    return linear(o * sigmoid(linear(h, P[p + "g"])), P[p + "o"])
+
+
+def softmax_attention(q, keys, values, scale):
+    """One query over all given keys: q [n], keys [m, n], values [m, vdim]."""
+    s = keys @ q * scale
+    e = np.exp(s - s.max())
+    return (e / e.sum()) @ values
+
+
+def latent_attention(h, P, p, cfg, eps, cache):
+    """Mixer: h [T, width]; cache is a list of (latent, rotated key part), one entry per earlier token."""
+    H, d, rd, vd, R = (cfg[n] for n in ("heads", "dim", "rot_dim", "vdim", "kv_rank"))
+    T, first = len(h), len(cache)
+    pos = np.arange(first, first + T)
+    base, dims = cfg["rot"]["base"], cfg["rot"]["dims"]
+    q = linear(rms_norm(linear(h, P[p + "dq"]), P[p + "dq.norm"], eps), P[p + "uq"]).reshape(T, H, d + rd)
+    q_plain, q_rot = q[..., :d], rotate_half(q[..., d:], pos, base, dims)
+    kv = linear(h, P[p + "dkv"])
+    c = rms_norm(kv[:, :R], P[p + "dkv.norm"], eps)
+    k_rot = rotate_half(kv[:, R:], pos, base, dims)
+    cache.extend(zip(c, k_rot))
+    lat = np.array([e[0] for e in cache])
+    rot = np.array([e[1] for e in cache])
+    keys = linear(lat, P[p + "uk"]).reshape(-1, H, d)
+    values = linear(lat, P[p + "uv"]).reshape(-1, H, vd)
+    out = np.zeros((T, H, vd))
+    for t in range(T):
+        n = first + t + 1
+        for i in range(H):
+            k_full = np.concatenate([keys[:n, i], rot[:n]], axis=1)
+            out[t, i] = softmax_attention(np.concatenate([q_plain[t, i], q_rot[t, i]]), k_full, values[:n, i], cfg["scale"])
+    return linear(out.reshape(T, H * vd) * sigmoid(linear(h, P[p + "g"])), P[p + "o"])
+
+
+def dense_ff(h, P, p):
+    g = linear(h, P[p + "gate"], P[p + "gate.b"])
+    u = linear(h, P[p + "up"], P[p + "up.b"])
+    return linear(silu(g) * u, P[p + "down"], P[p + "down.b"])
+
+
+def depth_average(weights, xs):
+    return sum(F(w) * x for w, x in zip(np.asarray(weights, F), xs))
+
+
+class Decoder:
+    """One sequence through the stack; `feed` takes any number of tokens and returns their logits."""
+
+    def __init__(self, cfg: dict, params: Dict[str, np.ndarray]):
+        self.cfg, self.P = cfg, params
+        self.memory: List = []
+        for layer in cfg["layers"]:
+            m = layer["mixer"]
+            self.memory.append(np.zeros((m["heads"], m["dim"], m["dim"])) if layer["type"] == "general_delta" else [])
+
+    def feed(self, tokens, trace: Optional[list] = None):
+        cfg, P, eps = self.cfg, self.P, self.cfg["norm"]["eps"]
+        x = embed(P["embed"], tokens, cfg["embedding"]["scale"])
+        xs = [x]
+        mixers = {"general_delta": general_delta, "latent_attention": latent_attention}
+        for i, layer in enumerate(cfg["layers"]):
+            p = f"l{i}."
+            x = x + mixers[layer["type"]](rms_norm(x, P[p + "norm1"], eps), P, p + "mix.", layer["mixer"], eps, self.memory[i])
+            if layer["mlp"] is not None:
+                x = x + dense_ff(rms_norm(x, P[p + "norm2"], eps), P, p + "mlp.")
+            xs.append(x)
+            x = depth_average(P[p + "dwa"], xs)
+            if trace is not None:
+                trace.append(x.copy())
+        return linear(rms_norm(x, P["final.norm"], eps), P["embed"])

@@ -1,4 +1,4 @@
-"""ctypes bindings of every symbol declared in include/ternary_b200.h.
+"""ctypes bindings of every symbol declared in include/ternary_b200.h and include/layer_stack.h.
 
 Pointers are passed as integers (``tensor.data_ptr()`` for device memory, ``array.ctypes.data`` for
 host memory); nothing here copies, allocates or falls back to a CPU path.
@@ -10,14 +10,15 @@ import os
 
 HERE = os.path.dirname(os.path.abspath(__file__))
 LIB_PATH = os.path.join(HERE, "libternary_b200.so")
+STACK_LIB_PATH = os.path.join(HERE, "libstack_b200.so")
 
 
 class TernaryB200Error(RuntimeError):
     """A C-ABI call returned a non-zero status."""
 
-    def __init__(self, status: int, where: str):
+    def __init__(self, status: int, where: str, library=None):
         self.status = status
-        msg = lib().tbl_status_string(status).decode()
+        msg = (library or lib()).tbl_status_string(status).decode()
         super().__init__(f"{where}: status {status} ({msg})")
 
 
@@ -81,6 +82,47 @@ class DecodeModel(C.Structure):
                 ("blocks", C.POINTER(DecodeBlock)), ("final_norm_w", C.c_void_p), ("final_norm_eps", C.c_float),
                 ("head", LinearView)]
 
+
+class DenseView(C.Structure):
+    """tbl_dense_view."""
+
+    _fields_ = [("weight", C.c_void_p), ("bias", C.c_void_p), ("inputs", C.c_int), ("outputs", C.c_int)]
+
+
+class DeltaMixer(C.Structure):
+    """tbl_delta_mixer."""
+
+    _fields_ = [("in_", DenseView), ("decay_up", DenseView), ("out", DenseView), ("norm", C.c_void_p), ("heads", C.c_int),
+                ("dim", C.c_int), ("rank", C.c_int), ("decay_rate", C.c_float), ("key_eps", C.c_float)]
+
+
+class LatentMixer(C.Structure):
+    """tbl_latent_mixer."""
+
+    _fields_ = [("in_", DenseView), ("uq", DenseView), ("uk", DenseView), ("uv", DenseView), ("out", DenseView),
+                ("q_norm", C.c_void_p), ("kv_norm", C.c_void_p), ("rope_cos", C.c_void_p), ("rope_sin", C.c_void_p),
+                ("heads", C.c_int), ("dim", C.c_int), ("rot_dim", C.c_int), ("vdim", C.c_int), ("q_rank", C.c_int),
+                ("kv_rank", C.c_int), ("rope_positions", C.c_int), ("scale", C.c_float)]
+
+
+class StackLayer(C.Structure):
+    """tbl_stack_layer."""
+
+    _fields_ = [("mixer", C.c_int), ("norm1", C.c_void_p), ("delta", DeltaMixer), ("latent", LatentMixer), ("ff", C.c_int),
+                ("norm2", C.c_void_p), ("gate_up", DenseView), ("down", DenseView), ("depth_weights", C.c_void_p)]
+
+
+class StackModel(C.Structure):
+    """tbl_stack_model."""
+
+    _fields_ = [("width", C.c_int), ("vocab", C.c_int), ("n_layers", C.c_int), ("embedding", C.c_void_p),
+                ("embedding_scale", C.c_float), ("norm_eps", C.c_float), ("layers", C.POINTER(StackLayer)),
+                ("final_norm", C.c_void_p), ("head", DenseView)]
+
+
+F32, BF16 = 0, 1
+MIXER_GENERAL_DELTA, MIXER_LATENT_ATTENTION = 0, 1
+PAIR_BLOCK = 32
 
 _vp = C.c_void_p
 _SIGNATURES = {
@@ -147,26 +189,59 @@ _SIGNATURES = {
 
 EXPORTED_SYMBOLS = tuple(_SIGNATURES)
 
+_sz, _int, _float = C.c_size_t, C.c_int, C.c_float
+_STACK_SIGNATURES = {
+    "tbl_stack_state_bytes": (_sz, [C.POINTER(StackModel), _int, _int, _int]),
+    "tbl_stack_state_reset": (_int, [C.POINTER(StackModel), _int, _int, _int, _int, _vp, _sz, _vp]),
+    "tbl_stack_workspace_bytes": (_sz, [C.POINTER(StackModel), _int, _int, _int, _int]),
+    "tbl_stack_step": (_int, [C.POINTER(StackModel), _int, _int, _int, _vp, _vp, _int, _int, _int, _vp, _vp, _int, _vp, _vp,
+                              _vp, _sz, _vp]),
+    "tbl_dense_forward": (_int, [C.POINTER(DenseView), _int, _int, _vp, _int, _int, _vp, _vp, _vp]),
+    "tbl_gated_dense_forward": (_int, [C.POINTER(DenseView), _int, _int, _vp, _int, _int, _int, _vp, _vp]),
+    "tbl_delta_workspace_bytes": (_sz, [C.POINTER(DeltaMixer), _int, _int]),
+    "tbl_delta_forward": (_int, [C.POINTER(DeltaMixer), _int, _int, _float, _vp, _vp, _vp, _int, _int, _vp, _vp, _sz, _vp]),
+    "tbl_latent_workspace_bytes": (_sz, [C.POINTER(LatentMixer), _int, _int, _int, _int]),
+    "tbl_latent_forward": (_int, [C.POINTER(LatentMixer), _int, _int, _float, _vp, _vp, _int, _vp, _vp, _int, _int, _int, _vp,
+                                  _vp, _sz, _vp]),
+    "tbl_depth_norm": (_int, [_vp, _sz, _int, _vp, _int, _vp, _int, _int, _float, _vp, _vp, _vp, _vp]),
+}
+STACK_SYMBOLS = tuple(_STACK_SIGNATURES)
+# declared in ternary_b200.h, present in every library (csrc/runtime.cu)
+_RUNTIME_SYMBOLS = ("tbl_status_string", "tbl_device_status", "tbl_launch_count")
+
 _lib = None
+_stack_lib = None
+
+
+def _open(path: str, name: str, signatures) -> C.CDLL:
+    if not os.path.exists(path):
+        raise ImportError(f"{path} is missing: build it with `python -m reimagined_b200.build {name}` "
+                          "(there is no CPU or PyTorch fallback)")
+    handle = C.CDLL(path)
+    for symbol, (restype, argtypes) in signatures.items():
+        fn = getattr(handle, symbol)
+        fn.restype = restype
+        fn.argtypes = argtypes
+    return handle
 
 
 def lib() -> C.CDLL:
     """Loads libternary_b200.so (once).  Raises if it has not been built: there is no fallback."""
     global _lib
     if _lib is None:
-        if not os.path.exists(LIB_PATH):
-            raise ImportError(
-                f"{LIB_PATH} is missing: build it with `python -m reimagined_b200.build` "
-                "(the ternary linear path has no CPU or PyTorch fallback)")
-        handle = C.CDLL(LIB_PATH)
-        for name, (restype, argtypes) in _SIGNATURES.items():
-            fn = getattr(handle, name)
-            fn.restype = restype
-            fn.argtypes = argtypes
-        _lib = handle
+        _lib = _open(LIB_PATH, "ternary", _SIGNATURES)
     return _lib
 
 
-def check(status: int, where: str) -> None:
+def stack_lib() -> C.CDLL:
+    """Loads libstack_b200.so (once), like lib()."""
+    global _stack_lib
+    if _stack_lib is None:
+        shared = {n: _SIGNATURES[n] for n in _RUNTIME_SYMBOLS}
+        _stack_lib = _open(STACK_LIB_PATH, "stack", {**_STACK_SIGNATURES, **shared})
+    return _stack_lib
+
+
+def check(status: int, where: str, library=None) -> None:
     if status != 0:
-        raise TernaryB200Error(status, where)
+        raise TernaryB200Error(status, where, library)

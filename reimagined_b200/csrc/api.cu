@@ -1,6 +1,5 @@
 // extern "C" entry points: validation, workspace carving and kernel selection.  No allocation,
 // no synchronisation (except tbl_device_status), no exceptions across the boundary.
-#include <atomic>
 #include <climits>
 #include <cmath>
 
@@ -8,9 +7,6 @@
 #include "kernels.cuh"
 
 namespace tbl {
-
-static std::atomic<uint64_t> g_launches{0};
-void note_launch(int n) { g_launches.fetch_add(static_cast<uint64_t>(n), std::memory_order_relaxed); }
 
 namespace {
 
@@ -133,28 +129,7 @@ using namespace tbl;
 
 extern "C" {
 
-const char* tbl_status_string(int status) {
-    switch (status) {
-        case TBL_OK: return "ok";
-        case TBL_ERR_INVALID_ARG: return "invalid argument (null pointer, non-positive size or bad flag)";
-        case TBL_ERR_SHAPE: return "unsupported shape (K must be a multiple of 16, M*N <= INT_MAX, M within the kernel's range)";
-        case TBL_ERR_OVERFLOW: return "K too large: int32 accumulation could overflow";
-        case TBL_ERR_SCALE: return "weight_scale must be finite and positive";
-        case TBL_ERR_BITS: return "activation bits must be in [2,8]";
-        case TBL_ERR_ALIGNMENT: return "device pointer must be 16-byte aligned";
-        case TBL_ERR_WORKSPACE: return "workspace too small";
-        case TBL_ERR_FORMAT: return "edge pack malformed";
-        case TBL_ERR_INTEGRITY: return "edge pack integrity trailer missing or digest mismatch";
-        case TBL_ERR_CODE: return "packed words contain the reserved code 0b11";
-        case TBL_ERR_CUDA: return "CUDA runtime error";
-        case TBL_ERR_UNSUPPORTED: return "descriptor mode not implemented";
-        default: return "unknown status";
-    }
-}
-
 int tbl_abi_version(void) { return 3; }
-
-uint64_t tbl_launch_count(void) { return g_launches.load(std::memory_order_relaxed); }
 
 void tbl_set_kernel_events(void* start_event, void* stop_event) {
     set_gemv_events(static_cast<cudaEvent_t>(start_event), static_cast<cudaEvent_t>(stop_event));
@@ -169,14 +144,6 @@ int tbl_selftest_bounded_wait(int* gave_up_dev, void* stream) {
     bounded_wait_selftest_kernel<<<1, 32, 0, static_cast<cudaStream_t>(stream)>>>(status, gave_up_dev);
     note_launch();
     return cuda_status(cudaGetLastError());
-}
-
-int tbl_device_status(void* stream) {
-    cudaError_t e = cudaStreamSynchronize(static_cast<cudaStream_t>(stream));
-    if (e != cudaSuccess) return TBL_ERR_CUDA;
-    int status = 0;
-    if (read_and_clear_device_status(&status) != 0) return TBL_ERR_CUDA;
-    return status;
 }
 
 size_t tbl_strip_bytes(int N, int K) {

@@ -1,0 +1,476 @@
+// The generalized delta rule (per head: S <- diag(w) S - (a*u)(u^T S) + k v^T, o = S^T r) with its decays, removal
+// rates, unit keys, head norm and output gate.  Everything here is fp32; states are stored [head][value][key].
+//
+// A value column j of a state evolves on its own:  s_j <- w*s_j + (k v_j - (a*u) (u.s_j)),  o_j = r.s_j,  so the
+// columns are spread over threads and CTAs and only the two dot products over the keys cross lanes: eight lanes share
+// a column, each holding every eighth group of four keys in registers, and the arithmetic runs on packed fp32 pairs.
+//
+//   delta_scan_kernel   a sequence of tokens: a CTA owns 32 columns of a head.  Four producer warps turn the raw
+//                       projections of the next chunk of tokens into (u, w, a*u, k, r, v) records in shared memory while
+//                       four consumer warps walk the current chunk token by token with the state in registers.
+//   delta_step_kernel   one token: a CTA per head also computes the low-rank decay product, the head norm and the gate.
+#include "stack.cuh"
+
+namespace tbl {
+namespace stack {
+namespace {
+
+using pair2 = unsigned long long;      // two packed fp32
+
+__device__ __forceinline__ pair2 dup2(float v) { pair2 r; asm("mov.b64 %0, {%1, %1};" : "=l"(r) : "f"(v)); return r; }
+__device__ __forceinline__ pair2 make2(float a, float b) { pair2 r; asm("mov.b64 %0, {%1, %2};" : "=l"(r) : "f"(a), "f"(b)); return r; }
+__device__ __forceinline__ void split2(pair2 v, float& a, float& b) { asm("mov.b64 {%0, %1}, %2;" : "=f"(a), "=f"(b) : "l"(v)); }
+__device__ __forceinline__ pair2 fma2(pair2 a, pair2 b, pair2 c) { pair2 d; asm("fma.rn.f32x2 %0, %1, %2, %3;" : "=l"(d) : "l"(a), "l"(b), "l"(c)); return d; }
+__device__ __forceinline__ pair2 mul2(pair2 a, pair2 b) { pair2 d; asm("mul.rn.f32x2 %0, %1, %2;" : "=l"(d) : "l"(a), "l"(b)); return d; }
+__device__ __forceinline__ pair2 add2(pair2 a, pair2 b) { pair2 d; asm("add.rn.f32x2 %0, %1, %2;" : "=l"(d) : "l"(a), "l"(b)); return d; }
+__device__ __forceinline__ float sum2(pair2 v) { float a, b; split2(v, a, b); return a + b; }
+__device__ __forceinline__ float sum8lanes(float v) {
+    v += __shfl_xor_sync(0xffffffffu, v, 1);
+    v += __shfl_xor_sync(0xffffffffu, v, 2);
+    v += __shfl_xor_sync(0xffffffffu, v, 4);
+    return v;
+}
+__device__ __forceinline__ void bar_sync(int id, int n) { asm volatile("bar.sync %0, %1;" ::"r"(id), "r"(n) : "memory"); }
+__device__ __forceinline__ void bar_arrive(int id, int n) { asm volatile("bar.arrive %0, %1;" ::"r"(id), "r"(n) : "memory"); }
+
+// Four keys of one column (key index c .. c+3, clipped at dim): state <-> registers.
+__device__ __forceinline__ ulonglong2 load_state4(const float* col, int c, int dim) {
+    if ((dim & 3) == 0) {
+        if (c >= dim) return make_ulonglong2(0, 0);
+        return *reinterpret_cast<const ulonglong2*>(col + c);
+    }
+    const float a = c < dim ? col[c] : 0.0f, b = c + 1 < dim ? col[c + 1] : 0.0f;
+    const float d = c + 2 < dim ? col[c + 2] : 0.0f, e = c + 3 < dim ? col[c + 3] : 0.0f;
+    return make_ulonglong2(make2(a, b), make2(d, e));
+}
+__device__ __forceinline__ void store_state4(float* col, int c, int dim, ulonglong2 v) {
+    if ((dim & 3) == 0) {
+        if (c < dim) *reinterpret_cast<ulonglong2*>(col + c) = v;
+        return;
+    }
+    float f[4];
+    split2(v.x, f[0], f[1]);
+    split2(v.y, f[2], f[3]);
+#pragma unroll
+    for (int i = 0; i < 4; ++i)
+        if (c + i < dim) col[c + i] = f[i];
+}
+
+struct DeltaParams {
+    const float* proj;       // [rows][ld]: r | k | v | g | a | w1 (raw products, biases added)
+    const float* z;          // [rows][heads*dim] decay products W_w2 tanh(.) (scan kernel)
+    const bf16* w2;          // [heads*dim][rank] (step kernel)
+    const float* w0;         // [heads*dim]
+    const float* norm;       // [heads*dim]
+    float* states;           // [slots][heads][dim][dim]
+    const int32_t* slots;
+    float* o;                // [rows][heads*dim] raw readouts (scan kernel)
+    void* out;
+    int ld, heads, dim, rank, n_tok;
+    float rate, key_eps, eps;
+};
+
+constexpr int kScanCols = 32;          // value columns per CTA
+constexpr int kScanThreads = 256;      // four consumer warps, four producer warps
+
+template <int DKP>
+struct ScanShape {
+    static constexpr int kChunk = DKP <= 128 ? 16 : 8;                 // tokens per buffer
+    static constexpr int kRecord = 5 * DKP + kScanCols;                // floats per token: u | w | a*u | k | r | v
+    static constexpr size_t kSmem = sizeof(float) * 2 * kChunk * kRecord;
+};
+
+template <int DKP>
+__global__ void __launch_bounds__(kScanThreads) delta_scan_kernel(const DeltaParams p) {
+    constexpr int CT = ScanShape<DKP>::kChunk, REC = ScanShape<DKP>::kRecord;
+    constexpr int G = DKP / 32;                // float4 groups per lane
+    constexpr int NI = DKP / 32;               // channels per producer lane
+    extern __shared__ __align__(16) float sm[];
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+    const int head = blockIdx.y, seq = blockIdx.z, j0 = blockIdx.x * kScanCols;
+    const int dim = p.dim, HD = p.heads * dim;
+    const int chunks = (p.n_tok + CT - 1) / CT;
+    const size_t row0 = static_cast<size_t>(seq) * p.n_tok;
+    pdl_launch_dependents();
+    pdl_wait();
+    if (warp >= 4) {
+        // ---- producers: warp w takes tokens w, w + 4, ... ----
+        const int pw = warp - 4;
+        float w0[NI];
+#pragma unroll
+        for (int i = 0; i < NI; ++i) w0[i] = lane + 32 * i < dim ? __ldg(p.w0 + head * dim + lane + 32 * i) : 0.0f;
+        float nr[NI], nk[NI], na[NI], nz[NI], nv = 0.0f;
+        auto fetch = [&](int t) {
+            const bool live = t < p.n_tok;
+            const float* row = p.proj + (row0 + (live ? t : 0)) * p.ld + head * dim;
+            const float* zr = p.z + (row0 + (live ? t : 0)) * HD + head * dim;
+#pragma unroll
+            for (int i = 0; i < NI; ++i) {
+                const int c = lane + 32 * i;
+                const bool ok = live && c < dim;
+                nr[i] = ok ? row[c] : 0.0f;
+                nk[i] = ok ? row[HD + c] : 0.0f;
+                na[i] = ok ? row[4 * HD + c] : 0.0f;
+                nz[i] = ok ? zr[c] : 0.0f;
+            }
+            nv = live && j0 + lane < dim ? row[2 * HD + j0 + lane] : 0.0f;
+        };
+        fetch(pw);
+        for (int ch = 0; ch < chunks; ++ch) {
+            const int b = ch & 1;
+            if (ch >= 2) bar_sync(3 + b, kScanThreads);
+            for (int i0 = pw; i0 < CT; i0 += 4) {
+                const int t = ch * CT + i0;
+                if (t >= p.n_tok) break;
+                float r[NI], k[NI], a[NI], z[NI];
+                float ss = 0.0f;
+#pragma unroll
+                for (int i = 0; i < NI; ++i) { r[i] = nr[i]; k[i] = nk[i]; a[i] = na[i]; z[i] = nz[i]; ss = fmaf(k[i], k[i], ss); }
+                const float v = nv;
+                fetch(t + 4);
+                const float inv = 1.0f / sqrtf(warp_sum(ss) + p.key_eps);
+                float* rec = sm + static_cast<size_t>(b * CT + i0) * REC;
+#pragma unroll
+                for (int i = 0; i < NI; ++i) {
+                    const int c = lane + 32 * i;
+                    const float u = k[i] * inv;
+                    rec[c] = u;
+                    rec[DKP + c] = expf(-p.rate * sigmoid_f(z[i] + w0[i]));
+                    rec[2 * DKP + c] = sigmoid_f(a[i]) * u;
+                    rec[3 * DKP + c] = k[i];
+                    rec[4 * DKP + c] = r[i];
+                }
+                rec[5 * DKP + lane] = v;
+            }
+            __threadfence_block();
+            bar_arrive(1 + b, kScanThreads);
+        }
+        return;
+    }
+    // ---- consumers: two columns per group of eight lanes ----
+    const int l8 = lane & 7, cl = warp * 8 + (lane >> 3) * 2;           // first of this lane's columns within the CTA
+    const int slot = p.slots[seq];
+    float* st = p.states + (static_cast<size_t>(slot) * p.heads + head) * dim * dim;
+    ulonglong2 S[2][G];
+#pragma unroll
+    for (int n = 0; n < 2; ++n)
+#pragma unroll
+        for (int g = 0; g < G; ++g)
+            S[n][g] = j0 + cl + n < dim ? load_state4(st + static_cast<size_t>(j0 + cl + n) * dim, 4 * (l8 + 8 * g), dim)
+                                        : make_ulonglong2(0, 0);
+    float* o = p.o + row0 * HD + head * dim + j0 + cl;
+    const bool ok0 = j0 + cl < dim, ok1 = j0 + cl + 1 < dim;
+    for (int ch = 0; ch < chunks; ++ch) {
+        const int b = ch & 1;
+        bar_sync(1 + b, kScanThreads);
+        const int n = min(CT, p.n_tok - ch * CT);
+#pragma unroll 1
+        for (int i = 0; i < n; ++i) {
+            const float* rec = sm + static_cast<size_t>(b * CT + i) * REC;
+            const ulonglong2* q = reinterpret_cast<const ulonglong2*>(rec) + l8;
+            pair2 d0 = 0, d1 = 0, e0 = 0, e1 = 0;
+#pragma unroll
+            for (int g = 0; g < G; ++g) {
+                const ulonglong2 u = q[8 * g];
+                d0 = fma2(u.x, S[0][g].x, d0); e0 = fma2(u.y, S[0][g].y, e0);
+                d1 = fma2(u.x, S[1][g].x, d1); e1 = fma2(u.y, S[1][g].y, e1);
+            }
+            const float2 v = *reinterpret_cast<const float2*>(rec + 5 * DKP + cl);
+            const pair2 m0 = dup2(-sum8lanes(sum2(add2(d0, e0)))), m1 = dup2(-sum8lanes(sum2(add2(d1, e1))));
+            const pair2 v0 = dup2(v.x), v1 = dup2(v.y);
+            pair2 o0 = 0, o1 = 0, f0 = 0, f1 = 0;
+#pragma unroll
+            for (int g = 0; g < G; ++g) {
+                const ulonglong2 w = q[DKP / 4 + 8 * g], au = q[2 * (DKP / 4) + 8 * g], k = q[3 * (DKP / 4) + 8 * g],
+                                 r = q[4 * (DKP / 4) + 8 * g];
+                S[0][g].x = fma2(w.x, S[0][g].x, fma2(au.x, m0, mul2(k.x, v0)));
+                S[0][g].y = fma2(w.y, S[0][g].y, fma2(au.y, m0, mul2(k.y, v0)));
+                S[1][g].x = fma2(w.x, S[1][g].x, fma2(au.x, m1, mul2(k.x, v1)));
+                S[1][g].y = fma2(w.y, S[1][g].y, fma2(au.y, m1, mul2(k.y, v1)));
+                o0 = fma2(r.x, S[0][g].x, o0); f0 = fma2(r.y, S[0][g].y, f0);
+                o1 = fma2(r.x, S[1][g].x, o1); f1 = fma2(r.y, S[1][g].y, f1);
+            }
+            const float r0 = sum8lanes(sum2(add2(o0, f0))), r1 = sum8lanes(sum2(add2(o1, f1)));
+            if (l8 == 0) {
+                float* ot = o + static_cast<size_t>(ch * CT + i) * HD;
+                if (ok0) ot[0] = r0;
+                if (ok1) ot[1] = r1;
+            }
+        }
+        if (ch + 2 < chunks) bar_arrive(3 + b, kScanThreads);
+    }
+#pragma unroll
+    for (int n = 0; n < 2; ++n)
+#pragma unroll
+        for (int g = 0; g < G; ++g)
+            if (j0 + cl + n < dim) store_state4(st + static_cast<size_t>(j0 + cl + n) * dim, 4 * (l8 + 8 * g), dim, S[n][g]);
+}
+
+// tanh of the low-rank decay projection, in the precision's type, for the GEMM with W_w2
+template <typename T>
+__global__ void __launch_bounds__(256) delta_tanh_kernel(const float* __restrict__ proj, int ld, int offset, int rows, int rank,
+                                                         int ldt, T* __restrict__ out) {
+    pdl_launch_dependents();
+    pdl_wait();
+    const size_t i = static_cast<size_t>(blockIdx.x) * 256 + threadIdx.x;
+    const size_t row = i / rank;
+    const int c = static_cast<int>(i - row * rank);
+    if (row < static_cast<size_t>(rows)) out[row * ldt + c] = from_f<T>(tanhf(proj[row * ld + offset + c]));
+}
+
+// head norm, weight and output gate of the scan's readouts: one warp per (row, head)
+template <typename T>
+__global__ void __launch_bounds__(256) delta_out_kernel(const DeltaParams p, int rows) {
+    pdl_launch_dependents();
+    pdl_wait();
+    const size_t unit = static_cast<size_t>(blockIdx.x) * 8 + (threadIdx.x >> 5);
+    const int lane = threadIdx.x & 31, dim = p.dim, HD = p.heads * dim;
+    if (unit >= static_cast<size_t>(rows) * p.heads) return;
+    const size_t row = unit / p.heads;
+    const int head = static_cast<int>(unit - row * p.heads);
+    const float* o = p.o + row * HD + head * dim;
+    const float* g = p.proj + row * p.ld + 3 * HD + head * dim;
+    T* out = static_cast<T*>(p.out) + row * HD + head * dim;
+    float ov[TBL_MAX_DELTA_DIM / 32], gv[TBL_MAX_DELTA_DIM / 32], ss = 0.0f;
+#pragma unroll
+    for (int i = 0; i < TBL_MAX_DELTA_DIM / 32; ++i) {
+        const int c = lane + 32 * i;
+        ov[i] = c < dim ? o[c] : 0.0f;
+        gv[i] = c < dim ? g[c] : 0.0f;
+        ss = fmaf(ov[i], ov[i], ss);
+    }
+    const float inv = 1.0f / sqrtf(warp_sum(ss) / static_cast<float>(dim) + p.eps);
+#pragma unroll
+    for (int i = 0; i < TBL_MAX_DELTA_DIM / 32; ++i) {
+        const int c = lane + 32 * i;
+        if (c < dim) out[c] = from_f<T>(ov[i] * inv * __ldg(p.norm + head * dim + c) * sigmoid_f(gv[i]));
+    }
+}
+
+// ---- one token ------------------------------------------------------------------------------------------------------
+// THREADS / 8 column groups; a thread's columns are its group + i * THREADS / 8, taken NCP at a time.
+template <typename T, int DKP, int THREADS, int NCP>
+__global__ void __launch_bounds__(THREADS) delta_step_kernel(const DeltaParams p) {
+    constexpr int G = DKP / 32, GROUPS = THREADS / 8, PASSES = DKP / (GROUPS * NCP);
+    static_assert(PASSES >= 1 && PASSES * GROUPS * NCP == DKP, "columns of a head");
+    __shared__ __align__(16) float su[DKP], sw[DKP], sau[DKP], sk[DKP], sr[DKP], sv[DKP], so[DKP], part[THREADS];
+    extern __shared__ float st_tanh[];         // [rank]
+    const int tid = threadIdx.x, lane = tid & 31;
+    const int head = blockIdx.x, row = blockIdx.y;
+    const int dim = p.dim, HD = p.heads * dim;
+    pdl_launch_dependents();
+    float* st = p.states + (static_cast<size_t>(p.slots[row]) * p.heads + head) * dim * dim;
+    for (int e = tid * 32; e < dim * dim; e += THREADS * 32) asm volatile("prefetch.global.L2 [%0];" ::"l"(st + e));
+    pdl_wait();
+    const float* pr = p.proj + static_cast<size_t>(row) * p.ld;
+    const int l8 = tid & 7, group = tid >> 3;
+    ulonglong2 S[NCP][G];
+    auto load_pass = [&](int ps) {
+#pragma unroll
+        for (int n = 0; n < NCP; ++n) {
+            const int j = (ps * NCP + n) * GROUPS + group;
+#pragma unroll
+            for (int g = 0; g < G; ++g)
+                S[n][g] = j < dim ? load_state4(st + static_cast<size_t>(j) * dim, 4 * (l8 + 8 * g), dim) : make_ulonglong2(0, 0);
+        }
+    };
+    load_pass(0);
+    for (int e = tid; e < p.rank; e += THREADS) st_tanh[e] = tanhf(pr[5 * HD + e]);
+    float ss = 0.0f;                            // every warp takes the key's norm for itself
+#pragma unroll
+    for (int i = 0; i < DKP / 32; ++i) {
+        const int c = lane + 32 * i;
+        const float k = c < dim ? pr[HD + head * dim + c] : 0.0f;
+        ss = fmaf(k, k, ss);
+    }
+    const float inv_key = 1.0f / sqrtf(warp_sum(ss) + p.key_eps);
+    __syncthreads();
+    // decay products: THREADS / DKP threads per channel
+    {
+        constexpr int TPC = THREADS / DKP;
+        const int c = tid / TPC, sub = tid % TPC;
+        float z = 0.0f;
+        if (c < dim) {
+            const bf16* w2 = p.w2 + static_cast<size_t>(head * dim + c) * p.rank;
+            if ((p.rank & 7) == 0) {
+                for (int e = sub * 8; e < p.rank; e += TPC * 8) {
+                    const uint4 w = __ldg(reinterpret_cast<const uint4*>(w2 + e));
+                    z = fmaf(bf_lo(w.x), st_tanh[e], z); z = fmaf(bf_hi(w.x), st_tanh[e + 1], z);
+                    z = fmaf(bf_lo(w.y), st_tanh[e + 2], z); z = fmaf(bf_hi(w.y), st_tanh[e + 3], z);
+                    z = fmaf(bf_lo(w.z), st_tanh[e + 4], z); z = fmaf(bf_hi(w.z), st_tanh[e + 5], z);
+                    z = fmaf(bf_lo(w.w), st_tanh[e + 6], z); z = fmaf(bf_hi(w.w), st_tanh[e + 7], z);
+                }
+            } else {
+                for (int e = sub; e < p.rank; e += TPC) z = fmaf(to_f(w2[e]), st_tanh[e], z);
+            }
+        }
+        part[tid] = z;
+        __syncthreads();
+        if (tid < DKP) {
+            float zc = 0.0f;
+#pragma unroll
+            for (int s = 0; s < TPC; ++s) zc += part[tid * TPC + s];
+            const bool ok = tid < dim;
+            const int hc = head * dim + tid;
+            const float k = ok ? pr[HD + hc] : 0.0f, u = k * inv_key;
+            su[tid] = u;
+            sk[tid] = k;
+            sr[tid] = ok ? pr[hc] : 0.0f;
+            sv[tid] = ok ? pr[2 * HD + hc] : 0.0f;
+            sw[tid] = ok ? expf(-p.rate * sigmoid_f(zc + __ldg(p.w0 + hc))) : 0.0f;
+            sau[tid] = ok ? sigmoid_f(pr[4 * HD + hc]) * u : 0.0f;
+        }
+    }
+    __syncthreads();
+    const ulonglong2 *qu = reinterpret_cast<const ulonglong2*>(su) + l8, *qw = reinterpret_cast<const ulonglong2*>(sw) + l8,
+                     *qa = reinterpret_cast<const ulonglong2*>(sau) + l8, *qk = reinterpret_cast<const ulonglong2*>(sk) + l8,
+                     *qr = reinterpret_cast<const ulonglong2*>(sr) + l8;
+#pragma unroll 1
+    for (int ps = 0; ps < PASSES; ++ps) {
+        if (ps > 0) load_pass(ps);
+        pair2 m[NCP], vv[NCP];
+#pragma unroll
+        for (int n = 0; n < NCP; ++n) {
+            pair2 d = 0, e = 0;
+#pragma unroll
+            for (int g = 0; g < G; ++g) { d = fma2(qu[8 * g].x, S[n][g].x, d); e = fma2(qu[8 * g].y, S[n][g].y, e); }
+            m[n] = dup2(-sum8lanes(sum2(add2(d, e))));
+            vv[n] = dup2(sv[(ps * NCP + n) * GROUPS + group]);
+        }
+#pragma unroll
+        for (int n = 0; n < NCP; ++n) {
+            const int j = (ps * NCP + n) * GROUPS + group;
+            pair2 o = 0, f = 0;
+#pragma unroll
+            for (int g = 0; g < G; ++g) {
+                S[n][g].x = fma2(qw[8 * g].x, S[n][g].x, fma2(qa[8 * g].x, m[n], mul2(qk[8 * g].x, vv[n])));
+                S[n][g].y = fma2(qw[8 * g].y, S[n][g].y, fma2(qa[8 * g].y, m[n], mul2(qk[8 * g].y, vv[n])));
+                o = fma2(qr[8 * g].x, S[n][g].x, o);
+                f = fma2(qr[8 * g].y, S[n][g].y, f);
+                if (j < dim) store_state4(st + static_cast<size_t>(j) * dim, 4 * (l8 + 8 * g), dim, S[n][g]);
+            }
+            const float r = sum8lanes(sum2(add2(o, f)));
+            if (l8 == 0) so[j] = r;
+        }
+    }
+    __syncthreads();
+    float sq = 0.0f;
+#pragma unroll
+    for (int i = 0; i < DKP / 32; ++i) { const float v = so[lane + 32 * i]; sq = fmaf(v, v, sq); }   // zero past dim
+    const float inv = 1.0f / sqrtf(warp_sum(sq) / static_cast<float>(dim) + p.eps);
+    if (tid < dim) {
+        const int hc = head * dim + tid;
+        static_cast<T*>(p.out)[static_cast<size_t>(row) * HD + hc] =
+            from_f<T>(so[tid] * inv * __ldg(p.norm + hc) * sigmoid_f(pr[3 * HD + hc]));
+    }
+}
+
+template <typename T>
+int launch_step(const DeltaParams& p, int n_seq, cudaStream_t st) {
+    const dim3 grid(p.heads, n_seq);
+    const size_t smem = sizeof(float) * p.rank;
+    if (n_seq > 65535 || smem > 32 * 1024) return TBL_ERR_SHAPE;
+    cudaError_t e;
+    if (p.dim <= 32) e = launch_dependent(delta_step_kernel<T, 32, 256, 1>, grid, dim3(256), smem, st, p);
+    else if (p.dim <= 64) e = launch_dependent(delta_step_kernel<T, 64, 256, 2>, grid, dim3(256), smem, st, p);
+    else if (p.dim <= 128) e = launch_dependent(delta_step_kernel<T, 128, 256, 4>, grid, dim3(256), smem, st, p);
+    else e = launch_dependent(delta_step_kernel<T, 256, 512, 1>, grid, dim3(512), smem, st, p);
+    return e == cudaSuccess ? TBL_OK : TBL_ERR_CUDA;
+}
+
+template <int DKP>
+int launch_scan_d(const DeltaParams& p, int n_seq, cudaStream_t st) {
+    static bool done[64] = {};
+    if (allow_smem(delta_scan_kernel<DKP>, ScanShape<DKP>::kSmem, done) != cudaSuccess) return TBL_ERR_CUDA;
+    const dim3 grid(ceil_div(p.dim, kScanCols), p.heads, n_seq);
+    if (p.heads > 65535 || n_seq > 65535) return TBL_ERR_SHAPE;
+    return launch_dependent(delta_scan_kernel<DKP>, grid, dim3(kScanThreads), ScanShape<DKP>::kSmem, st, p) == cudaSuccess ? TBL_OK
+                                                                                                                      : TBL_ERR_CUDA;
+}
+
+template <typename T>
+int launch_scan(const tbl_delta_mixer& m, DeltaParams p, int precision, int n_seq, void* ws, cudaStream_t st) {
+    const int rows = n_seq * p.n_tok, HD = p.heads * p.dim, ldt = static_cast<int>(round_up(p.rank, 8));
+    uint8_t* base = static_cast<uint8_t*>(ws);
+    float* z = reinterpret_cast<float*>(base);
+    base += round_up(sizeof(float) * static_cast<size_t>(rows) * HD, 256);
+    p.o = reinterpret_cast<float*>(base);
+    base += round_up(sizeof(float) * static_cast<size_t>(rows) * HD, 256);
+    T* th = reinterpret_cast<T*>(base);
+    if (launch_dependent(delta_tanh_kernel<T>, dim3(ceil_div(static_cast<long long>(rows) * p.rank, 256)), dim3(256), 0, st, p.proj, p.ld, 5 * HD,
+                         rows, p.rank, ldt, th) != cudaSuccess)
+        return TBL_ERR_CUDA;
+    DenseCall c{};
+    c.x = th; c.w = static_cast<const bf16*>(m.decay_up.weight); c.ldx = ldt; c.M = rows; c.K = p.rank; c.N = HD;
+    c.out_f32 = z; c.ldo = HD;
+    int rc = launch_dense(precision, kDenseAuto, c, st);
+    if (rc != TBL_OK) return rc;
+    p.z = z;
+    if (p.dim <= 32) rc = launch_scan_d<32>(p, n_seq, st);
+    else if (p.dim <= 64) rc = launch_scan_d<64>(p, n_seq, st);
+    else if (p.dim <= 128) rc = launch_scan_d<128>(p, n_seq, st);
+    else rc = launch_scan_d<256>(p, n_seq, st);
+    if (rc != TBL_OK) return rc;
+    const cudaError_t e = launch_dependent(delta_out_kernel<T>, dim3(ceil_div(static_cast<long long>(rows) * p.heads, 8)), dim3(256), 0, st, p, rows);
+    return e == cudaSuccess ? TBL_OK : TBL_ERR_CUDA;
+}
+
+}  // namespace
+
+int check_delta(const tbl_delta_mixer& m, int width) {
+    if (m.heads <= 0 || m.dim <= 0 || m.dim > TBL_MAX_DELTA_DIM || m.rank <= 0) return TBL_ERR_SHAPE;
+    const int HD = m.heads * m.dim;
+    if (m.in.inputs != width || m.in.outputs != 5 * HD + m.rank || m.decay_up.inputs != m.rank || m.decay_up.outputs != HD ||
+        m.out.inputs != HD || m.out.outputs != width)
+        return TBL_ERR_SHAPE;
+    if (!m.in.weight || !m.in.bias || !m.decay_up.weight || !m.decay_up.bias || !m.out.weight || !m.norm) return TBL_ERR_INVALID_ARG;
+    return TBL_OK;
+}
+
+size_t delta_workspace(const tbl_delta_mixer& m, int precision, int rows) {
+    const size_t HD = static_cast<size_t>(m.heads) * m.dim, e = precision == TBL_BF16 ? 2 : 4;
+    return 2 * round_up(sizeof(float) * rows * HD, 256) + round_up(e * rows * round_up(m.rank, 8), 256);
+}
+
+int launch_delta(const tbl_delta_mixer& m, int precision, int route, float eps, const float* proj, float* states,
+                 const int32_t* slots, int n_seq, int n_tok, void* out, void* ws, cudaStream_t st) {
+    DeltaParams p{};
+    p.proj = proj; p.w2 = static_cast<const bf16*>(m.decay_up.weight); p.w0 = m.decay_up.bias; p.norm = m.norm;
+    p.states = states; p.slots = slots; p.out = out; p.ld = m.in.outputs; p.heads = m.heads; p.dim = m.dim; p.rank = m.rank;
+    p.n_tok = n_tok; p.rate = m.decay_rate; p.key_eps = m.key_eps; p.eps = eps;
+    if (route == 0) route = n_tok == 1 ? 2 : 1;
+    if (route == 2) {
+        if (n_tok != 1) return TBL_ERR_SHAPE;
+        return precision == TBL_BF16 ? launch_step<bf16>(p, n_seq, st) : launch_step<float>(p, n_seq, st);
+    }
+    if (route != 1) return TBL_ERR_INVALID_ARG;
+    return precision == TBL_BF16 ? launch_scan<bf16>(m, p, precision, n_seq, ws, st) : launch_scan<float>(m, p, precision, n_seq, ws, st);
+}
+
+}  // namespace stack
+}  // namespace tbl
+
+using namespace tbl;
+using namespace tbl::stack;
+
+extern "C" {
+
+size_t tbl_delta_workspace_bytes(const tbl_delta_mixer* mixer, int precision, int rows) {
+    return mixer && rows > 0 ? delta_workspace(*mixer, precision, rows) : 0;
+}
+
+int tbl_delta_forward(const tbl_delta_mixer* mixer, int precision, int route, float eps, const float* proj_dev, float* states_dev,
+                      const int32_t* slots_dev, int n_seq, int n_tok, void* out_dev, void* workspace_dev, size_t workspace_bytes,
+                      void* stream) {
+    if (!mixer || !proj_dev || !states_dev || !slots_dev || !out_dev || n_seq <= 0 || n_tok <= 0 ||
+        (precision != TBL_F32 && precision != TBL_BF16))
+        return TBL_ERR_INVALID_ARG;
+    const int rc = check_delta(*mixer, mixer->in.inputs);
+    if (rc != TBL_OK) return rc;
+    if (!workspace_dev || workspace_bytes < delta_workspace(*mixer, precision, n_seq * n_tok)) return TBL_ERR_WORKSPACE;
+    if ((reinterpret_cast<uintptr_t>(workspace_dev) & 255) || (reinterpret_cast<uintptr_t>(states_dev) & 15)) return TBL_ERR_ALIGNMENT;
+    return launch_delta(*mixer, precision, route, eps, proj_dev, states_dev, slots_dev, n_seq, n_tok, out_dev, workspace_dev,
+                        static_cast<cudaStream_t>(stream));
+}
+
+}  // extern "C"

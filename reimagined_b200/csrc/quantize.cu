@@ -8,31 +8,6 @@
 
 namespace tbl {
 
-__device__ int g_device_status = 0;
-
-int* device_status_ptr() {
-    static int* cached[64] = {};
-    int dev = 0;
-    if (cudaGetDevice(&dev) != cudaSuccess || dev < 0 || dev >= 64) return nullptr;
-    if (!cached[dev]) {
-        void* p = nullptr;
-        if (cudaGetSymbolAddress(&p, g_device_status) != cudaSuccess) return nullptr;
-        cached[dev] = static_cast<int*>(p);
-    }
-    return cached[dev];
-}
-
-int read_and_clear_device_status(int* out) {
-    int status = 0;
-    if (cudaMemcpyFromSymbol(&status, g_device_status, sizeof(int)) != cudaSuccess) return -1;
-    if (status != 0) {
-        const int zero = 0;
-        if (cudaMemcpyToSymbol(g_device_status, &zero, sizeof(int)) != cudaSuccess) return -1;
-    }
-    *out = status;
-    return 0;
-}
-
 namespace {
 
 constexpr int kQuantThreads = 256;

@@ -247,6 +247,34 @@ class DecodeEngine:
         return self.launches_per_step
 
 
+class DecodeSession:
+    """The registry's engine interface over a DecodeEngine of one sequence (prompts are fed token by token)."""
+
+    slots = 1
+
+    def __init__(self, params: Dict[str, np.ndarray], capacity: int = 1024):
+        self.engine = DecodeEngine(params, batch=1, capacity=capacity)
+        self.vocab, self.capacity = self.engine.vocab, self.engine.capacity
+
+    def open(self) -> int:
+        self.engine.reset()
+        return 0
+
+    def close(self, slot: int) -> None:
+        pass
+
+    def feed(self, slot: int, tokens, want=None) -> torch.Tensor:
+        want = [len(tokens) - 1] if want is None else list(want)
+        rows = [self.engine.step([t]).clone() if i in want else self.engine.step([t])[:0] for i, t in enumerate(tokens)]
+        return torch.cat([rows[i] for i in want]) if want else rows[0][:0]
+
+    def step(self, slots, tokens) -> torch.Tensor:
+        return self.feed(slots[0], tokens[0])
+
+    def device_status(self) -> int:
+        return self.engine.L.tbl_device_status(torch.cuda.current_stream().cuda_stream)
+
+
 def main() -> None:
     ap = argparse.ArgumentParser(description="time one decode step of the D768 / 16-block hybrid")
     ap.add_argument("--batch", type=int, default=1)
