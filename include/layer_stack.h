@@ -89,7 +89,8 @@ typedef struct tbl_stack_model {
 
 /* Device state of `slots` sequences with room for `capacity` tokens each: positions, delta-rule states (fp32,
  * [head][value][key]) and latent caches [token][kv_rank + rot_dim].  reset clears one slot (its position and
- * recurrent states; cached rows are only read below the position), or every slot when slot < 0. */
+ * recurrent states), or the whole state when slot < 0: the latter once before the first use, so that cached rows
+ * nobody has written hold finite numbers (they are read under a zero weight). */
 size_t tbl_stack_state_bytes(const tbl_stack_model* model, int precision, int slots, int capacity);
 int tbl_stack_state_reset(const tbl_stack_model* model, int precision, int slots, int capacity, int slot,
                           void* state_dev, size_t state_bytes, void* stream);

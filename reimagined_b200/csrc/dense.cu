@@ -41,7 +41,7 @@ __global__ void __launch_bounds__(256) dense_simt_kernel(const DenseCall c) {
             const int e = threadIdx.x + i * 256, k = e & 15, r = e >> 4;
             const int kk = k0 + k;
             xs[k][r] = (m0 + r < c.M && kk < c.K) ? to_f(x[static_cast<size_t>(m0 + r) * c.ldx + kk]) : 0.0f;
-            ws[k][r] = (n0 + r < c.N && kk < c.K) ? to_f(c.w[static_cast<size_t>(n0 + r) * c.K + kk]) : 0.0f;
+            ws[k][r] = (n0 + r < c.N && kk < c.K) ? to_f(c.w[static_cast<size_t>(n0 + r) * c.ldw + kk]) : 0.0f;
         }
         __syncthreads();
 #pragma unroll
@@ -101,8 +101,8 @@ __global__ void __launch_bounds__(32 * kGemvWarps) dense_gemv_kernel(const Dense
     }
     const bf16* wp[R];
 #pragma unroll
-    for (int i = 0; i < R; ++i) wp[i] = c.w + static_cast<size_t>(min(rows[i], c.N - 1)) * c.K;
-    const bool vec = (c.K & 7) == 0;
+    for (int i = 0; i < R; ++i) wp[i] = c.w + static_cast<size_t>(min(rows[i], c.N - 1)) * c.ldw;
+    const bool vec = ((c.K | c.ldw) & 7) == 0;
     const int kv = vec ? c.K : 0;
     uint4 w[R], wn[R];
     const int k_first = lane * 8;
@@ -212,8 +212,10 @@ bool gemv_supported(const DenseCall& c) {
 
 }  // namespace
 
-int launch_dense(int precision, int route, const DenseCall& c, cudaStream_t st) {
-    if (c.M <= 0) return TBL_OK;
+int launch_dense(int precision, int route, const DenseCall& call, cudaStream_t st) {
+    if (call.M <= 0) return TBL_OK;
+    DenseCall c = call;
+    if (c.ldw == 0) c.ldw = c.K;
     const bool tensor = precision == TBL_BF16 && dense_tensor_supported(c);
     if (route == kDenseAuto) route = gemv_supported(c) ? kDenseGemv : (tensor ? kDenseTensor : kDenseSimt);
     if (route == kDenseTensor) {

@@ -148,9 +148,7 @@ dense_tcgen05_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_con
     } else if (warp == 1) {
         // ---------------- MMA issuer ----------------
         if (lane == 0) {
-            // kind::f16 instruction descriptor: D = fp32, A = B = bf16, both K-major, N = BN, M = 128
-            const uint32_t idesc = (1u << 4) | (1u << 7) | (1u << 10) | (static_cast<uint32_t>(BN >> 3) << 17) |
-                                   (static_cast<uint32_t>(BM >> 4) << 24);
+            const uint32_t idesc = idesc_bf16(BN);
             int it = 0, local = 0, row0, tn;
             bool alive = true;
             for (int tile = blockIdx.x; alive && decode_tile<MT>(p, tile, row0, tn); tile += gridDim.x, ++local) {
@@ -294,7 +292,7 @@ cudaError_t launch_bn(const CUtensorMap& ma, const CUtensorMap& mb, const Params
 }  // namespace
 
 bool dense_tensor_supported(const DenseCall& c) {
-    return c.K % 8 == 0 && c.ldx % 8 == 0 && (reinterpret_cast<uintptr_t>(c.x) & 15) == 0 &&
+    return c.K % 8 == 0 && c.ldx % 8 == 0 && c.ldw % 8 == 0 && (reinterpret_cast<uintptr_t>(c.x) & 15) == 0 &&
            (reinterpret_cast<uintptr_t>(c.w) & 15) == 0 && (!c.pair_cols || c.N % 64 == 0);
 }
 
@@ -325,7 +323,7 @@ cudaError_t launch_dense_tensor(const DenseCall& c, cudaStream_t st) {
     CUtensorMap ma, mb;
     if (!make_map(&ma, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, c.x, c.M, c.K, BKE, BM, CU_TENSOR_MAP_SWIZZLE_128B, c.ldx))
         return cudaErrorUnknown;
-    if (!make_map(&mb, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, c.w, c.N, c.K, BKE, bn)) return cudaErrorUnknown;
+    if (!make_map(&mb, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, c.w, c.N, c.K, BKE, bn, CU_TENSOR_MAP_SWIZZLE_128B, c.ldw)) return cudaErrorUnknown;
     if (tall) return launch_bn<256, 2>(ma, mb, p, st);
     return bn == 256 ? launch_bn<256, 1>(ma, mb, p, st) : (bn == 128 ? launch_bn<128, 1>(ma, mb, p, st) : launch_bn<64, 1>(ma, mb, p, st));
 }

@@ -15,10 +15,10 @@ struct LatentParams {
     void *cq, *qa;               // query latent [rows][ldq]; absorbed query [rows][H][cw], or the rotated query
     float* q;                    // [rows][H][d + rd]
     float *part_m, *part_l, *part_o;   // [rows][H][splits] ([R])
-    bf16 *keys, *values;         // expanded [sequence][context][H*d], [H*vd]
+    bf16 *keys, *values, *gathered;    // expanded context: [sequence x context][H*d], [H*vd][sequence x context]; its latents
     void* out;                   // [rows][H*vd]
     int* status;
-    int ld, ldq, cw, H, d, rd, vd, R, q_rank, capacity, rope_positions, n_tok, splits, context;
+    int ld, ldq, cw, H, d, rd, vd, R, q_rank, capacity, rope_positions, n_tok, splits, context, log2_parts;     // log2_parts: part_m in units of log 2
     float scale, eps;
 };
 
@@ -29,7 +29,8 @@ cudaError_t launch_latent_tensor(const LatentParams& p, int rows, cudaStream_t s
 
 // latent_prefill.cu: attention over expanded keys and values on tensor cores
 bool latent_expanded_supported(const tbl_latent_mixer& m);
-int launch_latent_expanded(const tbl_latent_mixer& m, const LatentParams& p, int n_seq, int context, cudaStream_t st);
+int latent_expanded_context(int context);                // padded to whole blocks
+int launch_latent_expanded(const tbl_latent_mixer& m, const LatentParams& p, int n_seq, cudaStream_t st);
 
 }  // namespace stack
 }  // namespace tbl

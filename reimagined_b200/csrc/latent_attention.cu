@@ -174,7 +174,7 @@ __global__ void __launch_bounds__(256) latent_value_kernel(const LatentParams p)
         for (int s = lane; s < p.splits; s += 32) m = fmaxf(m, p.part_m[unit + s]);
         m = warp_max(m);
         for (int s = lane; s < p.splits; s += 32) {
-            const float ms = p.part_m[unit + s], f = ms == -INFINITY ? 0.0f : expf(ms - m);
+            const float ms = p.part_m[unit + s], f = ms == -INFINITY ? 0.0f : (p.log2_parts ? exp2f(ms - m) : expf(ms - m));
             fac[s] = f;
             l = fmaf(p.part_l[unit + s], f, l);
         }
@@ -242,7 +242,7 @@ int pick_splits(const tbl_latent_mixer& m, int route, int rows, int context) {
 
 struct Plan {
     int route, splits;
-    size_t cq, q, qa, pm, pl, po, ek, ev, bytes;      // offsets
+    size_t cq, q, qa, pm, pl, po, ek, ev, ec, bytes;      // offsets
 };
 
 Plan make_plan(const tbl_latent_mixer& m, int precision, int route, int n_seq, int n_tok, int context) {
@@ -254,8 +254,10 @@ Plan make_plan(const tbl_latent_mixer& m, int precision, int route, int n_seq, i
     w.cq = take(e * rows * round_up(m.q_rank, 8));
     w.q = take(sizeof(float) * rows * m.heads * (m.dim + m.rot_dim));
     if (w.route == kExpanded) {
-        w.ek = take(e * n_seq * static_cast<size_t>(context) * m.heads * m.dim);
-        w.ev = take(e * n_seq * static_cast<size_t>(context) * m.heads * m.vdim);
+        const size_t padded = static_cast<size_t>(n_seq) * latent_expanded_context(context);
+        w.ek = take(e * padded * m.heads * m.dim);
+        w.ev = take(e * padded * m.heads * m.vdim);
+        w.ec = take(e * padded * latent_cache_width(m));
         w.qa = take(e * rows * m.heads * (m.dim + m.rot_dim));
     } else {
         w.splits = pick_splits(m, w.route, static_cast<int>(rows), context);
@@ -277,7 +279,10 @@ int run(const tbl_latent_mixer& m, LatentParams p, const Plan& w, int precision,
     c.N = p.H * (p.d + p.rd); c.out_f32 = p.q; c.ldo = c.N;
     int rc = launch_dense(precision, kDenseAuto, c, st);
     if (rc != TBL_OK) return rc;
-    if (w.route == kExpanded) return launch_latent_expanded(m, p, n_seq, context, st);
+    if (w.route == kExpanded) {
+        p.context = latent_expanded_context(context);
+        return launch_latent_expanded(m, p, n_seq, st);
+    }
     if (launch_dependent(latent_absorb_kernel<T>, dim3(rows, p.H), dim3(128), sizeof(float) * (p.d + p.rd), st, p) != cudaSuccess)
         return TBL_ERR_CUDA;
     if (w.route == kCacheTensor) {
@@ -328,9 +333,10 @@ int launch_latent(const tbl_latent_mixer& m, int precision, int route, float eps
     p.part_m = reinterpret_cast<float*>(base + w.pm); p.part_l = reinterpret_cast<float*>(base + w.pl);
     p.part_o = reinterpret_cast<float*>(base + w.po);
     p.keys = reinterpret_cast<bf16*>(base + w.ek); p.values = reinterpret_cast<bf16*>(base + w.ev);
+    p.gathered = reinterpret_cast<bf16*>(base + w.ec);
     p.ld = m.in.outputs; p.ldq = static_cast<int>(round_up(m.q_rank, 8)); p.cw = latent_cache_width(m);
     p.H = m.heads; p.d = m.dim; p.rd = m.rot_dim; p.vd = m.vdim; p.R = m.kv_rank; p.q_rank = m.q_rank;
-    p.capacity = capacity; p.rope_positions = m.rope_positions; p.n_tok = n_tok; p.splits = w.splits; p.context = context;
+    p.capacity = capacity; p.rope_positions = m.rope_positions; p.n_tok = n_tok; p.splits = w.splits; p.context = context; p.log2_parts = w.route == kCacheTensor;
     p.scale = m.scale; p.eps = eps;
     return precision == TBL_BF16 ? run<bf16>(m, p, w, precision, n_seq, context, st) : run<float>(m, p, w, precision, n_seq, context, st);
 }

@@ -122,11 +122,11 @@ int tbl_stack_state_reset(const tbl_stack_model* model, int precision, int slots
     if (!state_dev || state_bytes < tbl_stack_state_bytes(model, precision, slots, capacity)) return TBL_ERR_WORKSPACE;
     const StateLayout L = carve_state(*model, precision, slots, capacity, state_dev);
     cudaStream_t st = static_cast<cudaStream_t>(stream);
-    const int first = slot < 0 ? 0 : slot, count = slot < 0 ? slots : 1;
-    if (cudaMemsetAsync(L.positions + first, 0, sizeof(int32_t) * count, st) != cudaSuccess) return TBL_ERR_CUDA;
+    if (slot < 0) return cudaMemsetAsync(state_dev, 0, L.bytes, st) == cudaSuccess ? TBL_OK : TBL_ERR_CUDA;
+    if (cudaMemsetAsync(L.positions + slot, 0, sizeof(int32_t), st) != cudaSuccess) return TBL_ERR_CUDA;
     for (int i = 0; i < model->n_layers; ++i) {
         if (model->layers[i].mixer != TBL_MIXER_GENERAL_DELTA) continue;
-        if (cudaMemsetAsync(L.layer[i] + first * L.slot_bytes[i], 0, L.slot_bytes[i] * count, st) != cudaSuccess) return TBL_ERR_CUDA;
+        if (cudaMemsetAsync(L.layer[i] + slot * L.slot_bytes[i], 0, L.slot_bytes[i], st) != cudaSuccess) return TBL_ERR_CUDA;
     }
     return TBL_OK;
 }

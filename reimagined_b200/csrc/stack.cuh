@@ -76,9 +76,9 @@ cudaError_t allow_smem(Kernel kernel, size_t bytes, bool (&done)[64]) {
 // ---- dense.cu / dense_tcgen05.cu: y = W x + b with bf16 weights ------------------------------------------------
 struct DenseCall {
     const void* x;           // activations, the precision's type
-    const bf16* w;           // [N, K]
+    const bf16* w;           // [N, K], ldw between rows (0: K)
     const float* bias;       // [N] or null
-    int ldx, M, K, N;
+    int ldx, M, K, N, ldw;
     float* out_f32;          // exactly one of the two outputs
     bf16* out_b16;
     int ldo;

@@ -42,6 +42,15 @@ def tbl():
 
 
 @pytest.fixture(scope="session")
+def stack_lib():
+    """The layer-stack library through ctypes; built on demand."""
+    from reimagined_b200 import build
+    build.build(libraries=("stack",))
+    from reimagined_b200 import capi
+    return capi.stack_lib()
+
+
+@pytest.fixture(scope="session")
 def cuda():
     """torch with a live CUDA device.  A GPU test without a device fails (no silent skip on the GPU box)."""
     import torch
