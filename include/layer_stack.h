@@ -114,8 +114,8 @@ int tbl_stack_step(const tbl_stack_model* model, int precision, int slots, int c
  * Activations `x` have the precision's type (bf16 or fp32), strides in elements. */
 
 /* out[m, :] = W x[m, :] + b [+ residual[m, :]], fp32 out (ld = outputs of the view).  route: 0 the kernel the step
- * would take, 1 the SIMT kernel, 2 the GEMV, 3 the tcgen05 GEMM (bf16 only); TBL_ERR_SHAPE when the route does
- * not take the shape. */
+ * would take, 1 the SIMT kernel, 2 the GEMV, 3 the tcgen05 GEMM (bf16 only), 4 the row-streaming kernel (bf16 only);
+ * TBL_ERR_SHAPE when the route does not take the shape. */
 int tbl_dense_forward(const tbl_dense_view* view, int precision, int route, const void* x_dev, int ldx, int rows,
                       const float* residual_dev, float* out_dev, void* stream);
 /* out[m, :ff] (precision's type, ld = ff) = silu(gate) * up for a gate_up view of 2*round_up(ff, 32) rows. */

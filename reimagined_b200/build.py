@@ -23,7 +23,7 @@ LIBRARIES = {
                  "gemv_chain.cu", "gemm_tcgen05.cu", "gemm_widen.cu", "moe.cu", "glue.cu", "decode.cu", "packer.cpp",
                  "edge_pack.cpp"]),
     "stack": (os.path.join(HERE, "libstack_b200.so"),
-              ["runtime.cu", "stack.cu", "stack_glue.cu", "dense.cu", "dense_tcgen05.cu", "delta_rule.cu",
+              ["runtime.cu", "stack.cu", "stack_glue.cu", "dense.cu", "dense_rows.cu", "dense_tcgen05.cu", "delta_rule.cu",
                "latent_attention.cu", "latent_decode.cu", "latent_prefill.cu"]),
 }
 LIB, SOURCES = LIBRARIES["ternary"]

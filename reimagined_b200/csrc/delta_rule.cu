@@ -5,7 +5,7 @@
 // columns are spread over threads and CTAs and only the two dot products over the keys cross lanes: eight lanes share
 // a column, each holding every eighth group of four keys in registers, and the arithmetic runs on packed fp32 pairs.
 //
-//   delta_scan_kernel   a sequence of tokens: a CTA owns 32 columns of a head.  Four producer warps turn the raw
+//   delta_scan_kernel   a sequence of tokens: a CTA owns 32 columns of a head.  Eight producer warps turn the raw
 //                       projections of the next chunk of tokens into (u, w, a*u, k, r, v) records in shared memory while
 //                       four consumer warps walk the current chunk token by token with the state in registers.
 //   delta_step_kernel   one token: a CTA per head also computes the low-rank decay product, the head norm and the gate.
@@ -28,6 +28,13 @@ __device__ __forceinline__ float sum8lanes(float v) {
     v += __shfl_xor_sync(0xffffffffu, v, 1);
     v += __shfl_xor_sync(0xffffffffu, v, 2);
     v += __shfl_xor_sync(0xffffffffu, v, 4);
+    return v;
+}
+// Sums of a and b over a group of eight lanes: lanes 0-3 return a's, lanes 4-7 (upper) b's.
+__device__ __forceinline__ float sum_halves(float a, float b, bool upper) {
+    float v = (upper ? b : a) + __shfl_xor_sync(0xffffffffu, upper ? a : b, 4);
+    v += __shfl_xor_sync(0xffffffffu, v, 1);
+    v += __shfl_xor_sync(0xffffffffu, v, 2);
     return v;
 }
 __device__ __forceinline__ void bar_sync(int id, int n) { asm volatile("bar.sync %0, %1;" ::"r"(id), "r"(n) : "memory"); }
@@ -71,11 +78,12 @@ struct DeltaParams {
 };
 
 constexpr int kScanCols = 32;          // value columns per CTA
-constexpr int kScanThreads = 256;      // four consumer warps, four producer warps
+constexpr int kProducers = 8;          // producer warps: enough tokens in flight to cover the loads' latency
+constexpr int kScanThreads = 32 * (4 + kProducers);
 
 template <int DKP>
 struct ScanShape {
-    static constexpr int kChunk = DKP <= 128 ? 16 : 8;                 // tokens per buffer
+    static constexpr int kChunk = DKP <= 128 ? 16 : 8;                 // tokens per buffer, a multiple of kProducers
     static constexpr int kRecord = 5 * DKP + kScanCols;                // floats per token: u | w | a*u | k | r | v
     static constexpr size_t kSmem = sizeof(float) * 2 * kChunk * kRecord;
 };
@@ -84,7 +92,7 @@ template <int DKP>
 __global__ void __launch_bounds__(kScanThreads) delta_scan_kernel(const DeltaParams p) {
     constexpr int CT = ScanShape<DKP>::kChunk, REC = ScanShape<DKP>::kRecord;
     constexpr int G = DKP / 32;                // float4 groups per lane
-    constexpr int NI = DKP / 32;               // channels per producer lane
+    constexpr int NI = (DKP + 127) / 128;      // groups of four channels per producer lane
     extern __shared__ __align__(16) float sm[];
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     const int head = blockIdx.y, seq = blockIdx.z, j0 = blockIdx.x * kScanCols;
@@ -94,24 +102,34 @@ __global__ void __launch_bounds__(kScanThreads) delta_scan_kernel(const DeltaPar
     pdl_launch_dependents();
     pdl_wait();
     if (warp >= 4) {
-        // ---- producers: warp w takes tokens w, w + 4, ... ----
+        // ---- producers: warp w takes tokens w, w + kProducers, ...; lane l channels 4l .. 4l + 3 (+ 128) ----
         const int pw = warp - 4;
-        float w0[NI];
+        const bool vec = ((dim | p.ld) & 3) == 0;      // every row and head starts on 16 bytes
+        auto load4 = [&](const float* base, int c, bool live) {
+            float4 v = make_float4(0.0f, 0.0f, 0.0f, 0.0f);
+            if (!live || c >= dim) return v;
+            if (vec) return *reinterpret_cast<const float4*>(base + c);
+            v.x = base[c];
+            if (c + 1 < dim) v.y = base[c + 1];
+            if (c + 2 < dim) v.z = base[c + 2];
+            if (c + 3 < dim) v.w = base[c + 3];
+            return v;
+        };
+        float4 w0[NI], nr[NI], nk[NI], na[NI], nz[NI];
+        float nv = 0.0f;
 #pragma unroll
-        for (int i = 0; i < NI; ++i) w0[i] = lane + 32 * i < dim ? __ldg(p.w0 + head * dim + lane + 32 * i) : 0.0f;
-        float nr[NI], nk[NI], na[NI], nz[NI], nv = 0.0f;
+        for (int i = 0; i < NI; ++i) w0[i] = load4(p.w0 + head * dim, 4 * lane + 128 * i, true);
         auto fetch = [&](int t) {
             const bool live = t < p.n_tok;
             const float* row = p.proj + (row0 + (live ? t : 0)) * p.ld + head * dim;
             const float* zr = p.z + (row0 + (live ? t : 0)) * HD + head * dim;
 #pragma unroll
             for (int i = 0; i < NI; ++i) {
-                const int c = lane + 32 * i;
-                const bool ok = live && c < dim;
-                nr[i] = ok ? row[c] : 0.0f;
-                nk[i] = ok ? row[HD + c] : 0.0f;
-                na[i] = ok ? row[4 * HD + c] : 0.0f;
-                nz[i] = ok ? zr[c] : 0.0f;
+                const int c = 4 * lane + 128 * i;
+                nr[i] = load4(row, c, live);
+                nk[i] = load4(row + HD, c, live);
+                na[i] = load4(row + 4 * HD, c, live);
+                nz[i] = load4(zr, c, live);
             }
             nv = live && j0 + lane < dim ? row[2 * HD + j0 + lane] : 0.0f;
         };
@@ -119,26 +137,33 @@ __global__ void __launch_bounds__(kScanThreads) delta_scan_kernel(const DeltaPar
         for (int ch = 0; ch < chunks; ++ch) {
             const int b = ch & 1;
             if (ch >= 2) bar_sync(3 + b, kScanThreads);
-            for (int i0 = pw; i0 < CT; i0 += 4) {
+            for (int i0 = pw; i0 < CT; i0 += kProducers) {
                 const int t = ch * CT + i0;
                 if (t >= p.n_tok) break;
-                float r[NI], k[NI], a[NI], z[NI];
+                float4 r[NI], k[NI], a[NI], z[NI];
                 float ss = 0.0f;
 #pragma unroll
-                for (int i = 0; i < NI; ++i) { r[i] = nr[i]; k[i] = nk[i]; a[i] = na[i]; z[i] = nz[i]; ss = fmaf(k[i], k[i], ss); }
+                for (int i = 0; i < NI; ++i) {
+                    r[i] = nr[i]; k[i] = nk[i]; a[i] = na[i]; z[i] = nz[i];
+                    ss += k[i].x * k[i].x + k[i].y * k[i].y + k[i].z * k[i].z + k[i].w * k[i].w;
+                }
                 const float v = nv;
-                fetch(t + 4);
+                fetch(t + kProducers);
                 const float inv = 1.0f / sqrtf(warp_sum(ss) + p.key_eps);
                 float* rec = sm + static_cast<size_t>(b * CT + i0) * REC;
+                auto decay = [&](float zz) { return expf(-p.rate * sigmoid_f(zz)); };
 #pragma unroll
                 for (int i = 0; i < NI; ++i) {
-                    const int c = lane + 32 * i;
-                    const float u = k[i] * inv;
-                    rec[c] = u;
-                    rec[DKP + c] = expf(-p.rate * sigmoid_f(z[i] + w0[i]));
-                    rec[2 * DKP + c] = sigmoid_f(a[i]) * u;
-                    rec[3 * DKP + c] = k[i];
-                    rec[4 * DKP + c] = r[i];
+                    const int c = 4 * lane + 128 * i;
+                    if (c >= DKP) break;
+                    const float4 u = make_float4(k[i].x * inv, k[i].y * inv, k[i].z * inv, k[i].w * inv);
+                    *reinterpret_cast<float4*>(rec + c) = u;
+                    *reinterpret_cast<float4*>(rec + DKP + c) =
+                        make_float4(decay(z[i].x + w0[i].x), decay(z[i].y + w0[i].y), decay(z[i].z + w0[i].z), decay(z[i].w + w0[i].w));
+                    *reinterpret_cast<float4*>(rec + 2 * DKP + c) =
+                        make_float4(sigmoid_f(a[i].x) * u.x, sigmoid_f(a[i].y) * u.y, sigmoid_f(a[i].z) * u.z, sigmoid_f(a[i].w) * u.w);
+                    *reinterpret_cast<float4*>(rec + 3 * DKP + c) = k[i];
+                    *reinterpret_cast<float4*>(rec + 4 * DKP + c) = r[i];
                 }
                 rec[5 * DKP + lane] = v;
             }
@@ -158,13 +183,14 @@ __global__ void __launch_bounds__(kScanThreads) delta_scan_kernel(const DeltaPar
         for (int g = 0; g < G; ++g)
             S[n][g] = j0 + cl + n < dim ? load_state4(st + static_cast<size_t>(j0 + cl + n) * dim, 4 * (l8 + 8 * g), dim)
                                         : make_ulonglong2(0, 0);
-    float* o = p.o + row0 * HD + head * dim + j0 + cl;
-    const bool ok0 = j0 + cl < dim, ok1 = j0 + cl + 1 < dim;
+    const bool upper = (l8 & 4) != 0;                  // lanes 0-3 of a group end up with the first column's sums, 4-7 with the second's
+    float* o = p.o + row0 * HD + head * dim + j0 + cl + (upper ? 1 : 0);
+    const bool writes = (l8 & 3) == 0 && j0 + cl + (upper ? 1 : 0) < dim;
     for (int ch = 0; ch < chunks; ++ch) {
         const int b = ch & 1;
         bar_sync(1 + b, kScanThreads);
         const int n = min(CT, p.n_tok - ch * CT);
-#pragma unroll 1
+#pragma unroll 2
         for (int i = 0; i < n; ++i) {
             const float* rec = sm + static_cast<size_t>(b * CT + i) * REC;
             const ulonglong2* q = reinterpret_cast<const ulonglong2*>(rec) + l8;
@@ -176,7 +202,10 @@ __global__ void __launch_bounds__(kScanThreads) delta_scan_kernel(const DeltaPar
                 d1 = fma2(u.x, S[1][g].x, d1); e1 = fma2(u.y, S[1][g].y, e1);
             }
             const float2 v = *reinterpret_cast<const float2*>(rec + 5 * DKP + cl);
-            const pair2 m0 = dup2(-sum8lanes(sum2(add2(d0, e0)))), m1 = dup2(-sum8lanes(sum2(add2(d1, e1))));
+            // both columns' sums over the eight lanes: each half of the lanes adds up one column, then they swap
+            const float own = sum_halves(sum2(add2(d0, e0)), sum2(add2(d1, e1)), upper);
+            const float other = __shfl_xor_sync(0xffffffffu, own, 4);
+            const pair2 m0 = dup2(upper ? -other : -own), m1 = dup2(upper ? -own : -other);
             const pair2 v0 = dup2(v.x), v1 = dup2(v.y);
             pair2 o0 = 0, o1 = 0, f0 = 0, f1 = 0;
 #pragma unroll
@@ -190,12 +219,8 @@ __global__ void __launch_bounds__(kScanThreads) delta_scan_kernel(const DeltaPar
                 o0 = fma2(r.x, S[0][g].x, o0); f0 = fma2(r.y, S[0][g].y, f0);
                 o1 = fma2(r.x, S[1][g].x, o1); f1 = fma2(r.y, S[1][g].y, f1);
             }
-            const float r0 = sum8lanes(sum2(add2(o0, f0))), r1 = sum8lanes(sum2(add2(o1, f1)));
-            if (l8 == 0) {
-                float* ot = o + static_cast<size_t>(ch * CT + i) * HD;
-                if (ok0) ot[0] = r0;
-                if (ok1) ot[1] = r1;
-            }
+            const float ro = sum_halves(sum2(add2(o0, f0)), sum2(add2(o1, f1)), upper);
+            if (writes) o[static_cast<size_t>(ch * CT + i) * HD] = ro;
         }
         if (ch + 2 < chunks) bar_arrive(3 + b, kScanThreads);
     }
@@ -249,11 +274,11 @@ __global__ void __launch_bounds__(256) delta_out_kernel(const DeltaParams p, int
 
 // ---- one token ------------------------------------------------------------------------------------------------------
 // THREADS / 8 column groups; a thread's columns are its group + i * THREADS / 8, taken NCP at a time.
-template <typename T, int DKP, int THREADS, int NCP>
-__global__ void __launch_bounds__(THREADS) delta_step_kernel(const DeltaParams p) {
+template <typename T, int DKP, int THREADS, int NCP, bool FUSED>
+__global__ void __launch_bounds__(THREADS, DKP == 128 ? 2 : 1) delta_step_kernel(const DeltaParams p) {
     constexpr int G = DKP / 32, GROUPS = THREADS / 8, PASSES = DKP / (GROUPS * NCP);
     static_assert(PASSES >= 1 && PASSES * GROUPS * NCP == DKP, "columns of a head");
-    __shared__ __align__(16) float su[DKP], sw[DKP], sau[DKP], sk[DKP], sr[DKP], sv[DKP], so[DKP], part[THREADS];
+    __shared__ __align__(16) float su[DKP], sw[DKP], sau[DKP], sk[DKP], sr[DKP], sv[DKP], so[DKP], part[FUSED ? THREADS : 1];
     extern __shared__ float st_tanh[];         // [rank]
     const int tid = threadIdx.x, lane = tid & 31;
     const int head = blockIdx.x, row = blockIdx.y;
@@ -274,25 +299,27 @@ __global__ void __launch_bounds__(THREADS) delta_step_kernel(const DeltaParams p
                 S[n][g] = j < dim ? load_state4(st + static_cast<size_t>(j) * dim, 4 * (l8 + 8 * g), dim) : make_ulonglong2(0, 0);
         }
     };
-    load_pass(0);
-    for (int e = tid; e < p.rank; e += THREADS) st_tanh[e] = tanhf(pr[5 * HD + e]);
-    float ss = 0.0f;                            // every warp takes the key's norm for itself
+    // everything that depends on this step's projections is requested first, then the state
+    const int hc = head * dim + tid;
+    const bool ch = tid < dim;
+    const float k_in = ch ? pr[HD + hc] : 0.0f, r_in = ch ? pr[hc] : 0.0f, v_in = ch ? pr[2 * HD + hc] : 0.0f;
+    const float g_in = ch ? pr[3 * HD + hc] : 0.0f, a_in = ch ? pr[4 * HD + hc] : 0.0f;
+    float z_in = !FUSED && ch ? p.z[static_cast<size_t>(row) * HD + hc] : 0.0f;
+    float kn[DKP / 32];
 #pragma unroll
-    for (int i = 0; i < DKP / 32; ++i) {
-        const int c = lane + 32 * i;
-        const float k = c < dim ? pr[HD + head * dim + c] : 0.0f;
-        ss = fmaf(k, k, ss);
-    }
-    const float inv_key = 1.0f / sqrtf(warp_sum(ss) + p.key_eps);
-    __syncthreads();
-    // decay products: THREADS / DKP threads per channel
-    {
+    for (int i = 0; i < DKP / 32; ++i) kn[i] = lane + 32 * i < dim ? pr[HD + head * dim + lane + 32 * i] : 0.0f;
+    load_pass(0);
+    if constexpr (FUSED) {
+        for (int e = tid; e < p.rank; e += THREADS) st_tanh[e] = tanhf(pr[5 * HD + e]);
+        __syncthreads();
+        // decay products: THREADS / DKP threads per channel
         constexpr int TPC = THREADS / DKP;
         const int c = tid / TPC, sub = tid % TPC;
         float z = 0.0f;
         if (c < dim) {
             const bf16* w2 = p.w2 + static_cast<size_t>(head * dim + c) * p.rank;
             if ((p.rank & 7) == 0) {
+#pragma unroll 4
                 for (int e = sub * 8; e < p.rank; e += TPC * 8) {
                     const uint4 w = __ldg(reinterpret_cast<const uint4*>(w2 + e));
                     z = fmaf(bf_lo(w.x), st_tanh[e], z); z = fmaf(bf_hi(w.x), st_tanh[e + 1], z);
@@ -306,20 +333,23 @@ __global__ void __launch_bounds__(THREADS) delta_step_kernel(const DeltaParams p
         }
         part[tid] = z;
         __syncthreads();
-        if (tid < DKP) {
-            float zc = 0.0f;
+        if (ch) {
 #pragma unroll
-            for (int s = 0; s < TPC; ++s) zc += part[tid * TPC + s];
-            const bool ok = tid < dim;
-            const int hc = head * dim + tid;
-            const float k = ok ? pr[HD + hc] : 0.0f, u = k * inv_key;
-            su[tid] = u;
-            sk[tid] = k;
-            sr[tid] = ok ? pr[hc] : 0.0f;
-            sv[tid] = ok ? pr[2 * HD + hc] : 0.0f;
-            sw[tid] = ok ? expf(-p.rate * sigmoid_f(zc + __ldg(p.w0 + hc))) : 0.0f;
-            sau[tid] = ok ? sigmoid_f(pr[4 * HD + hc]) * u : 0.0f;
+            for (int s = 0; s < TPC; ++s) z_in += part[tid * TPC + s];
         }
+    }
+    float ss = 0.0f;                            // every warp takes the key's norm for itself
+#pragma unroll
+    for (int i = 0; i < DKP / 32; ++i) ss = fmaf(kn[i], kn[i], ss);
+    const float inv_key = 1.0f / sqrtf(warp_sum(ss) + p.key_eps);
+    if (tid < DKP) {
+        const float u = k_in * inv_key;
+        su[tid] = u;
+        sk[tid] = k_in;
+        sr[tid] = r_in;
+        sv[tid] = v_in;
+        sw[tid] = ch ? expf(-p.rate * sigmoid_f(z_in + __ldg(p.w0 + hc))) : 0.0f;
+        sau[tid] = sigmoid_f(a_in) * u;
     }
     __syncthreads();
     const ulonglong2 *qu = reinterpret_cast<const ulonglong2*>(su) + l8, *qw = reinterpret_cast<const ulonglong2*>(sw) + l8,
@@ -358,23 +388,62 @@ __global__ void __launch_bounds__(THREADS) delta_step_kernel(const DeltaParams p
 #pragma unroll
     for (int i = 0; i < DKP / 32; ++i) { const float v = so[lane + 32 * i]; sq = fmaf(v, v, sq); }   // zero past dim
     const float inv = 1.0f / sqrtf(warp_sum(sq) / static_cast<float>(dim) + p.eps);
-    if (tid < dim) {
-        const int hc = head * dim + tid;
-        static_cast<T*>(p.out)[static_cast<size_t>(row) * HD + hc] =
-            from_f<T>(so[tid] * inv * __ldg(p.norm + hc) * sigmoid_f(pr[3 * HD + hc]));
-    }
+    if (ch) static_cast<T*>(p.out)[static_cast<size_t>(row) * HD + hc] = from_f<T>(so[tid] * inv * __ldg(p.norm + hc) * sigmoid_f(g_in));
+}
+
+// From this many rows on W_w2 is one product over all of them instead of a part of every head's CTA.
+constexpr int kStepFusedRows = 4;
+
+// z = W_w2 tanh(low-rank part), fp32 [rows][heads*dim]
+template <typename T>
+int decay_products(const tbl_delta_mixer& m, const DeltaParams& p, int precision, int rows, T* th, float* z, cudaStream_t st) {
+    const int HD = p.heads * p.dim, ldt = static_cast<int>(round_up(p.rank, 8));
+    if (launch_dependent(delta_tanh_kernel<T>, dim3(ceil_div(static_cast<long long>(rows) * p.rank, 256)), dim3(256), 0, st, p.proj, p.ld, 5 * HD,
+                         rows, p.rank, ldt, th) != cudaSuccess)
+        return TBL_ERR_CUDA;
+    DenseCall c{};
+    c.x = th; c.w = static_cast<const bf16*>(m.decay_up.weight); c.ldx = ldt; c.M = rows; c.K = p.rank; c.N = HD;
+    c.out_f32 = z; c.ldo = HD;
+    return launch_dense(precision, kDenseAuto, c, st);
+}
+
+template <typename T, int DKP, int THREADS, int NCP>
+cudaError_t launch_step_d(const DeltaParams& p, dim3 grid, cudaStream_t st) {
+    return p.z ? launch_dependent(delta_step_kernel<T, DKP, THREADS, NCP, false>, grid, dim3(THREADS), 0, st, p)
+               : launch_dependent(delta_step_kernel<T, DKP, THREADS, NCP, true>, grid, dim3(THREADS), sizeof(float) * p.rank, st, p);
+}
+
+struct Workspace {
+    float *z, *o;
+    void* th;
+    size_t bytes;
+};
+Workspace carve(const tbl_delta_mixer& m, int precision, size_t rows, void* base) {
+    Workspace w{};
+    const size_t HD = static_cast<size_t>(m.heads) * m.dim, e = precision == TBL_BF16 ? 2 : 4;
+    uint8_t* p = static_cast<uint8_t*>(base);
+    auto take = [&](size_t bytes) { uint8_t* r = p + w.bytes; w.bytes += round_up(bytes, 256); return r; };
+    w.z = reinterpret_cast<float*>(take(sizeof(float) * rows * HD));
+    w.o = reinterpret_cast<float*>(take(sizeof(float) * rows * HD));
+    w.th = take(e * rows * round_up(m.rank, 8));
+    return w;
 }
 
 template <typename T>
-int launch_step(const DeltaParams& p, int n_seq, cudaStream_t st) {
+int launch_step(const tbl_delta_mixer& m, DeltaParams p, int precision, int n_seq, void* ws, cudaStream_t st) {
     const dim3 grid(p.heads, n_seq);
-    const size_t smem = sizeof(float) * p.rank;
-    if (n_seq > 65535 || smem > 32 * 1024) return TBL_ERR_SHAPE;
+    if (n_seq > 65535 || p.rank > 8192) return TBL_ERR_SHAPE;
+    if (n_seq >= kStepFusedRows) {
+        const Workspace w = carve(m, precision, n_seq, ws);
+        const int rc = decay_products<T>(m, p, precision, n_seq, static_cast<T*>(w.th), w.z, st);
+        if (rc != TBL_OK) return rc;
+        p.z = w.z;
+    }
     cudaError_t e;
-    if (p.dim <= 32) e = launch_dependent(delta_step_kernel<T, 32, 256, 1>, grid, dim3(256), smem, st, p);
-    else if (p.dim <= 64) e = launch_dependent(delta_step_kernel<T, 64, 256, 2>, grid, dim3(256), smem, st, p);
-    else if (p.dim <= 128) e = launch_dependent(delta_step_kernel<T, 128, 256, 4>, grid, dim3(256), smem, st, p);
-    else e = launch_dependent(delta_step_kernel<T, 256, 512, 1>, grid, dim3(512), smem, st, p);
+    if (p.dim <= 32) e = launch_step_d<T, 32, 256, 1>(p, grid, st);
+    else if (p.dim <= 64) e = launch_step_d<T, 64, 256, 2>(p, grid, st);
+    else if (p.dim <= 128) e = launch_step_d<T, 128, 256, 4>(p, grid, st);
+    else e = launch_step_d<T, 256, 512, 1>(p, grid, st);
     return e == cudaSuccess ? TBL_OK : TBL_ERR_CUDA;
 }
 
@@ -390,22 +459,12 @@ int launch_scan_d(const DeltaParams& p, int n_seq, cudaStream_t st) {
 
 template <typename T>
 int launch_scan(const tbl_delta_mixer& m, DeltaParams p, int precision, int n_seq, void* ws, cudaStream_t st) {
-    const int rows = n_seq * p.n_tok, HD = p.heads * p.dim, ldt = static_cast<int>(round_up(p.rank, 8));
-    uint8_t* base = static_cast<uint8_t*>(ws);
-    float* z = reinterpret_cast<float*>(base);
-    base += round_up(sizeof(float) * static_cast<size_t>(rows) * HD, 256);
-    p.o = reinterpret_cast<float*>(base);
-    base += round_up(sizeof(float) * static_cast<size_t>(rows) * HD, 256);
-    T* th = reinterpret_cast<T*>(base);
-    if (launch_dependent(delta_tanh_kernel<T>, dim3(ceil_div(static_cast<long long>(rows) * p.rank, 256)), dim3(256), 0, st, p.proj, p.ld, 5 * HD,
-                         rows, p.rank, ldt, th) != cudaSuccess)
-        return TBL_ERR_CUDA;
-    DenseCall c{};
-    c.x = th; c.w = static_cast<const bf16*>(m.decay_up.weight); c.ldx = ldt; c.M = rows; c.K = p.rank; c.N = HD;
-    c.out_f32 = z; c.ldo = HD;
-    int rc = launch_dense(precision, kDenseAuto, c, st);
+    const int rows = n_seq * p.n_tok;
+    const Workspace w = carve(m, precision, rows, ws);
+    p.o = w.o;
+    int rc = decay_products<T>(m, p, precision, rows, static_cast<T*>(w.th), w.z, st);
     if (rc != TBL_OK) return rc;
-    p.z = z;
+    p.z = w.z;
     if (p.dim <= 32) rc = launch_scan_d<32>(p, n_seq, st);
     else if (p.dim <= 64) rc = launch_scan_d<64>(p, n_seq, st);
     else if (p.dim <= 128) rc = launch_scan_d<128>(p, n_seq, st);
@@ -427,10 +486,7 @@ int check_delta(const tbl_delta_mixer& m, int width) {
     return TBL_OK;
 }
 
-size_t delta_workspace(const tbl_delta_mixer& m, int precision, int rows) {
-    const size_t HD = static_cast<size_t>(m.heads) * m.dim, e = precision == TBL_BF16 ? 2 : 4;
-    return 2 * round_up(sizeof(float) * rows * HD, 256) + round_up(e * rows * round_up(m.rank, 8), 256);
-}
+size_t delta_workspace(const tbl_delta_mixer& m, int precision, int rows) { return carve(m, precision, rows, nullptr).bytes; }
 
 int launch_delta(const tbl_delta_mixer& m, int precision, int route, float eps, const float* proj, float* states,
                  const int32_t* slots, int n_seq, int n_tok, void* out, void* ws, cudaStream_t st) {
@@ -441,7 +497,7 @@ int launch_delta(const tbl_delta_mixer& m, int precision, int route, float eps, 
     if (route == 0) route = n_tok == 1 ? 2 : 1;
     if (route == 2) {
         if (n_tok != 1) return TBL_ERR_SHAPE;
-        return precision == TBL_BF16 ? launch_step<bf16>(p, n_seq, st) : launch_step<float>(p, n_seq, st);
+        return precision == TBL_BF16 ? launch_step<bf16>(m, p, precision, n_seq, ws, st) : launch_step<float>(m, p, precision, n_seq, ws, st);
     }
     if (route != 1) return TBL_ERR_INVALID_ARG;
     return precision == TBL_BF16 ? launch_scan<bf16>(m, p, precision, n_seq, ws, st) : launch_scan<float>(m, p, precision, n_seq, ws, st);

@@ -1,5 +1,6 @@
-// Linear layers with bf16 weights: the kernel choice, the SIMT kernel (any shape, true fp32 arithmetic) and the
-// weight-streaming GEMV for a few rows.  The tensor-core GEMM is in dense_tcgen05.cu.
+// Linear layers with bf16 weights: the kernel choice, the SIMT kernel (any shape, true fp32 arithmetic) and the fp32
+// GEMV for a few rows.  The weight-streaming kernel for bf16 rows is in dense_rows.cu, the tcgen05 GEMM in
+// dense_tcgen05.cu.
 #include "stack.cuh"
 
 namespace tbl {
@@ -210,6 +211,8 @@ bool gemv_supported(const DenseCall& c) {
     return c.M <= kGemvMaxRows && sizeof(float) * c.M * c.K <= kGemvMaxSmem && (c.K % 4 == 0 || c.M == 1);
 }
 
+constexpr int kRowsMax = 32;      // rows up to which streaming the weights through warp-level MMAs beats the tcgen05 GEMM
+
 }  // namespace
 
 int launch_dense(int precision, int route, const DenseCall& call, cudaStream_t st) {
@@ -217,7 +220,13 @@ int launch_dense(int precision, int route, const DenseCall& call, cudaStream_t s
     DenseCall c = call;
     if (c.ldw == 0) c.ldw = c.K;
     const bool tensor = precision == TBL_BF16 && dense_tensor_supported(c);
-    if (route == kDenseAuto) route = gemv_supported(c) ? kDenseGemv : (tensor ? kDenseTensor : kDenseSimt);
+    const bool rows = precision == TBL_BF16 && dense_rows_supported(c);
+    if (route == kDenseAuto)
+        route = rows && c.M <= kRowsMax ? kDenseRows : (gemv_supported(c) ? kDenseGemv : (tensor ? kDenseTensor : kDenseSimt));
+    if (route == kDenseRows) {
+        if (!rows) return TBL_ERR_SHAPE;
+        return launch_dense_rows(c, st) == cudaSuccess ? TBL_OK : TBL_ERR_CUDA;
+    }
     if (route == kDenseTensor) {
         if (!tensor) return TBL_ERR_SHAPE;
         return launch_dense_tensor(c, st) == cudaSuccess ? TBL_OK : TBL_ERR_CUDA;

@@ -35,6 +35,12 @@ __device__ __forceinline__ uint32_t pack_bf16(float lo, float hi) {
     return *reinterpret_cast<const uint32_t*>(&v);
 }
 
+// warp-level MMA 16 x 8 x 16, bf16 operands, fp32 accumulators
+__device__ __forceinline__ void mma16816(float (&d)[4], uint32_t a0, uint32_t a1, uint32_t a2, uint32_t a3, uint32_t b0, uint32_t b1) {
+    asm volatile("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0,%1,%2,%3}, {%4,%5,%6,%7}, {%8,%9}, {%0,%1,%2,%3};"
+                 : "+f"(d[0]), "+f"(d[1]), "+f"(d[2]), "+f"(d[3]) : "r"(a0), "r"(a1), "r"(a2), "r"(a3), "r"(b0), "r"(b1));
+}
+
 __device__ __forceinline__ float warp_sum(float v) {
 #pragma unroll
     for (int o = 16; o; o >>= 1) v += __shfl_xor_sync(0xffffffffu, v, o);
@@ -85,9 +91,16 @@ struct DenseCall {
     const float* residual;   // fp32, ld = ldo, added to out_f32 (may alias it); null: none
     int pair_cols;           // > 0: rows of w alternate in blocks of 32 gate / 32 up rows, out = silu(gate) * up,
                              //      clipped at this many columns
+    // row-streaming kernel only: `batch` products of one launch (0: one), their strides in elements, and an output
+    // gate: out *= sigmoid(gate[m * ldg + n])
+    int batch, ldg, batch_gate;
+    long long batch_w, batch_x, batch_out;
+    const float* gate;
 };
-enum DenseRoute { kDenseAuto = 0, kDenseSimt = 1, kDenseGemv = 2, kDenseTensor = 3 };
+enum DenseRoute { kDenseAuto = 0, kDenseSimt = 1, kDenseGemv = 2, kDenseTensor = 3, kDenseRows = 4 };
 int launch_dense(int precision, int route, const DenseCall& c, cudaStream_t st);
+bool dense_rows_supported(const DenseCall& c);
+cudaError_t launch_dense_rows(const DenseCall& c, cudaStream_t st);
 bool dense_tensor_supported(const DenseCall& c);
 cudaError_t launch_dense_tensor(const DenseCall& c, cudaStream_t st);
 

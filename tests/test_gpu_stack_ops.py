@@ -9,7 +9,7 @@ from oracle import layer_stack as O
 
 pytestmark = pytest.mark.gpu
 
-SIMT, GEMV, TENSOR = 1, 2, 3
+SIMT, GEMV, TENSOR, ROWS = 1, 2, 3, 4
 DELTA_SCAN, DELTA_STEP = 1, 2
 CACHE_SIMT, CACHE_TENSOR, EXPANDED = 1, 2, 3
 
@@ -53,8 +53,8 @@ def assert_close(got, want, rel, what=""):
 
 
 # ---- linear layers ------------------------------------------------------------------------------------------------------
-@pytest.mark.parametrize("route,precision", [(SIMT, 0), (SIMT, 1), (GEMV, 0), (GEMV, 1), (TENSOR, 1), (0, 0), (0, 1)])
-@pytest.mark.parametrize("m,k,n", [(1, 64, 40), (3, 200, 77), (4, 1032, 5000), (2, 36, 9), (1, 37, 19), (5, 24, 8), (70, 72, 130), (129, 520, 257),
+@pytest.mark.parametrize("route,precision", [(SIMT, 0), (SIMT, 1), (GEMV, 0), (GEMV, 1), (TENSOR, 1), (ROWS, 1), (0, 0), (0, 1)])
+@pytest.mark.parametrize("m,k,n", [(1, 64, 40), (8, 2048, 48), (13, 200, 100), (27, 4104, 33), (64, 264, 38000), (3, 200, 77), (4, 1032, 5000), (2, 36, 9), (1, 37, 19), (5, 24, 8), (70, 72, 130), (129, 520, 257),
                                    (300, 264, 700)])
 def test_dense(cuda, stack_lib, route, precision, m, k, n):
     torch, rng = cuda, np.random.default_rng(m * k + n)
@@ -68,12 +68,13 @@ def test_dense(cuda, stack_lib, route, precision, m, k, n):
         out = torch.full((m, n), float("nan"), device="cuda")
         rc = stack_lib.tbl_dense_forward(C.byref(v), precision, route, x.data_ptr(), ldx, m, b.f32(res) if with_extras else None,
                                          out.data_ptr(), stream(torch))
-        if (route == GEMV and (m > 4 or (k % 4 and m > 1))) or (route == TENSOR and k % 8):
+        if (route == GEMV and (m > 4 or (k % 4 and m > 1))) or (route in (TENSOR, ROWS) and k % 8):
             assert rc == -2
             return
         assert rc == 0
         want = O.linear(f64(x)[:, :k], f64(w), bias if with_extras else None) + (res if with_extras else 0.0)
-        assert_close(f64(out), want, 3e-6, "dense")
+        # (the tensor cores' fp32 accumulators drop the bits they shift out, which adds up with K)
+        assert_close(f64(out), want, 1e-5 if precision else 3e-6, "dense")
 
 
 def test_dense_tall_tiles_and_the_residual_in_place(cuda, stack_lib):
@@ -85,11 +86,11 @@ def test_dense_tall_tiles_and_the_residual_in_place(cuda, stack_lib):
     out = torch.randn(m, n, device="cuda")
     want = out.double() + x.double() @ w.cuda().double().T
     assert stack_lib.tbl_dense_forward(C.byref(b.view(w)), 1, TENSOR, x.data_ptr(), k, m, out.data_ptr(), out.data_ptr(), stream(torch)) == 0
-    assert float((out.double() - want).abs().max() / want.abs().max()) < 3e-6
+    assert float((out.double() - want).abs().max() / want.abs().max()) < 1e-5
 
 
-@pytest.mark.parametrize("route,precision", [(SIMT, 0), (GEMV, 0), (GEMV, 1), (SIMT, 1), (TENSOR, 1)])
-@pytest.mark.parametrize("m,k,ff", [(1, 64, 32), (3, 40, 37), (4, 128, 200), (1, 1024, 3000), (150, 72, 100), (260, 136, 333)])
+@pytest.mark.parametrize("route,precision", [(SIMT, 0), (GEMV, 0), (GEMV, 1), (SIMT, 1), (TENSOR, 1), (ROWS, 1)])
+@pytest.mark.parametrize("m,k,ff", [(9, 512, 70), (1, 64, 32), (3, 40, 37), (4, 128, 200), (1, 1024, 3000), (150, 72, 100), (260, 136, 333)])
 def test_gated_dense(cuda, stack_lib, route, precision, m, k, ff):
     from reimagined_b200.stack import StackEngine
     torch, rng = cuda, np.random.default_rng(ff)
