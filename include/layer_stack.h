@@ -59,6 +59,8 @@ typedef struct tbl_delta_mixer {
  * [rope_positions, rot_dim/2]: entry i rotates dimension i with i + rot_dim/2. */
 typedef struct tbl_latent_mixer {
     tbl_dense_view in, uq, uk, uv, out;
+    const void* uk_t;                /* bf16 [heads][kv_rank][dim]: W_uk once more, transposed per head; NULL: the
+                                        attention over the latent cache stays off the tensor cores */
     const float *q_norm, *kv_norm;   /* [q_rank], [kv_rank]                      */
     const float *rope_cos, *rope_sin;
     int heads, dim, rot_dim, vdim, q_rank, kv_rank, rope_positions;

@@ -100,7 +100,7 @@ class LatentMixer(C.Structure):
     """tbl_latent_mixer."""
 
     _fields_ = [("in_", DenseView), ("uq", DenseView), ("uk", DenseView), ("uv", DenseView), ("out", DenseView),
-                ("q_norm", C.c_void_p), ("kv_norm", C.c_void_p), ("rope_cos", C.c_void_p), ("rope_sin", C.c_void_p),
+                ("uk_t", C.c_void_p), ("q_norm", C.c_void_p), ("kv_norm", C.c_void_p), ("rope_cos", C.c_void_p), ("rope_sin", C.c_void_p),
                 ("heads", C.c_int), ("dim", C.c_int), ("rot_dim", C.c_int), ("vdim", C.c_int), ("q_rank", C.c_int),
                 ("kv_rank", C.c_int), ("rope_positions", C.c_int), ("scale", C.c_float)]
 

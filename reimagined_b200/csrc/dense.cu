@@ -211,7 +211,11 @@ bool gemv_supported(const DenseCall& c) {
     return c.M <= kGemvMaxRows && sizeof(float) * c.M * c.K <= kGemvMaxSmem && (c.K % 4 == 0 || c.M == 1);
 }
 
-constexpr int kRowsMax = 32;      // rows up to which streaming the weights through warp-level MMAs beats the tcgen05 GEMM
+// Streaming the weights through warp-level MMAs beats the tcgen05 GEMM up to 16 rows, on narrow layers (too few tiles for
+// the GEMM to fill the GPU) longer.
+bool rows_pay(const DenseCall& c) {
+    return c.batch > 0 || c.M <= 16 || static_cast<long long>(c.M) * c.N <= 32 * 4096;
+}
 
 }  // namespace
 
@@ -222,7 +226,7 @@ int launch_dense(int precision, int route, const DenseCall& call, cudaStream_t s
     const bool tensor = precision == TBL_BF16 && dense_tensor_supported(c);
     const bool rows = precision == TBL_BF16 && dense_rows_supported(c);
     if (route == kDenseAuto)
-        route = rows && c.M <= kRowsMax ? kDenseRows : (gemv_supported(c) ? kDenseGemv : (tensor ? kDenseTensor : kDenseSimt));
+        route = rows && rows_pay(c) ? kDenseRows : (gemv_supported(c) ? kDenseGemv : (tensor ? kDenseTensor : kDenseSimt));
     if (route == kDenseRows) {
         if (!rows) return TBL_ERR_SHAPE;
         return launch_dense_rows(c, st) == cudaSuccess ? TBL_OK : TBL_ERR_CUDA;

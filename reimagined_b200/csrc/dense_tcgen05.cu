@@ -3,8 +3,9 @@
 // bf16, in the 128-byte-swizzled K-major layout TMA writes; an MMA takes 32 bytes of K).
 //
 // One persistent CTA per SM, ten warps: TMA producer, MMA issuer (tcgen05.mma kind::f16, fp32 accumulators in TMEM,
-// two buffers of BN columns), eight epilogue warps.  MT = 1: 128 x BN tiles, the two accumulators double-buffer
-// tiles.  MT = 2: 256 x 256 tiles, two M = 128 MMAs per weight box, the accumulators are the halves of one tile.
+// two buffers of BN columns), eight epilogue warps.  128 x BN tiles; the two accumulators double-buffer tiles.  (256 x
+// 256 tiles, which the int8 kernel uses for large problems, gain nothing here: these epilogues -- residual, gated pair --
+// are longer, and a tall tile cannot hide them.)
 // The epilogue adds the bias and either adds the fp32 residual and stores fp32, stores bf16, or -- for a gated
 // feed-forward, whose weight rows alternate in blocks of 32 gate and 32 up rows -- combines two neighbouring
 // 32-column blocks into silu(gate) * up and stores that.
@@ -29,9 +30,9 @@ constexpr int kMaxStages = 8;
 constexpr int kEpiWarps = 8;
 constexpr int kThreads = 32 * (2 + kEpiWarps);
 
-__host__ __device__ constexpr int stages_for(int bn, int mt) { return mt == 2 ? 3 : (bn >= 256 ? 4 : (bn >= 128 ? 6 : 8)); }
-constexpr size_t smem_for(int bn, int mt) {
-    return 1024 + static_cast<size_t>(stages_for(bn, mt)) * (mt * BM * BKB + bn * BKB) + kEpiWarps * 4096 + 256;
+__host__ __device__ constexpr int stages_for(int bn) { return bn >= 256 ? 4 : (bn >= 128 ? 6 : 8); }
+constexpr size_t smem_for(int bn) {
+    return 1024 + static_cast<size_t>(stages_for(bn)) * (BM * BKB + bn * BKB) + kEpiWarps * 4096 + 256;
 }
 
 struct Params {
@@ -41,59 +42,73 @@ struct Params {
     int* status;
 };
 
-template <int MT>
 __device__ __forceinline__ bool decode_tile(const Params& p, int t, int& row0, int& tn) {
     if (t >= p.tiles_m * p.tiles_n) return false;
     const int per_group = kGroupM * p.tiles_n;
     const int grp = t / per_group, in_grp = t - grp * per_group;
     const int gm = min(kGroupM, p.tiles_m - grp * kGroupM);
     tn = in_grp / gm;
-    row0 = (grp * kGroupM + in_grp % gm) * (BM * MT);
+    row0 = (grp * kGroupM + in_grp % gm) * BM;
     return true;
 }
 
 // Stores one 32 x 32 block staged in shared memory (row = lane order, 16-byte chunk j of row r at j ^ (r & 7)).
+template <bool RES>
 __device__ __forceinline__ void store_block(const Params& p, const uint8_t* stage, int lane, int row0, int valid, int col0,
                                             int ncols) {
     const DenseCall& c = p.c;
     const int chunk = lane & 7, rsub = lane >> 3, col = col0 + 4 * chunk;
     if (col >= ncols) return;
+    if (RES && p.vec) {
+        // residual rows are requested together: one memory round trip per block, not one per row
+        float4 res[8];
+        {
+#pragma unroll
+            for (int i8 = 0; i8 < 8; ++i8) {
+                const int rr = 4 * i8 + rsub;
+                res[i8] = rr < valid ? *reinterpret_cast<const float4*>(c.residual + static_cast<size_t>(row0 + rr) * c.ldo + col)
+                                     : make_float4(0.0f, 0.0f, 0.0f, 0.0f);
+            }
+        }
+#pragma unroll
+        for (int i8 = 0; i8 < 8; ++i8) {
+            const int rr = 4 * i8 + rsub;
+            if (rr >= valid) continue;
+            float4 f = *reinterpret_cast<const float4*>(stage + rr * 128 + ((chunk ^ (rr & 7)) << 4));
+            f.x += res[i8].x; f.y += res[i8].y; f.z += res[i8].z; f.w += res[i8].w;
+            *reinterpret_cast<float4*>(c.out_f32 + static_cast<size_t>(row0 + rr) * c.ldo + col) = f;
+        }
+        return;
+    }
 #pragma unroll
     for (int i8 = 0; i8 < 8; ++i8) {
         const int rr = 4 * i8 + rsub;
         if (rr >= valid) continue;
-        float4 f = *reinterpret_cast<const float4*>(stage + rr * 128 + ((chunk ^ (rr & 7)) << 4));
+        const float4 f = *reinterpret_cast<const float4*>(stage + rr * 128 + ((chunk ^ (rr & 7)) << 4));
         const size_t o = static_cast<size_t>(row0 + rr) * c.ldo + col;
-        if (p.vec) {
-            if (c.out_f32) {
-                if (c.residual) {
-                    const float4 a = *reinterpret_cast<const float4*>(c.residual + o);
-                    f.x += a.x; f.y += a.y; f.z += a.z; f.w += a.w;
-                }
-                *reinterpret_cast<float4*>(c.out_f32 + o) = f;
-            } else {
-                *reinterpret_cast<uint2*>(c.out_b16 + o) = make_uint2(pack_bf16(f.x, f.y), pack_bf16(f.z, f.w));
-            }
+        if (p.vec && c.out_f32) {
+            *reinterpret_cast<float4*>(c.out_f32 + o) = f;
+        } else if (p.vec) {
+            *reinterpret_cast<uint2*>(c.out_b16 + o) = make_uint2(pack_bf16(f.x, f.y), pack_bf16(f.z, f.w));
         } else {
             const float v[4] = {f.x, f.y, f.z, f.w};
 #pragma unroll
             for (int e = 0; e < 4; ++e) {
                 if (col + e >= ncols) break;
-                if (c.out_f32) c.out_f32[o + e] = c.residual ? c.residual[o + e] + v[e] : v[e];
+                if (c.out_f32) c.out_f32[o + e] = RES ? c.residual[o + e] + v[e] : v[e];
                 else c.out_b16[o + e] = __float2bfloat16_rn(v[e]);
             }
         }
     }
 }
 
-template <int BN, int MT>
+template <int BN, bool RES>
 __global__ void __launch_bounds__(kThreads, 1)
 dense_tcgen05_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_constant__ CUtensorMap map_b, const Params p) {
     extern __shared__ __align__(1024) uint8_t smem_raw[];
     uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~uintptr_t(1023));
-    static_assert(MT == 1 || BN == 256, "tall tiles are 256 x 256");
-    constexpr int kStages = stages_for(BN, MT);
-    constexpr int kABytes = MT * BM * BKB;
+    constexpr int kStages = stages_for(BN);
+    constexpr int kABytes = BM * BKB;
     constexpr int kBBytes = BN * BKB;
     constexpr int kStageBytes = kABytes + kBBytes;
     constexpr uint32_t kTmemCols = 2 * BN;
@@ -130,7 +145,7 @@ dense_tcgen05_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_con
         if (lane == 0) {
             int it = 0, row0, tn;
             bool alive = true;
-            for (int tile = blockIdx.x; alive && decode_tile<MT>(p, tile, row0, tn); tile += gridDim.x) {
+            for (int tile = blockIdx.x; alive && decode_tile(p, tile, row0, tn); tile += gridDim.x) {
                 for (int kb = 0; kb < kblocks; ++kb, ++it) {
                     const int s = it % kStages;
                     if (it >= kStages) {
@@ -140,7 +155,6 @@ dense_tcgen05_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_con
                     uint8_t* a_dst = smem + s * kStageBytes;
                     mbar_arrive_expect_tx(&full[s], kStageBytes);
                     tma_load_2d(a_dst, &map_a, kb * BKE, row0, &full[s]);
-                    if constexpr (MT == 2) tma_load_2d(a_dst + BM * BKB, &map_a, kb * BKE, row0 + BM, &full[s]);
                     tma_load_2d(a_dst + kABytes, &map_b, kb * BKE, tn * BN, &full[s]);
                 }
             }
@@ -151,16 +165,14 @@ dense_tcgen05_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_con
             const uint32_t idesc = idesc_bf16(BN);
             int it = 0, local = 0, row0, tn;
             bool alive = true;
-            for (int tile = blockIdx.x; alive && decode_tile<MT>(p, tile, row0, tn); tile += gridDim.x, ++local) {
+            for (int tile = blockIdx.x; alive && decode_tile(p, tile, row0, tn); tile += gridDim.x, ++local) {
                 const int buf = local & 1;
-                if constexpr (MT == 1) {
-                    if (local >= 2) {
-                        alive = mbar_wait_bounded(&tmem_empty[buf], ((local >> 1) - 1) & 1, p.status);
-                        if (!alive) break;
-                    }
+                if (local >= 2) {
+                    alive = mbar_wait_bounded(&tmem_empty[buf], ((local >> 1) - 1) & 1, p.status);
+                    if (!alive) break;
                 }
                 tc_fence_after();
-                const uint32_t d_tmem = tmem_base + (MT == 1 ? buf * BN : 0);
+                const uint32_t d_tmem = tmem_base + buf * BN;
                 for (int kb = 0; kb < kblocks; ++kb, ++it) {
                     const int s = it % kStages;
                     alive = mbar_wait_bounded(&full[s], (it / kStages) & 1, p.status);
@@ -169,31 +181,11 @@ dense_tcgen05_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_con
                     const uint32_t a_addr = smem_u32(smem + s * kStageBytes);
                     const uint32_t b_addr = a_addr + kABytes;
 #pragma unroll
-                    for (int h = 0; h < MT; ++h) {
-                        if constexpr (MT == 2) {
-                            // a half is waited for just before the first MMA that writes it: the epilogue drains half 0 first
-                            if (kb == 0 && local >= 1) {
-                                alive = mbar_wait_bounded(&tmem_empty[h], (local - 1) & 1, p.status);
-                                if (!alive) break;
-                                tc_fence_after();
-                            }
-                        }
-#pragma unroll
-                        for (int kk = 0; kk < BKB / 32; ++kk)
-                            umma_f16(d_tmem + h * BN, smem_desc_sw128(a_addr + h * (BM * BKB) + kk * 32),
-                                     smem_desc_sw128(b_addr + kk * 32), idesc, (kb | kk) != 0 ? 1u : 0u);
-                    }
-                    if (!alive) break;
+                    for (int kk = 0; kk < BKB / 32; ++kk)
+                        umma_f16(d_tmem, smem_desc_sw128(a_addr + kk * 32), smem_desc_sw128(b_addr + kk * 32), idesc, (kb | kk) != 0 ? 1u : 0u);
                     umma_commit(&empty[s]);
                 }
-                if (alive) {
-                    if constexpr (MT == 1) {
-                        umma_commit(&tmem_full[buf]);
-                    } else {
-                        umma_commit(&tmem_full[0]);
-                        umma_commit(&tmem_full[1]);
-                    }
-                }
+                if (alive) umma_commit(&tmem_full[buf]);
             }
         }
     } else {
@@ -204,68 +196,66 @@ dense_tcgen05_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_con
         const bool pair = p.c.pair_cols > 0;
         int local = 0, tile_row0, tn;
         bool alive = true;
-        for (int tile = blockIdx.x; alive && decode_tile<MT>(p, tile, tile_row0, tn); tile += gridDim.x, ++local) {
-            for (int h = 0; h < MT && alive; ++h) {
-                const int buf = MT == 1 ? (local & 1) : h;
-                alive = mbar_wait_bounded(&tmem_full[buf], (MT == 1 ? (local >> 1) : local) & 1, p.status);
-                alive = __all_sync(0xffffffffu, alive);
-                if (!alive) break;
-                tc_fence_after();
-                const int row0 = tile_row0 + h * BM + quarter * 32;
-                const int valid = min(32, p.c.M - row0);
-                const uint32_t t_row = tmem_base + (static_cast<uint32_t>(quarter * 32) << 16) + buf * BN;
-                const int nblocks = min(BN / 32, (p.c.N - tn * BN + 31) / 32);
-                // blocks of 32 columns: every other one is this warp's -- of a gated layer every other pair
-                const int step = pair ? 2 : 1;
-                uint32_t r[32], rn[32];
-                if (half * step < nblocks) tmem_ld32(t_row + half * step * 32, r);
+        for (int tile = blockIdx.x; alive && decode_tile(p, tile, tile_row0, tn); tile += gridDim.x, ++local) {
+            const int buf = local & 1;
+            alive = mbar_wait_bounded(&tmem_full[buf], (local >> 1) & 1, p.status);
+            alive = __all_sync(0xffffffffu, alive);
+            if (!alive) break;
+            tc_fence_after();
+            const int row0 = tile_row0 + quarter * 32;
+            const int valid = min(32, p.c.M - row0);
+            const uint32_t t_row = tmem_base + (static_cast<uint32_t>(quarter * 32) << 16) + buf * BN;
+            const int nblocks = min(BN / 32, (p.c.N - tn * BN + 31) / 32);
+            // blocks of 32 columns: every other one is this warp's -- of a gated layer every other pair
+            const int step = pair ? 2 : 1;
+            uint32_t r[32], rn[32];
+            if (half * step < nblocks) tmem_ld32(t_row + half * step * 32, r);
 #pragma unroll 1
-                for (int b = half * step; b < nblocks; b += 2 * step) {
-                    const int n0 = tn * BN + b * 32;
-                    const float bias_l = p.c.bias && n0 + lane < p.c.N ? __ldg(p.c.bias + n0 + lane) : 0.0f;
-                    int col0 = n0, ncols = p.c.N;
-                    float v[32];
+            for (int b = half * step; b < nblocks; b += 2 * step) {
+                const int n0 = tn * BN + b * 32;
+                const float bias_l = p.c.bias && n0 + lane < p.c.N ? __ldg(p.c.bias + n0 + lane) : 0.0f;
+                int col0 = n0, ncols = p.c.N;
+                float v[32];
+                tmem_ld_wait();
+                if (pair) {
+                    tmem_ld32(t_row + (b + 1) * 32, rn);      // N is a multiple of 64
+                    const float bias_u = p.c.bias ? __ldg(p.c.bias + n0 + 32 + lane) : 0.0f;
                     tmem_ld_wait();
-                    if (pair) {
-                        tmem_ld32(t_row + (b + 1) * 32, rn);      // N is a multiple of 64
-                        const float bias_u = p.c.bias ? __ldg(p.c.bias + n0 + 32 + lane) : 0.0f;
-                        tmem_ld_wait();
 #pragma unroll
-                        for (int i = 0; i < 32; ++i) {
-                            const float g = __uint_as_float(r[i]) + __shfl_sync(0xffffffffu, bias_l, i);
-                            const float u = __uint_as_float(rn[i]) + __shfl_sync(0xffffffffu, bias_u, i);
-                            v[i] = silu_f(g) * u;
-                        }
-                        if (b + 4 < nblocks) tmem_ld32(t_row + (b + 4) * 32, r);
-                        col0 = n0 >> 1;
-                        ncols = p.c.pair_cols;
-                    } else {
-                        if (b + 2 < nblocks) tmem_ld32(t_row + (b + 2) * 32, rn);   // in flight while this block is stored
-                        if (p.c.bias) {
-#pragma unroll
-                            for (int i = 0; i < 32; ++i) v[i] = __uint_as_float(r[i]) + __shfl_sync(0xffffffffu, bias_l, i);
-                        } else {
-#pragma unroll
-                            for (int i = 0; i < 32; ++i) v[i] = __uint_as_float(r[i]);
-                        }
+                    for (int i = 0; i < 32; ++i) {
+                        const float g = __uint_as_float(r[i]) + __shfl_sync(0xffffffffu, bias_l, i);
+                        const float u = __uint_as_float(rn[i]) + __shfl_sync(0xffffffffu, bias_u, i);
+                        v[i] = silu_f(g) * u;
                     }
-                    __syncwarp();
+                    if (b + 4 < nblocks) tmem_ld32(t_row + (b + 4) * 32, r);
+                    col0 = n0 >> 1;
+                    ncols = p.c.pair_cols;
+                } else {
+                    if (b + 2 < nblocks) tmem_ld32(t_row + (b + 2) * 32, rn);   // in flight while this block is stored
+                    if (p.c.bias) {
 #pragma unroll
-                    for (int j = 0; j < 8; ++j)
-                        *reinterpret_cast<float4*>(stage + lane * 128 + ((j ^ (lane & 7)) << 4)) =
-                            make_float4(v[4 * j], v[4 * j + 1], v[4 * j + 2], v[4 * j + 3]);
-                    __syncwarp();
-                    if (valid > 0) store_block(p, stage, lane, row0, valid, col0, ncols);
-                    if (!pair) {
+                        for (int i = 0; i < 32; ++i) v[i] = __uint_as_float(r[i]) + __shfl_sync(0xffffffffu, bias_l, i);
+                    } else {
 #pragma unroll
-                        for (int i = 0; i < 32; ++i) r[i] = rn[i];
+                        for (int i = 0; i < 32; ++i) v[i] = __uint_as_float(r[i]);
                     }
                 }
-                tmem_ld_wait();
-                tc_fence_before();
                 __syncwarp();
-                if (lane == 0) mbar_arrive(&tmem_empty[buf]);
+#pragma unroll
+                for (int j = 0; j < 8; ++j)
+                    *reinterpret_cast<float4*>(stage + lane * 128 + ((j ^ (lane & 7)) << 4)) =
+                        make_float4(v[4 * j], v[4 * j + 1], v[4 * j + 2], v[4 * j + 3]);
+                __syncwarp();
+                if (valid > 0) store_block<RES>(p, stage, lane, row0, valid, col0, ncols);
+                if (!pair) {
+#pragma unroll
+                    for (int i = 0; i < 32; ++i) r[i] = rn[i];
+                }
             }
+            tmem_ld_wait();
+            tc_fence_before();
+            __syncwarp();
+            if (lane == 0) mbar_arrive(&tmem_empty[buf]);
         }
     }
 
@@ -278,15 +268,19 @@ dense_tcgen05_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_con
     }
 }
 
-template <int BN, int MT>
-cudaError_t launch_bn(const CUtensorMap& ma, const CUtensorMap& mb, const Params& p, cudaStream_t st) {
+template <int BN, bool RES>
+cudaError_t launch_kernel(const CUtensorMap& ma, const CUtensorMap& mb, const Params& p, cudaStream_t st) {
     static bool done[64] = {};
-    constexpr size_t smem = smem_for(BN, MT);
+    constexpr size_t smem = smem_for(BN);
     static_assert(smem <= 227 * 1024, "shared memory of a CTA");
-    const cudaError_t e = allow_smem(dense_tcgen05_kernel<BN, MT>, smem, done);
+    const cudaError_t e = allow_smem(dense_tcgen05_kernel<BN, RES>, smem, done);
     if (e != cudaSuccess) return e;
     const int tiles = p.tiles_m * p.tiles_n;
-    return launch_dependent(dense_tcgen05_kernel<BN, MT>, dim3(tiles < kNumSm ? tiles : kNumSm), dim3(kThreads), smem, st, ma, mb, p);
+    return launch_dependent(dense_tcgen05_kernel<BN, RES>, dim3(tiles < kNumSm ? tiles : kNumSm), dim3(kThreads), smem, st, ma, mb, p);
+}
+template <int BN>
+cudaError_t launch_bn(const CUtensorMap& ma, const CUtensorMap& mb, const Params& p, cudaStream_t st) {
+    return p.c.residual ? launch_kernel<BN, true>(ma, mb, p, st) : launch_kernel<BN, false>(ma, mb, p, st);
 }
 
 }  // namespace
@@ -304,28 +298,23 @@ cudaError_t launch_dense_tensor(const DenseCall& c, cudaStream_t st) {
     const int cols = c.pair_cols ? c.pair_cols : c.N;
     p.vec = (cols % 4 == 0) && (c.ldo % 4 == 0) && (reinterpret_cast<uintptr_t>(c.out_f32) & 15) == 0 &&
             (reinterpret_cast<uintptr_t>(c.out_b16) & 7) == 0 && (reinterpret_cast<uintptr_t>(c.residual) & 15) == 0;
-    // tall tiles for at least a wave of them, otherwise the widest tile that fills the SMs
-    const long long tall_tiles = static_cast<long long>((c.M + 2 * BM - 1) / (2 * BM)) * ((c.N + 255) / 256);
-    const bool tall = c.N >= 256 && (tall_tiles >= 4 * kNumSm || (tall_tiles >= kNumSm && c.K >= 2048));
+    // the widest tile that fills the SMs
     int bn = c.N > 128 ? 256 : (c.N > 64 ? 128 : 64);
-    if (!tall) {
-        const long long tm = (c.M + BM - 1) / BM;
-        auto tiles = [&](int b) { return tm * ((c.N + b - 1) / b); };
-        auto fill = [&](int b) {
-            const long long t = tiles(b);
-            return static_cast<double>(t) / (static_cast<double>((t + kNumSm - 1) / kNumSm) * kNumSm);
-        };
-        if (bn == 256 && fill(128) > 1.15 * fill(256)) bn = 128;
-        if (bn == 128 && tiles(128) < 100 && c.N > 64) bn = 64;
-    }
-    p.tiles_m = tall ? (c.M + 2 * BM - 1) / (2 * BM) : (c.M + BM - 1) / BM;
+    const long long tm = (c.M + BM - 1) / BM;
+    auto tiles = [&](int b) { return tm * ((c.N + b - 1) / b); };
+    auto fill = [&](int b) {
+        const long long t = tiles(b);
+        return static_cast<double>(t) / (static_cast<double>((t + kNumSm - 1) / kNumSm) * kNumSm);
+    };
+    if (bn == 256 && fill(128) > 1.15 * fill(256)) bn = 128;
+    if (bn == 128 && tiles(128) < 100 && c.N > 64) bn = 64;
+    p.tiles_m = static_cast<int>(tm);
     p.tiles_n = (c.N + bn - 1) / bn;
     CUtensorMap ma, mb;
     if (!make_map(&ma, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, c.x, c.M, c.K, BKE, BM, CU_TENSOR_MAP_SWIZZLE_128B, c.ldx))
         return cudaErrorUnknown;
     if (!make_map(&mb, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, c.w, c.N, c.K, BKE, bn, CU_TENSOR_MAP_SWIZZLE_128B, c.ldw)) return cudaErrorUnknown;
-    if (tall) return launch_bn<256, 2>(ma, mb, p, st);
-    return bn == 256 ? launch_bn<256, 1>(ma, mb, p, st) : (bn == 128 ? launch_bn<128, 1>(ma, mb, p, st) : launch_bn<64, 1>(ma, mb, p, st));
+    return bn == 256 ? launch_bn<256>(ma, mb, p, st) : (bn == 128 ? launch_bn<128>(ma, mb, p, st) : launch_bn<64>(ma, mb, p, st));
 }
 
 }  // namespace stack

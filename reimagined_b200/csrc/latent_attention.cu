@@ -2,7 +2,7 @@
 // heads, so a token costs kv_rank + rot_dim cached numbers whatever the head count.
 //
 //   latent_prep_kernel     norms of the query latent and of the cached latent, rotation of the shared key part, append
-//   latent_absorb_kernel   query side of W_uk: q' = W_uk^T q per head (and the rotation of the query's rotated part), so
+//   latent_absorb_kernel   (fp32 and odd sizes) query side of W_uk: q' = W_uk^T q per head (and the rotation of the query's rotated part), so
 //                          that scores are dot products with the cache itself
 //   latent_simt_kernel     attention over the cache, any sizes, fp32 arithmetic; split over the context
 //   latent_value_kernel    merges the splits, applies W_uv per head and the output gate
@@ -13,10 +13,12 @@ namespace tbl {
 namespace stack {
 namespace {
 
-// One CTA per row of the step.
+// One CTA per row of the step; a thread keeps its numbers in registers between the sum of squares and the stores.
+constexpr int kPrepThreads = 256, kPrepQ = 8, kPrepC = TBL_MAX_LATENT / kPrepThreads;
+
 template <typename T>
-__global__ void __launch_bounds__(128) latent_prep_kernel(const LatentParams p) {
-    __shared__ float red[2][4];
+__global__ void __launch_bounds__(kPrepThreads) latent_prep_kernel(const LatentParams p) {
+    __shared__ float red[2][kPrepThreads / 32];
     pdl_launch_dependents();
     pdl_wait();
     const int row = blockIdx.x, tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
@@ -24,31 +26,52 @@ __global__ void __launch_bounds__(128) latent_prep_kernel(const LatentParams p) 
     const int pos = p.positions[slot] + row % p.n_tok;
     const float* pr = p.proj + static_cast<size_t>(row) * p.ld;
     const float* kv = pr + p.q_rank;
-    float sq = 0.0f, sc = 0.0f;
-    for (int e = tid; e < p.q_rank; e += 128) sq = fmaf(pr[e], pr[e], sq);
-    for (int e = tid; e < p.R; e += 128) sc = fmaf(kv[e], kv[e], sc);
+    float q[kPrepQ], c[kPrepC], sq = 0.0f, sc = 0.0f;
+#pragma unroll
+    for (int i = 0; i < kPrepQ; ++i) { const int e = tid + i * kPrepThreads; q[i] = e < p.q_rank ? pr[e] : 0.0f; }
+#pragma unroll
+    for (int i = 0; i < kPrepC; ++i) { const int e = tid + i * kPrepThreads; c[i] = e < p.R ? kv[e] : 0.0f; }
+    const bool room = pos >= 0 && pos < p.capacity && pos < p.rope_positions;
+    const int half = p.rd / 2, at = room ? pos : 0;
+    float u = 0.0f, v = 0.0f, cv = 0.0f, sv = 0.0f;
+    if (tid < half) {                                      // rd <= TBL_MAX_LATENT: one pair per thread for up to 512 dimensions
+        u = kv[p.R + tid]; v = kv[p.R + tid + half];
+        cv = __ldg(p.rope_cos + static_cast<size_t>(at) * half + tid); sv = __ldg(p.rope_sin + static_cast<size_t>(at) * half + tid);
+    }
+#pragma unroll
+    for (int i = 0; i < kPrepQ; ++i) sq = fmaf(q[i], q[i], sq);
+    for (int e = tid + kPrepQ * kPrepThreads; e < p.q_rank; e += kPrepThreads) sq = fmaf(pr[e], pr[e], sq);
+#pragma unroll
+    for (int i = 0; i < kPrepC; ++i) sc = fmaf(c[i], c[i], sc);
     sq = warp_sum(sq);
     sc = warp_sum(sc);
     if (lane == 0) { red[0][warp] = sq; red[1][warp] = sc; }
     __syncthreads();
-    sq = (red[0][0] + red[0][1]) + (red[0][2] + red[0][3]);
-    sc = (red[1][0] + red[1][1]) + (red[1][2] + red[1][3]);
+    sq = sc = 0.0f;
+#pragma unroll
+    for (int w = 0; w < kPrepThreads / 32; ++w) { sq += red[0][w]; sc += red[1][w]; }
     const float iq = 1.0f / sqrtf(sq / static_cast<float>(p.q_rank) + p.eps);
     const float ic = 1.0f / sqrtf(sc / static_cast<float>(p.R) + p.eps);
     T* cq = static_cast<T*>(p.cq) + static_cast<size_t>(row) * p.ldq;
-    for (int e = tid; e < p.q_rank; e += 128) cq[e] = from_f<T>(pr[e] * iq * __ldg(p.q_norm + e));
-    if (pos < 0 || pos >= p.capacity || pos >= p.rope_positions) {
+#pragma unroll
+    for (int i = 0; i < kPrepQ; ++i) { const int e = tid + i * kPrepThreads; if (e < p.q_rank) cq[e] = from_f<T>(q[i] * iq * __ldg(p.q_norm + e)); }
+    for (int e = tid + kPrepQ * kPrepThreads; e < p.q_rank; e += kPrepThreads) cq[e] = from_f<T>(pr[e] * iq * __ldg(p.q_norm + e));
+    if (!room) {
         if (tid == 0) atomicOr(p.status, TBL_DEV_CACHE_FULL);
         return;
     }
-    T* c = static_cast<T*>(p.cache) + (static_cast<size_t>(slot) * p.capacity + pos) * p.cw;
-    for (int e = tid; e < p.R; e += 128) c[e] = from_f<T>(kv[e] * ic * __ldg(p.kv_norm + e));
-    const int half = p.rd / 2;
-    for (int i = tid; i < half; i += 128) {
-        const float cv = __ldg(p.rope_cos + static_cast<size_t>(pos) * half + i), sv = __ldg(p.rope_sin + static_cast<size_t>(pos) * half + i);
-        const float u = kv[p.R + i], v = kv[p.R + i + half];
-        c[p.R + i] = from_f<T>(u * cv - v * sv);
-        c[p.R + half + i] = from_f<T>(v * cv + u * sv);
+    T* out = static_cast<T*>(p.cache) + (static_cast<size_t>(slot) * p.capacity + pos) * p.cw;
+#pragma unroll
+    for (int i = 0; i < kPrepC; ++i) { const int e = tid + i * kPrepThreads; if (e < p.R) out[e] = from_f<T>(c[i] * ic * __ldg(p.kv_norm + e)); }
+    if (tid < half) {
+        out[p.R + tid] = from_f<T>(u * cv - v * sv);
+        out[p.R + half + tid] = from_f<T>(v * cv + u * sv);
+    }
+    for (int i = tid + kPrepThreads; i < half; i += kPrepThreads) {
+        const float a = kv[p.R + i], b = kv[p.R + i + half];
+        const float ci = __ldg(p.rope_cos + static_cast<size_t>(pos) * half + i), si = __ldg(p.rope_sin + static_cast<size_t>(pos) * half + i);
+        out[p.R + i] = from_f<T>(a * ci - b * si);
+        out[p.R + half + i] = from_f<T>(b * ci + a * si);
     }
 }
 
@@ -174,7 +197,7 @@ __global__ void __launch_bounds__(256) latent_value_kernel(const LatentParams p)
         for (int s = lane; s < p.splits; s += 32) m = fmaxf(m, p.part_m[unit + s]);
         m = warp_max(m);
         for (int s = lane; s < p.splits; s += 32) {
-            const float ms = p.part_m[unit + s], f = ms == -INFINITY ? 0.0f : (p.log2_parts ? exp2f(ms - m) : expf(ms - m));
+            const float ms = p.part_m[unit + s], f = ms == -INFINITY ? 0.0f : expf(ms - m);
             fac[s] = f;
             l = fmaf(p.part_l[unit + s], f, l);
         }
@@ -242,7 +265,7 @@ int pick_splits(const tbl_latent_mixer& m, int route, int rows, int context) {
 
 struct Plan {
     int route, splits;
-    size_t cq, q, qa, pm, pl, po, ek, ev, ec, bytes;      // offsets
+    size_t cq, q, qa, lat, pm, pl, po, ek, ev, ec, bytes;      // offsets
 };
 
 Plan make_plan(const tbl_latent_mixer& m, int precision, int route, int n_seq, int n_tok, int context) {
@@ -252,7 +275,8 @@ Plan make_plan(const tbl_latent_mixer& m, int precision, int route, int n_seq, i
     size_t off = 0;
     auto take = [&](size_t bytes) { const size_t at = off; off += round_up(bytes, 256); return at; };
     w.cq = take(e * rows * round_up(m.q_rank, 8));
-    w.q = take(sizeof(float) * rows * m.heads * (m.dim + m.rot_dim));
+    w.q = take((w.route == kCacheTensor ? e : sizeof(float)) * rows * m.heads * (m.dim + m.rot_dim));
+    w.lat = take(w.route == kCacheTensor ? e * rows * m.heads * m.kv_rank : 0);
     if (w.route == kExpanded) {
         const size_t padded = static_cast<size_t>(n_seq) * latent_expanded_context(context);
         w.ek = take(e * padded * m.heads * m.dim);
@@ -273,24 +297,22 @@ Plan make_plan(const tbl_latent_mixer& m, int precision, int route, int n_seq, i
 template <typename T>
 int run(const tbl_latent_mixer& m, LatentParams p, const Plan& w, int precision, int n_seq, int context, cudaStream_t st) {
     const int rows = n_seq * p.n_tok;
-    if (launch_dependent(latent_prep_kernel<T>, dim3(rows), dim3(128), 0, st, p) != cudaSuccess) return TBL_ERR_CUDA;
+    if (launch_dependent(latent_prep_kernel<T>, dim3(rows), dim3(kPrepThreads), 0, st, p) != cudaSuccess) return TBL_ERR_CUDA;
     DenseCall c{};
     c.x = p.cq; c.w = static_cast<const bf16*>(m.uq.weight); c.bias = m.uq.bias; c.ldx = p.ldq; c.M = rows; c.K = p.q_rank;
-    c.N = p.H * (p.d + p.rd); c.out_f32 = p.q; c.ldo = c.N;
+    c.N = p.H * (p.d + p.rd); c.ldo = c.N;
+    if (w.route == kCacheTensor) c.out_b16 = p.q16; else c.out_f32 = p.q;
     int rc = launch_dense(precision, kDenseAuto, c, st);
     if (rc != TBL_OK) return rc;
     if (w.route == kExpanded) {
         p.context = latent_expanded_context(context);
         return launch_latent_expanded(m, p, n_seq, st);
     }
+    if (w.route == kCacheTensor) return launch_latent_tensor(p, rows, st);
     if (launch_dependent(latent_absorb_kernel<T>, dim3(rows, p.H), dim3(128), sizeof(float) * (p.d + p.rd), st, p) != cudaSuccess)
         return TBL_ERR_CUDA;
-    if (w.route == kCacheTensor) {
-        if (launch_latent_tensor(p, rows, st) != cudaSuccess) return TBL_ERR_CUDA;
-    } else {
-        rc = launch_simt<T>(p, rows, st);
-        if (rc != TBL_OK) return rc;
-    }
+    rc = launch_simt<T>(p, rows, st);
+    if (rc != TBL_OK) return rc;
     return launch_dependent(latent_value_kernel<T>, dim3(rows, p.H), dim3(256), sizeof(float) * (p.R + p.splits), st, p) == cudaSuccess
                ? TBL_OK : TBL_ERR_CUDA;
 }
@@ -326,17 +348,17 @@ int launch_latent(const tbl_latent_mixer& m, int precision, int route, float eps
     uint8_t* base = static_cast<uint8_t*>(ws);
     LatentParams p{};
     p.proj = proj; p.q_norm = m.q_norm; p.kv_norm = m.kv_norm; p.rope_cos = m.rope_cos; p.rope_sin = m.rope_sin;
-    p.uk = static_cast<const bf16*>(m.uk.weight); p.uv = static_cast<const bf16*>(m.uv.weight);
+    p.uk = static_cast<const bf16*>(m.uk.weight); p.uk_t = static_cast<const bf16*>(m.uk_t); p.uv = static_cast<const bf16*>(m.uv.weight);
     p.cache = cache; p.slots = slots; p.positions = positions; p.out = out; p.status = device_status_ptr();
     if (!p.status) return TBL_ERR_CUDA;
-    p.cq = base + w.cq; p.q = reinterpret_cast<float*>(base + w.q); p.qa = base + w.qa;
+    p.cq = base + w.cq; p.q = reinterpret_cast<float*>(base + w.q); p.q16 = reinterpret_cast<bf16*>(base + w.q); p.lat = reinterpret_cast<bf16*>(base + w.lat); p.qa = base + w.qa;
     p.part_m = reinterpret_cast<float*>(base + w.pm); p.part_l = reinterpret_cast<float*>(base + w.pl);
     p.part_o = reinterpret_cast<float*>(base + w.po);
     p.keys = reinterpret_cast<bf16*>(base + w.ek); p.values = reinterpret_cast<bf16*>(base + w.ev);
     p.gathered = reinterpret_cast<bf16*>(base + w.ec);
     p.ld = m.in.outputs; p.ldq = static_cast<int>(round_up(m.q_rank, 8)); p.cw = latent_cache_width(m);
     p.H = m.heads; p.d = m.dim; p.rd = m.rot_dim; p.vd = m.vdim; p.R = m.kv_rank; p.q_rank = m.q_rank;
-    p.capacity = capacity; p.rope_positions = m.rope_positions; p.n_tok = n_tok; p.splits = w.splits; p.context = context; p.log2_parts = w.route == kCacheTensor;
+    p.capacity = capacity; p.rope_positions = m.rope_positions; p.n_tok = n_tok; p.splits = w.splits; p.context = context;
     p.scale = m.scale; p.eps = eps;
     return precision == TBL_BF16 ? run<bf16>(m, p, w, precision, n_seq, context, st) : run<float>(m, p, w, precision, n_seq, context, st);
 }

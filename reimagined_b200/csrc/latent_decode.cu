@@ -2,7 +2,8 @@
 // tokens is one small product with the absorbed queries (S = Q' C^T) and one with the weights (O += P C), and the cache
 // is read from memory once per head block.  The products are warp-level MMAs (16 x 8 x 16, bf16): with 16 or 32 heads
 // the kernel is bound by the cache's bytes, not by the MMA rate.  Weights are kept as two bf16 terms (hi + lo).
-// A CTA handles (row, block of 16 MT heads, split of the context); latent_value_kernel merges the splits.
+// A CTA handles (row, block of 16 MT heads, split of the context).  The query side of W_uk before it and W_uv with the
+// output gate after it are batched products over the heads (dense_rows.cu).
 #include "latent.cuh"
 
 namespace tbl {
@@ -62,12 +63,28 @@ __global__ void __launch_bounds__(32 * kWarps) latent_tensor_kernel(const Latent
         asm volatile("cp.async.commit_group;" ::: "memory");
     };
     load_tile(0, t0);
-    const bf16* qa = static_cast<const bf16*>(p.qa) + static_cast<size_t>(row) * p.H * p.cw;
-    for (int i = tid; i < HB * chunks; i += 32 * kWarps) {
-        const int r = i / chunks, c = i - r * chunks;
+    const bf16* qa = static_cast<const bf16*>(p.qa) + static_cast<size_t>(row) * p.H * p.R;
+    const int lat_chunks = p.R / 8;
+    for (int i = tid; i < HB * lat_chunks; i += 32 * kWarps) {
+        const int r = i / lat_chunks, c = i - r * lat_chunks;
         uint4 v = make_uint4(0, 0, 0, 0);
-        if (h0 + r < p.H) v = *reinterpret_cast<const uint4*>(qa + static_cast<size_t>(h0 + r) * p.cw + c * 8);
+        if (h0 + r < p.H) v = *reinterpret_cast<const uint4*>(qa + static_cast<size_t>(h0 + r) * p.R + c * 8);
         *reinterpret_cast<uint4*>(q_s + r * ld + c * 8) = v;
+    }
+    // the rotated part of the queries, rotated here
+    const int half = p.rd / 2, pos = min(n - 1, p.rope_positions - 1);
+    const float *cs = p.rope_cos + static_cast<size_t>(pos) * half, *sn = p.rope_sin + static_cast<size_t>(pos) * half;
+    for (int i = tid; i < HB * half; i += 32 * kWarps) {
+        const int r = i / half, e = i - r * half;
+        float a = 0.0f, b = 0.0f;
+        if (h0 + r < p.H) {
+            const bf16* q = p.q16 + (static_cast<size_t>(row) * p.H + h0 + r) * (p.d + p.rd) + p.d;
+            const float u = to_f(q[e]), v = to_f(q[e + half]), c = __ldg(cs + e), s = __ldg(sn + e);
+            a = u * c - v * s;
+            b = v * c + u * s;
+        }
+        q_s[r * ld + p.R + e] = __float2bfloat16_rn(a);
+        q_s[r * ld + p.R + half + e] = __float2bfloat16_rn(b);
     }
     const int tiles16 = p.R / 16;                            // column tiles of O: warp, warp + 8, ...
     float o[MT][TPW][2][4];
@@ -176,16 +193,20 @@ __global__ void __launch_bounds__(32 * kWarps) latent_tensor_kernel(const Latent
             }
         }
     }
+    // one split: the result itself; several: the partial sums
+    const bool whole = p.splits == 1;
     const size_t unit0 = (static_cast<size_t>(row) * p.H + h0) * p.splits + split;
 #pragma unroll
     for (int i = 0; i < RPW; ++i) {
         const int r = warp * RPW + i;
         const float l = warp_sum(sum[i]);
-        if (lane == 0 && h0 + r < p.H) {
+        if (lane == 0) f_s[r] = 1.0f / l;
+        if (lane == 0 && !whole && h0 + r < p.H) {
             p.part_m[unit0 + static_cast<size_t>(r) * p.splits] = mx[i];
             p.part_l[unit0 + static_cast<size_t>(r) * p.splits] = l;
         }
     }
+    __syncthreads();
 #pragma unroll
     for (int m = 0; m < MT; ++m)
 #pragma unroll
@@ -196,12 +217,49 @@ __global__ void __launch_bounds__(32 * kWarps) latent_tensor_kernel(const Latent
             for (int q = 0; q < 2; ++q)
 #pragma unroll
                 for (int e = 0; e < 2; ++e) {
-                    const int r = m * 16 + e * 8 + (lane >> 2);
-                    if (h0 + r < p.H)
-                        *reinterpret_cast<float2*>(p.part_o + (unit0 + static_cast<size_t>(r) * p.splits) * p.R + c * 16 + q * 8 + (lane & 3) * 2) =
-                            make_float2(o[m][j][q][2 * e], o[m][j][q][2 * e + 1]);
+                    const int r = m * 16 + e * 8 + (lane >> 2), col = c * 16 + q * 8 + (lane & 3) * 2;
+                    if (h0 + r >= p.H) continue;
+                    const float a = o[m][j][q][2 * e], b = o[m][j][q][2 * e + 1];
+                    if (whole)
+                        *reinterpret_cast<uint32_t*>(p.lat + (static_cast<size_t>(row) * p.H + h0 + r) * p.R + col) = pack_bf16(a * f_s[r], b * f_s[r]);
+                    else
+                        *reinterpret_cast<float2*>(p.part_o + (unit0 + static_cast<size_t>(r) * p.splits) * p.R + col) = make_float2(a, b);
                 }
         }
+}
+
+// one CTA per (row, head): the splits of the context come together
+__global__ void __launch_bounds__(128) latent_merge_kernel(const LatentParams p) {
+    __shared__ float fac[1024];
+    __shared__ float total;
+    pdl_launch_dependents();
+    const int tid = threadIdx.x;
+    const size_t unit = (static_cast<size_t>(blockIdx.x) * p.H + blockIdx.y);
+    pdl_wait();
+    if (tid < 32) {
+        float m = -INFINITY, l = 0.0f;
+        for (int s = tid; s < p.splits; s += 32) m = fmaxf(m, p.part_m[unit * p.splits + s]);
+        m = warp_max(m);
+        for (int s = tid; s < p.splits; s += 32) {
+            const float f = ex2(p.part_m[unit * p.splits + s] - m);
+            fac[s] = f;
+            l = fmaf(p.part_l[unit * p.splits + s], f, l);
+        }
+        l = warp_sum(l);
+        if (tid == 0) total = 1.0f / l;
+    }
+    __syncthreads();
+    for (int e = 2 * tid; e < p.R; e += 256) {
+        const float* o = p.part_o + unit * p.splits * p.R + e;
+        float a = 0.0f, b = 0.0f;
+#pragma unroll 8
+        for (int s = 0; s < p.splits; ++s) {
+            const float2 v = *reinterpret_cast<const float2*>(o + static_cast<size_t>(s) * p.R);
+            a = fmaf(v.x, fac[s], a);
+            b = fmaf(v.y, fac[s], b);
+        }
+        *reinterpret_cast<uint32_t*>(p.lat + unit * p.R + e) = pack_bf16(a * total, b * total);
+    }
 }
 
 template <int MT, int TPW>
@@ -218,14 +276,29 @@ cudaError_t launch(const LatentParams& p, int rows, cudaStream_t st) {
 int latent_tensor_heads(const tbl_latent_mixer& m) { return m.heads > 16 ? 32 : 16; }
 
 bool latent_tensor_supported(const tbl_latent_mixer& m) {
-    return m.kv_rank % 16 == 0 && m.rot_dim % 16 == 0 && m.kv_rank <= 512 &&
+    return m.uk_t && m.dim % 8 == 0 && m.kv_rank % 16 == 0 && m.rot_dim % 16 == 0 && m.kv_rank <= 512 &&
            tensor_smem(m.kv_rank + m.rot_dim, latent_tensor_heads(m)) <= 227 * 1024;
 }
 
-cudaError_t launch_latent_tensor(const LatentParams& p, int rows, cudaStream_t st) {
+int launch_latent_tensor(const LatentParams& p, int rows, cudaStream_t st) {
+    DenseCall a{};              // q' = W_uk^T q, all heads in one launch
+    a.x = p.q16; a.w = p.uk_t; a.ldx = p.H * (p.d + p.rd); a.M = rows; a.K = p.d; a.N = p.R;
+    a.out_b16 = static_cast<bf16*>(p.qa); a.ldo = p.H * p.R;
+    a.batch = p.H; a.batch_x = p.d + p.rd; a.batch_w = static_cast<long long>(p.R) * p.d; a.batch_out = p.R;
+    int rc = launch_dense(TBL_BF16, kDenseRows, a, st);
+    if (rc != TBL_OK) return rc;
     const int tpw = ceil_div(p.R, 16 * kWarps);
-    if (p.H > 16) return tpw <= 1 ? launch<2, 1>(p, rows, st) : (tpw <= 2 ? launch<2, 2>(p, rows, st) : launch<2, 4>(p, rows, st));
-    return tpw <= 1 ? launch<1, 1>(p, rows, st) : (tpw <= 2 ? launch<1, 2>(p, rows, st) : launch<1, 4>(p, rows, st));
+    cudaError_t e;
+    if (p.H > 16) e = tpw <= 1 ? launch<2, 1>(p, rows, st) : (tpw <= 2 ? launch<2, 2>(p, rows, st) : launch<2, 4>(p, rows, st));
+    else e = tpw <= 1 ? launch<1, 1>(p, rows, st) : (tpw <= 2 ? launch<1, 2>(p, rows, st) : launch<1, 4>(p, rows, st));
+    if (e != cudaSuccess) return TBL_ERR_CUDA;
+    if (p.splits > 1 && launch_dependent(latent_merge_kernel, dim3(rows, p.H), dim3(128), 0, st, p) != cudaSuccess) return TBL_ERR_CUDA;
+    DenseCall v{};              // W_uv and the output gate
+    v.x = p.lat; v.w = p.uv; v.ldx = p.H * p.R; v.M = rows; v.K = p.R; v.N = p.vd;
+    v.out_b16 = static_cast<bf16*>(p.out); v.ldo = p.H * p.vd;
+    v.batch = p.H; v.batch_x = p.R; v.batch_w = static_cast<long long>(p.vd) * p.R; v.batch_out = p.vd;
+    v.gate = p.proj + p.q_rank + p.R + p.rd; v.ldg = p.ld; v.batch_gate = p.vd;
+    return launch_dense(TBL_BF16, kDenseRows, v, st);
 }
 
 }  // namespace stack

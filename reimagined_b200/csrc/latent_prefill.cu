@@ -237,49 +237,50 @@ latent_prefill_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_co
             tc_fence_after();
             const int last = pos - j * kBlock;                 // last visible column of the block
             const bool edge = __any_sync(0xffffffffu, last < kBlock - 1);
-            uint32_t x[32];
-            float mx = -INFINITY;
-#pragma unroll 1
-            for (int ch = 0; ch < 4; ++ch) {
-                tmem_ld32(s_col + ch * 32, x);
-                tmem_ld_wait();
-                if (edge) {
+            // the whole row at once: 128 scores in registers
+            uint32_t x[4][32];
 #pragma unroll
-                    for (int i = 0; i < 32; ++i) mx = fmaxf(mx, ch * 32 + i <= last ? __uint_as_float(x[i]) : -INFINITY);
-                } else {
+            for (int ch = 0; ch < 4; ++ch) tmem_ld32(s_col + ch * 32, x[ch]);
+            tmem_ld_wait();
+            if (edge) {
 #pragma unroll
-                    for (int i = 0; i < 32; i += 2) mx = fmaxf(mx, fmaxf(__uint_as_float(x[i]), __uint_as_float(x[i + 1])));
-                }
+                for (int ch = 0; ch < 4; ++ch)
+#pragma unroll
+                    for (int i = 0; i < 32; ++i)
+                        if (ch * 32 + i > last) x[ch][i] = 0xff800000u;         // -inf
             }
-            mx *= c;
+            float mx[4];
+#pragma unroll
+            for (int ch = 0; ch < 4; ++ch) {
+                mx[ch] = __uint_as_float(x[ch][0]);
+#pragma unroll
+                for (int i = 1; i < 32; ++i) mx[ch] = fmaxf(mx[ch], __uint_as_float(x[ch][i]));
+            }
+            const float top = fmaxf(fmaxf(mx[0], mx[1]), fmaxf(mx[2], mx[3])) * c;
             if (j == 0) {
-                m = mx;
-            } else if (__any_sync(0xffffffffu, mx > m + kRescale)) {
-                const float mn = fmaxf(m, mx), f = ex2(m - mn);
+                m = top;
+            } else if (__any_sync(0xffffffffu, top > m + kRescale)) {
+                const float mn = fmaxf(m, top), f = ex2(m - mn);
                 m = mn;
                 l *= f;
+#pragma unroll 1
                 for (int ch = 0; ch * 32 < p.vd; ++ch) {       // columns past vd are unused tensor memory
-                    tmem_ld32(o_col + ch * 32, x);
+                    uint32_t y[32];
+                    tmem_ld32(o_col + ch * 32, y);
                     tmem_ld_wait();
 #pragma unroll
-                    for (int i = 0; i < 32; ++i) x[i] = __float_as_uint(__uint_as_float(x[i]) * f);
-                    tmem_st32(o_col + ch * 32, x);
+                    for (int i = 0; i < 32; ++i) y[i] = __float_as_uint(__uint_as_float(y[i]) * f);
+                    tmem_st32(o_col + ch * 32, y);
                 }
             }
             float sum = 0.0f;
-#pragma unroll 1
+#pragma unroll
             for (int ch = 0; ch < 4; ++ch) {
-                tmem_ld32(s_col + ch * 32, x);
-                tmem_ld_wait();
                 float a0 = 0.0f, a1 = 0.0f;
                 uint32_t y[32];
 #pragma unroll
                 for (int i = 0; i < 16; ++i) {
-                    float p0 = ex2(fmaf(__uint_as_float(x[2 * i]), c, -m)), p1 = ex2(fmaf(__uint_as_float(x[2 * i + 1]), c, -m));
-                    if (edge) {
-                        p0 = ch * 32 + 2 * i <= last ? p0 : 0.0f;
-                        p1 = ch * 32 + 2 * i + 1 <= last ? p1 : 0.0f;
-                    }
+                    const float p0 = ex2(fmaf(__uint_as_float(x[ch][2 * i]), c, -m)), p1 = ex2(fmaf(__uint_as_float(x[ch][2 * i + 1]), c, -m));
                     a0 += p0;
                     a1 += p1;
                     const uint32_t hi = pack_bf16(p0, p1);

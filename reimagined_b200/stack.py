@@ -74,6 +74,8 @@ def _fill_latent(e: "StackEngine", layer: capi.StackLayer, p: str, m: dict) -> N
         raise ValueError("latent_attention rotates all of its rotated part (rot.dims == rot_dim)")
     a.in_ = e.dense([p + n for n in ("dq", "dkv", "g")])
     a.uq, a.uk, a.uv, a.out = (e.dense([p + n]) for n in ("uq", "uk", "uv", "o"))
+    uk = e.weights[p + "uk"].cuda().reshape(m["heads"], m["dim"], m["kv_rank"])
+    a.uk_t = e._bf16(uk.transpose(1, 2)).data_ptr()
     a.q_norm, a.kv_norm = e.f32(e.weights[p + "dq.norm"]), e.f32(e.weights[p + "dkv.norm"])
     a.rope_positions = e.capacity
     a.rope_cos, a.rope_sin = e.rotation(float(m["rot"]["base"]), m["rot_dim"])

@@ -230,6 +230,7 @@ class Latent:
         self.cols = q + R + rd + H * vd
         m.in_, m.out = capi.DenseView(dummy, None, 8, self.cols), capi.DenseView(dummy, None, H * vd, 8)
         m.uq, m.uk, m.uv = b.view(uq), b.view(uk), b.view(uv)
+        m.uk_t = b.view(uk.reshape(H, d, R).transpose(1, 2).reshape(H * R, d)).weight
         m.q_norm, m.kv_norm = b.f32(qn), b.f32(kn)
         ang = np.arange(capacity)[:, None] * cfg["rot"]["base"] ** (-2.0 * np.arange(rd // 2) / rd)
         m.rope_cos, m.rope_sin, m.rope_positions = b.f32(np.cos(ang)), b.f32(np.sin(ang)), capacity
