@@ -684,6 +684,30 @@ def run_ours(args):
         dist.destroy_process_group()
 
 
+def run_guselix(args):
+    """One JSON line: tokens/s of Guselix (prefill, decode) and of the hybrid at equal width and depth, one GPU."""
+    import torch
+    from reimagined_b200 import build as tbl_build, stack_shapes
+    if int(os.environ.get("RANK", "0")) != 0:
+        return
+    if not torch.cuda.is_available():
+        raise SystemExit("bench.py needs a CUDA device: there is no CPU fallback")
+    tbl_build.build()
+    torch.cuda.set_device(0)
+    stack_shapes.use_measured_peaks()
+    sampler = ClockSampler(0)
+    sampler.start()
+    records = []
+    for width, layers in ((2048, 8), (4096, 4)):
+        records += stack_shapes.time_guselix(width, layers, iters=args.steps)
+        records += stack_shapes.time_hybrid(width, layers, iters=args.steps)
+    best = max(r["tokens_per_s"] for r in records if r["model"] == "Guselix" and r["phase"] == "decode")
+    print(json.dumps({"metric": "guselix_decode_tokens_per_s", "value": best, "unit": "tokens/s", "n_gpus": 1, "steps": args.steps,
+                      "higher_is_better": True, "vs_baseline": None, "dtype": "bf16", "data": "synthetic", "clocks": sampler.stop(),
+                      "config": {"model": "Guselix, every 4th layer latent attention, random weights; weights exceed L2"},
+                      "records": records}))
+
+
 def main():
     ap = argparse.ArgumentParser()
     ap.add_argument("--gpus", type=int, default=1)
@@ -692,8 +716,13 @@ def main():
     ap.add_argument("--impl", default="ours", choices=["ours", "reference"])
     ap.add_argument("--headline-only", action="store_true",
                     help="skip the gemm / decode / colsplit sections (used for profiler captures of the headline kernel)")
+    ap.add_argument("--model", default="ternary", choices=["ternary", "guselix"],
+                    help="guselix: prefill and decode of the layer-stack model at real layer sizes (random weights) beside the "
+                         "hybrid of the same width and depth, instead of the headline")
     args = ap.parse_args()
-    if args.impl == "reference":
+    if args.model == "guselix":
+        run_guselix(args)
+    elif args.impl == "reference":
         run_reference(args)
     else:
         run_ours(args)

@@ -167,55 +167,72 @@ latent_prefill_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_co
             const uint32_t is = idesc_bf16(kBlock), iv = idesc_bf16(p.vd);
             bool alive = mbar_wait_bounded(q_full, 0, p.status);
             tc_fence_after();
-            auto scores = [&](int w, int j) {          // S_w = Q_w K_j^T
-                const uint32_t a = smem_u32(q_smem + w * q_bytes), b = smem_u32(k_smem + (j % p.k_stages) * k_bytes);
-                uint32_t acc = 0;
-                for (int k = 0; k < p.d / 16; ++k, acc = 1) {
-                    const uint32_t off = (k >> 2) * kSubBytes + (k & 3) * 32;
-                    umma_f16(tmem + w * kBlock, smem_desc_sw128(a + off), smem_desc_sw128(b + off), is, acc);
+            // One thread issues everything, so the loop carries ring positions and descriptors along instead of working them
+            // out per product (a descriptor counts 16-byte units).
+            const uint64_t q_desc = smem_desc_sw128(smem_u32(q_smem)), k_desc = smem_desc_sw128(smem_u32(k_smem)),
+                           v_desc = smem_desc_sw128(smem_u32(v_smem));
+            const int nd = p.d / 16, nr = p.rd / 16;
+            int ks = 0, v0 = 0, v1 = 1;       // ring slots of the next key block and of this block's value halves
+            uint32_t kp = 0, vp0 = 0, vp1 = 0;
+            auto products = [&](uint32_t d_tmem, uint64_t a, uint64_t b, int n, uint32_t acc) {
+                for (; n >= 4; n -= 4, a += kSubBytes / 16, b += kSubBytes / 16, acc = 1) {
+                    umma_f16(d_tmem, a, b, is, acc);
+                    umma_f16(d_tmem, a + 2, b + 2, is, 1);
+                    umma_f16(d_tmem, a + 4, b + 4, is, 1);
+                    umma_f16(d_tmem, a + 6, b + 6, is, 1);
                 }
-                for (int k = 0; k < p.rd / 16; ++k) {
-                    const uint32_t off = (sub_d + (k >> 2)) * kSubBytes + (k & 3) * 32;
-                    umma_f16(tmem + w * kBlock, smem_desc_sw128(a + off), smem_desc_sw128(b + off), is, 1);
-                }
-                umma_commit(&s_full[w]);
+                for (; n > 0; --n, a += 2, b += 2, acc = 1) umma_f16(d_tmem, a, b, is, acc);
             };
             // The order S0(0) S1(0) | PV0(j) S0(j+1) PV1(j) S1(j+1) | ...: each softmax runs under the other tile's products.
             for (int j = -1; alive && j < nmax; ++j) {
-                for (int w = 0; alive && w < 2; ++w) {
+#pragma unroll
+                for (int w = 0; w < 2; ++w) {
                     if (j >= 0 && j < nblk[w]) {
                         alive = mbar_wait_bounded(&p_full[w], j & 1, p.status);
                         if (!alive) break;
                         tc_fence_after();
+                        const uint32_t o = tmem + kOCol + w * 128;
+#pragma unroll
                         for (int h = 0; h < 2; ++h) {
-                            const int vi = 2 * j + h, vs = vi % p.v_stages;
-                            alive = mbar_wait_bounded(&v_full[vs], (vi / p.v_stages) & 1, p.status);
+                            const int vs = h ? v1 : v0;
+                            alive = mbar_wait_bounded(&v_full[vs], h ? vp1 : vp0, p.status);
                             if (!alive) break;
                             tc_fence_after();
-                            const uint32_t b = smem_u32(v_smem + vs * v_bytes);
+                            const uint64_t bd = v_desc + static_cast<uint64_t>(vs) * (v_bytes / 16);
+                            const uint32_t pc = tmem + w * kBlock + h * 64;
+#pragma unroll
                             for (int k = 0; k < 4; ++k) {          // 16 tokens each: columns 32 (k / 2) + 8 (k & 1), + 16 for the low term
-                                const uint32_t pc = tmem + w * kBlock + h * 64 + (k >> 1) * 32 + (k & 1) * 8;
-                                const uint64_t bd = smem_desc_sw128(b + k * 32);
-                                umma_f16_ta(tmem + kOCol + w * 128, pc, bd, iv, (j | h | k) != 0 ? 1u : 0u);
-                                umma_f16_ta(tmem + kOCol + w * 128, pc + 16, bd, iv, 1);
+                                umma_f16_ta(o, pc + (k >> 1) * 32 + (k & 1) * 8, bd + 2 * k, iv, (h | k) != 0 ? 1u : (j != 0 ? 1u : 0u));
+                                umma_f16_ta(o, pc + (k >> 1) * 32 + (k & 1) * 8 + 16, bd + 2 * k, iv, 1);
                             }
                             // the entry is free once the last tile that uses it has read it
                             if (w == 1 || j >= nblk[1]) umma_commit(&v_empty[vs]);
                         }
-                        if (alive && j == nblk[w] - 1) umma_commit(&o_full[w]);
+                        if (!alive) break;
+                        if (j == nblk[w] - 1) umma_commit(&o_full[w]);
                     }
-                    if (!alive) break;
                     const int jn = j + 1;
                     if (jn < nblk[w]) {
                         // first use of a key block waits for it
                         if (w == 0 || jn >= nblk[0]) {
-                            alive = mbar_wait_bounded(&k_full[jn % p.k_stages], (jn / p.k_stages) & 1, p.status);
+                            alive = mbar_wait_bounded(&k_full[ks], kp, p.status);
                             if (!alive) break;
                             tc_fence_after();
                         }
-                        scores(w, jn);
-                        if (w == 1 || jn >= nblk[1]) umma_commit(&k_empty[jn % p.k_stages]);
+                        const uint64_t a = q_desc + static_cast<uint64_t>(w) * (q_bytes / 16), b = k_desc + static_cast<uint64_t>(ks) * (k_bytes / 16);
+                        const uint64_t rot = static_cast<uint64_t>(sub_d) * (kSubBytes / 16);
+                        products(tmem + w * kBlock, a, b, nd, 0);
+                        products(tmem + w * kBlock, a + rot, b + rot, nr, 1);
+                        umma_commit(&s_full[w]);
+                        if (w == 1 || jn >= nblk[1]) umma_commit(&k_empty[ks]);
                     }
+                }
+                if (++ks == p.k_stages) { ks = 0; kp ^= 1; }
+                if (j >= 0) {                                      // two value halves further on
+                    v0 += 2;
+                    if (v0 >= p.v_stages) { v0 -= p.v_stages; vp0 ^= 1; }
+                    v1 += 2;
+                    if (v1 >= p.v_stages) { v1 -= p.v_stages; vp1 ^= 1; }
                 }
             }
         }
@@ -381,7 +398,7 @@ int launch_latent_expanded(const tbl_latent_mixer& m, const LatentParams& p, int
     const size_t room = 227 * 1024 - kFixedSmem - 2 * tile;
     f.k_stages = 2;
     f.v_stages = static_cast<int>((room - 2 * tile) / half);
-    f.v_stages = f.v_stages > 4 ? 4 : f.v_stages;
+    f.v_stages = f.v_stages > 4 ? 4 : f.v_stages;          // at least a whole block: two halves
     if (f.v_stages < 2) return TBL_ERR_SHAPE;
     const size_t smem = kFixedSmem + 4 * tile + f.v_stages * half;
     CUtensorMap mq, mk, mr, mv;

@@ -12,8 +12,6 @@ replayed from CUDA graphs.  torch owns device memory and streams only.
 
 Guselix is this family with the mixers `general_delta` (delta rule with per-channel decay and removal rate) and
 `latent_attention`, and a learned average over the depth after every layer.
-
-    python -m reimagined_b200.stack --rows 4096          # time prefill and decode of a synthetic model, one JSON line
 """
 from __future__ import annotations
 
