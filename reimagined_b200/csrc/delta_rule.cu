@@ -2,12 +2,12 @@
 // rates, unit keys, head norm and output gate.  Everything here is fp32; states are stored [head][value][key].
 //
 // A value column j of a state evolves on its own:  s_j <- w*s_j + (k v_j - (a*u) (u.s_j)),  o_j = r.s_j,  so the
-// columns are spread over threads and CTAs and only the two dot products over the keys cross lanes: eight lanes share
-// a column, each holding every eighth group of four keys in registers, and the arithmetic runs on packed fp32 pairs.
+// columns are spread over threads and CTAs and only the dot products over the keys cross lanes: eight or sixteen lanes
+// share a column, each holding its groups of four keys in registers, and the arithmetic runs on packed fp32 pairs.
 //
-//   delta_scan_kernel   a sequence of tokens: a CTA owns 32 columns of a head.  Eight producer warps turn the raw
-//                       projections of the next chunk of tokens into (u, w, a*u, k, r, v) records in shared memory while
-//                       four consumer warps walk the current chunk token by token with the state in registers.
+//   delta_scan_kernel   a sequence of tokens, two per round: a CTA owns 32 columns of a head.  Eight producer warps turn
+//                       the raw projections of the next sixteen tokens into records in shared memory while four
+//                       consumer warps walk the current ones with the state in registers.
 //   delta_step_kernel   one token: a CTA per head also computes the low-rank decay product, the head norm and the gate.
 #include "stack.cuh"
 
@@ -28,13 +28,6 @@ __device__ __forceinline__ float sum8lanes(float v) {
     v += __shfl_xor_sync(0xffffffffu, v, 1);
     v += __shfl_xor_sync(0xffffffffu, v, 2);
     v += __shfl_xor_sync(0xffffffffu, v, 4);
-    return v;
-}
-// Sums of a and b over a group of eight lanes: lanes 0-3 return a's, lanes 4-7 (upper) b's.
-__device__ __forceinline__ float sum_halves(float a, float b, bool upper) {
-    float v = (upper ? b : a) + __shfl_xor_sync(0xffffffffu, upper ? a : b, 4);
-    v += __shfl_xor_sync(0xffffffffu, v, 1);
-    v += __shfl_xor_sync(0xffffffffu, v, 2);
     return v;
 }
 __device__ __forceinline__ void bar_sync(int id, int n) { asm volatile("bar.sync %0, %1;" ::"r"(id), "r"(n) : "memory"); }
@@ -81,28 +74,49 @@ constexpr int kScanCols = 32;          // value columns per CTA
 constexpr int kProducers = 8;          // producer warps: enough tokens in flight to cover the loads' latency
 constexpr int kScanThreads = 32 * (4 + kProducers);
 
+// The scan takes two tokens per round.  With w, u, q = a * u, k, r, v of the two tokens (0 and 1) and the state S before
+// them, everything the round needs from S are four dot products per column, taken together:
+//     d0 = u0.S,   e1 = (u1 w0).S,   p0 = (r0 w0).S,   p1 = (r1 w0 w1).S
+// and the rest are products of the tokens with each other, the same for every column, which the producers work out:
+//     d1 = e1 + (u1.k0) v0 - (u1.q0) d0
+//     o0 = p0 + (r0.k0) v0 - (r0.q0) d0
+//     o1 = p1 + (r1.w1 k0) v0 - (r1.w1 q0) d0 + (r1.k1) v1 - (r1.q1) d1
+//     S  <- (w0 w1) S + (w1 k0) v0 - (w1 q0) d0 + k1 v1 - q1 d1
+// An odd last token is followed by one that changes nothing (w = 1, the others 0).
 template <int DKP>
 struct ScanShape {
-    static constexpr int kChunk = DKP <= 128 ? 16 : 8;                 // tokens per buffer, a multiple of kProducers
-    static constexpr int kRecord = 5 * DKP + kScanCols;                // floats per token: u | w | a*u | k | r | v
-    static constexpr size_t kSmem = sizeof(float) * 2 * kChunk * kRecord;
+    static constexpr int kPairs = kProducers;                          // rounds per buffer: one per producer warp
+    static constexpr int kScalars = 9 * DKP;                           // 12 products of the tokens with each other
+    static constexpr int kValues = kScalars + 16;                      // v of both tokens, this CTA's columns
+    static constexpr int kRecord = kValues + 2 * kScanCols;            // floats per round
+    static constexpr size_t kSmem = sizeof(float) * 2 * kPairs * kRecord;
 };
+
+__device__ __forceinline__ float pick4(const float (&v)[4], int n) {
+    const float a = n & 1 ? v[1] : v[0], b = n & 1 ? v[3] : v[2];
+    return n & 2 ? b : a;
+}
+__device__ __forceinline__ float4 mul4(float4 a, float4 b) { return make_float4(a.x * b.x, a.y * b.y, a.z * b.z, a.w * b.w); }
+__device__ __forceinline__ float dot4(float4 a, float4 b, float c) { return fmaf(a.x, b.x, fmaf(a.y, b.y, fmaf(a.z, b.z, fmaf(a.w, b.w, c)))); }
+// (a division good to two units in the last place)
+__device__ __forceinline__ float sigmoid_near(float z) { return __fdividef(1.0f, 1.0f + expf(-z)); }
 
 template <int DKP>
 __global__ void __launch_bounds__(kScanThreads) delta_scan_kernel(const DeltaParams p) {
-    constexpr int CT = ScanShape<DKP>::kChunk, REC = ScanShape<DKP>::kRecord;
-    constexpr int G = DKP / 32;                // float4 groups per lane
+    using Shape = ScanShape<DKP>;
+    constexpr int PAIRS = Shape::kPairs, REC = Shape::kRecord;
+    constexpr int G = DKP / 64;                // groups of four keys per consumer lane: 4 (l + 16 g), l = lane % 16
     constexpr int NI = (DKP + 127) / 128;      // groups of four channels per producer lane
     extern __shared__ __align__(16) float sm[];
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     const int head = blockIdx.y, seq = blockIdx.z, j0 = blockIdx.x * kScanCols;
     const int dim = p.dim, HD = p.heads * dim;
-    const int chunks = (p.n_tok + CT - 1) / CT;
+    const int chunks = (p.n_tok + 2 * PAIRS - 1) / (2 * PAIRS);
     const size_t row0 = static_cast<size_t>(seq) * p.n_tok;
     pdl_launch_dependents();
     pdl_wait();
     if (warp >= 4) {
-        // ---- producers: warp w takes tokens w, w + kProducers, ...; lane l channels 4l .. 4l + 3 (+ 128) ----
+        // ---- producers: warp w takes round w of every buffer; lane l channels 4l .. 4l + 3 (+ 128) ----
         const int pw = warp - 4;
         const bool vec = ((dim | p.ld) & 3) == 0;      // every row and head starts on 16 bytes
         auto load4 = [&](const float* base, int c, bool live) {
@@ -115,120 +129,184 @@ __global__ void __launch_bounds__(kScanThreads) delta_scan_kernel(const DeltaPar
             if (c + 3 < dim) v.w = base[c + 3];
             return v;
         };
-        float4 w0[NI], nr[NI], nk[NI], na[NI], nz[NI];
-        float nv = 0.0f;
+        float4 w0[NI], nr[2][NI], nk[2][NI], na[2][NI], nz[2][NI];
+        float nv[2];
 #pragma unroll
         for (int i = 0; i < NI; ++i) w0[i] = load4(p.w0 + head * dim, 4 * lane + 128 * i, true);
-        auto fetch = [&](int t) {
-            const bool live = t < p.n_tok;
-            const float* row = p.proj + (row0 + (live ? t : 0)) * p.ld + head * dim;
-            const float* zr = p.z + (row0 + (live ? t : 0)) * HD + head * dim;
+        auto fetch = [&](int t0) {
 #pragma unroll
-            for (int i = 0; i < NI; ++i) {
-                const int c = 4 * lane + 128 * i;
-                nr[i] = load4(row, c, live);
-                nk[i] = load4(row + HD, c, live);
-                na[i] = load4(row + 4 * HD, c, live);
-                nz[i] = load4(zr, c, live);
-            }
-            nv = live && j0 + lane < dim ? row[2 * HD + j0 + lane] : 0.0f;
-        };
-        fetch(pw);
-        for (int ch = 0; ch < chunks; ++ch) {
-            const int b = ch & 1;
-            if (ch >= 2) bar_sync(3 + b, kScanThreads);
-            for (int i0 = pw; i0 < CT; i0 += kProducers) {
-                const int t = ch * CT + i0;
-                if (t >= p.n_tok) break;
-                float4 r[NI], k[NI], a[NI], z[NI];
-                float ss = 0.0f;
-#pragma unroll
-                for (int i = 0; i < NI; ++i) {
-                    r[i] = nr[i]; k[i] = nk[i]; a[i] = na[i]; z[i] = nz[i];
-                    ss += k[i].x * k[i].x + k[i].y * k[i].y + k[i].z * k[i].z + k[i].w * k[i].w;
-                }
-                const float v = nv;
-                fetch(t + kProducers);
-                const float inv = 1.0f / sqrtf(warp_sum(ss) + p.key_eps);
-                float* rec = sm + static_cast<size_t>(b * CT + i0) * REC;
-                auto decay = [&](float zz) { return expf(-p.rate * sigmoid_f(zz)); };
+            for (int s = 0; s < 2; ++s) {
+                const bool live = t0 + s < p.n_tok;
+                const size_t at = row0 + (live ? t0 + s : 0);
+                const float* row = p.proj + at * p.ld + head * dim;
+                const float* zr = p.z + at * HD + head * dim;
 #pragma unroll
                 for (int i = 0; i < NI; ++i) {
                     const int c = 4 * lane + 128 * i;
-                    if (c >= DKP) break;
-                    const float4 u = make_float4(k[i].x * inv, k[i].y * inv, k[i].z * inv, k[i].w * inv);
-                    *reinterpret_cast<float4*>(rec + c) = u;
-                    *reinterpret_cast<float4*>(rec + DKP + c) =
-                        make_float4(decay(z[i].x + w0[i].x), decay(z[i].y + w0[i].y), decay(z[i].z + w0[i].z), decay(z[i].w + w0[i].w));
-                    *reinterpret_cast<float4*>(rec + 2 * DKP + c) =
-                        make_float4(sigmoid_f(a[i].x) * u.x, sigmoid_f(a[i].y) * u.y, sigmoid_f(a[i].z) * u.z, sigmoid_f(a[i].w) * u.w);
-                    *reinterpret_cast<float4*>(rec + 3 * DKP + c) = k[i];
-                    *reinterpret_cast<float4*>(rec + 4 * DKP + c) = r[i];
+                    nr[s][i] = load4(row, c, live);
+                    nk[s][i] = load4(row + HD, c, live);
+                    na[s][i] = load4(row + 4 * HD, c, live);
+                    nz[s][i] = load4(zr, c, live);
                 }
-                rec[5 * DKP + lane] = v;
+                nv[s] = live && j0 + lane < dim ? row[2 * HD + j0 + lane] : 0.0f;
+            }
+        };
+        fetch(2 * pw);
+        for (int ch = 0; ch < chunks; ++ch) {
+            const int b = ch & 1, t0 = 2 * (ch * PAIRS + pw);
+            if (ch >= 2) bar_sync(3 + b, kScanThreads);
+            if (t0 < p.n_tok) {
+                float4 r[2][NI], k[2][NI], u[2][NI], q[2][NI], w[2][NI];
+                const float v0 = nv[0], v1 = nv[1];
+                float s0 = 0.0f, s1 = 0.0f;
+#pragma unroll
+                for (int i = 0; i < NI; ++i) {
+                    s0 = dot4(nk[0][i], nk[0][i], s0);
+                    s1 = dot4(nk[1][i], nk[1][i], s1);
+                }
+                const float i0 = 1.0f / sqrtf(warp_sum(s0) + p.key_eps), i1 = 1.0f / sqrtf(warp_sum(s1) + p.key_eps);
+                const bool second = t0 + 1 < p.n_tok;
+                auto decay = [&](float z) { return expf(-p.rate * sigmoid_near(z)); };
+#pragma unroll
+                for (int s = 0; s < 2; ++s)
+#pragma unroll
+                    for (int i = 0; i < NI; ++i) {
+                        const float n = s ? i1 : i0;
+                        r[s][i] = nr[s][i];
+                        k[s][i] = nk[s][i];
+                        u[s][i] = mul4(k[s][i], make_float4(n, n, n, n));
+                        q[s][i] = mul4(make_float4(sigmoid_near(na[s][i].x), sigmoid_near(na[s][i].y), sigmoid_near(na[s][i].z), sigmoid_near(na[s][i].w)), u[s][i]);
+                        w[s][i] = make_float4(decay(nz[s][i].x + w0[i].x), decay(nz[s][i].y + w0[i].y), decay(nz[s][i].z + w0[i].z), decay(nz[s][i].w + w0[i].w));
+                        if (s == 1 && !second) w[s][i] = make_float4(1.0f, 1.0f, 1.0f, 1.0f);
+                    }
+                fetch(t0 + 2 * PAIRS);
+                float* rec = sm + static_cast<size_t>(b * PAIRS + pw) * REC;
+                float m[8] = {};
+#pragma unroll
+                for (int i = 0; i < NI; ++i) {
+                    const int c = 4 * lane + 128 * i;
+                    const float4 k0w = mul4(w[1][i], k[0][i]), q0w = mul4(w[1][i], q[0][i]), ww = mul4(w[0][i], w[1][i]);
+                    m[0] = dot4(r[0][i], k[0][i], m[0]); m[1] = dot4(r[0][i], q[0][i], m[1]);
+                    m[2] = dot4(r[1][i], k0w, m[2]);     m[3] = dot4(r[1][i], q0w, m[3]);
+                    m[4] = dot4(r[1][i], k[1][i], m[4]); m[5] = dot4(r[1][i], q[1][i], m[5]);
+                    m[6] = dot4(u[1][i], k[0][i], m[6]); m[7] = dot4(u[1][i], q[0][i], m[7]);
+                    if (c >= DKP) continue;
+                    *reinterpret_cast<float4*>(rec + c) = u[0][i];
+                    *reinterpret_cast<float4*>(rec + DKP + c) = mul4(u[1][i], w[0][i]);
+                    *reinterpret_cast<float4*>(rec + 2 * DKP + c) = mul4(r[0][i], w[0][i]);
+                    *reinterpret_cast<float4*>(rec + 3 * DKP + c) = mul4(r[1][i], ww);
+                    *reinterpret_cast<float4*>(rec + 4 * DKP + c) = ww;
+                    *reinterpret_cast<float4*>(rec + 5 * DKP + c) = k0w;
+                    *reinterpret_cast<float4*>(rec + 6 * DKP + c) = q0w;
+                    *reinterpret_cast<float4*>(rec + 7 * DKP + c) = k[1][i];
+                    *reinterpret_cast<float4*>(rec + 8 * DKP + c) = q[1][i];
+                }
+                // the eight products over the lanes: after three exchanges a lane holds one of them, number lane / 4
+                float m4[4], m2[2];
+#pragma unroll
+                for (int e = 0; e < 4; ++e)
+                    m4[e] = (lane & 16 ? m[e + 4] : m[e]) + __shfl_xor_sync(0xffffffffu, lane & 16 ? m[e] : m[e + 4], 16);
+#pragma unroll
+                for (int e = 0; e < 2; ++e)
+                    m2[e] = (lane & 8 ? m4[e + 2] : m4[e]) + __shfl_xor_sync(0xffffffffu, lane & 8 ? m4[e] : m4[e + 2], 8);
+                float m1 = (lane & 4 ? m2[1] : m2[0]) + __shfl_xor_sync(0xffffffffu, lane & 4 ? m2[0] : m2[1], 4);
+                m1 += __shfl_xor_sync(0xffffffffu, m1, 2);
+                m1 += __shfl_xor_sync(0xffffffffu, m1, 1);
+                // token 0: factors of v0, d0, v1, d1; token 1: the same; then those of d1
+                float* sc = rec + Shape::kScalars;
+                if ((lane & 3) == 0) {
+                    const int e = lane >> 2;
+                    sc[e < 2 ? e : e + 2] = m1;
+                    if (e < 2) sc[2 + e] = 0.0f;
+                }
+                rec[Shape::kValues + lane] = v0;
+                rec[Shape::kValues + kScanCols + lane] = v1;
             }
             __threadfence_block();
             bar_arrive(1 + b, kScanThreads);
         }
         return;
     }
-    // ---- consumers: two columns per group of eight lanes ----
-    const int l8 = lane & 7, cl = warp * 8 + (lane >> 3) * 2;           // first of this lane's columns within the CTA
-    const int slot = p.slots[seq];
-    float* st = p.states + (static_cast<size_t>(slot) * p.heads + head) * dim * dim;
-    ulonglong2 S[2][G];
+    // ---- consumers: sixteen lanes share the keys of four columns ----
+    const int l = lane & 15, base = lane & 16, cl = warp * 8 + (base >> 2);       // first of this lane's columns within the CTA
+    float* st = p.states + (static_cast<size_t>(p.slots[seq]) * p.heads + head) * dim * dim;
+    ulonglong2 S[4][G];
 #pragma unroll
-    for (int n = 0; n < 2; ++n)
+    for (int n = 0; n < 4; ++n)
 #pragma unroll
         for (int g = 0; g < G; ++g)
-            S[n][g] = j0 + cl + n < dim ? load_state4(st + static_cast<size_t>(j0 + cl + n) * dim, 4 * (l8 + 8 * g), dim)
-                                        : make_ulonglong2(0, 0);
-    const bool upper = (l8 & 4) != 0;                  // lanes 0-3 of a group end up with the first column's sums, 4-7 with the second's
-    float* o = p.o + row0 * HD + head * dim + j0 + cl + (upper ? 1 : 0);
-    const bool writes = (l8 & 3) == 0 && j0 + cl + (upper ? 1 : 0) < dim;
+            S[n][g] = j0 + cl + n < dim ? load_state4(st + static_cast<size_t>(j0 + cl + n) * dim, 4 * (l + 16 * g), dim) : make_ulonglong2(0, 0);
+    // after the sums over the lanes, lane l holds dot product l / 4 of column l % 4: lanes 8 .. 15 finish the two readouts
+    const int mine = l & 3, token = (l >> 2) & 1;
+    const bool writes = l >= 8 && j0 + cl + mine < dim;
+    float* o = p.o + (row0 + token) * HD + head * dim + j0 + cl + mine;
     for (int ch = 0; ch < chunks; ++ch) {
         const int b = ch & 1;
         bar_sync(1 + b, kScanThreads);
-        const int n = min(CT, p.n_tok - ch * CT);
-#pragma unroll 2
-        for (int i = 0; i < n; ++i) {
-            const float* rec = sm + static_cast<size_t>(b * CT + i) * REC;
-            const ulonglong2* q = reinterpret_cast<const ulonglong2*>(rec) + l8;
-            pair2 d0 = 0, d1 = 0, e0 = 0, e1 = 0;
+        const int t0 = 2 * ch * PAIRS, rounds = min(PAIRS, (p.n_tok - t0 + 1) / 2);
+#pragma unroll 1
+        for (int i = 0; i < rounds; ++i) {
+            const float* rec = sm + static_cast<size_t>(b * PAIRS + i) * REC;
+            const ulonglong2* q = reinterpret_cast<const ulonglong2*>(rec) + l;
+            constexpr int V = DKP / 4;                     // 16-byte units per vector
+            float x[4][4];
+#pragma unroll
+            for (int d = 0; d < 4; ++d) {
+                ulonglong2 c[G];
+#pragma unroll
+                for (int g = 0; g < G; ++g) c[g] = q[d * V + 16 * g];
+#pragma unroll
+                for (int n = 0; n < 4; ++n) {
+                    pair2 a = mul2(c[0].x, S[n][0].x), e = mul2(c[0].y, S[n][0].y);
+#pragma unroll
+                    for (int g = 1; g < G; ++g) { a = fma2(c[g].x, S[n][g].x, a); e = fma2(c[g].y, S[n][g].y, e); }
+                    x[d][n] = sum2(add2(a, e));
+                }
+            }
+            const float4 va = *reinterpret_cast<const float4*>(rec + Shape::kValues + cl), vb = *reinterpret_cast<const float4*>(rec + Shape::kValues + kScanCols + cl);
+            const float4 f = *reinterpret_cast<const float4*>(rec + Shape::kScalars + 4 * token);
+            const float2 fd = *reinterpret_cast<const float2*>(rec + Shape::kScalars + 8);
+            float y[2][4], z[4], h[2], r;
+#pragma unroll
+            for (int d = 0; d < 2; ++d)
+#pragma unroll
+                for (int n = 0; n < 4; ++n) y[d][n] = (l & 8 ? x[d + 2][n] : x[d][n]) + __shfl_xor_sync(0xffffffffu, l & 8 ? x[d][n] : x[d + 2][n], 8);
+#pragma unroll
+            for (int n = 0; n < 4; ++n) z[n] = (l & 4 ? y[1][n] : y[0][n]) + __shfl_xor_sync(0xffffffffu, l & 4 ? y[0][n] : y[1][n], 4);
+#pragma unroll
+            for (int n = 0; n < 2; ++n) h[n] = (l & 2 ? z[n + 2] : z[n]) + __shfl_xor_sync(0xffffffffu, l & 2 ? z[n] : z[n + 2], 2);
+            r = (l & 1 ? h[1] : h[0]) + __shfl_xor_sync(0xffffffffu, l & 1 ? h[0] : h[1], 1);
+            float d0[4], d1[4];
+            const float v0[4] = {va.x, va.y, va.z, va.w}, v1[4] = {vb.x, vb.y, vb.z, vb.w};
+#pragma unroll
+            for (int n = 0; n < 4; ++n) {
+                d0[n] = __shfl_sync(0xffffffffu, r, base + n);
+                d1[n] = __shfl_sync(0xffffffffu, r, base + 4 + n);
+            }
+#pragma unroll
+            for (int n = 0; n < 4; ++n) d1[n] = fmaf(fd.x, v0[n], fmaf(-fd.y, d0[n], d1[n]));
+            pair2 p0[4], p1[4], m0[4], m1[4];
+#pragma unroll
+            for (int n = 0; n < 4; ++n) { p0[n] = dup2(v0[n]); p1[n] = dup2(v1[n]); m0[n] = dup2(-d0[n]); m1[n] = dup2(-d1[n]); }
 #pragma unroll
             for (int g = 0; g < G; ++g) {
-                const ulonglong2 u = q[8 * g];
-                d0 = fma2(u.x, S[0][g].x, d0); e0 = fma2(u.y, S[0][g].y, e0);
-                d1 = fma2(u.x, S[1][g].x, d1); e1 = fma2(u.y, S[1][g].y, e1);
-            }
-            const float2 v = *reinterpret_cast<const float2*>(rec + 5 * DKP + cl);
-            // both columns' sums over the eight lanes: each half of the lanes adds up one column, then they swap
-            const float own = sum_halves(sum2(add2(d0, e0)), sum2(add2(d1, e1)), upper);
-            const float other = __shfl_xor_sync(0xffffffffu, own, 4);
-            const pair2 m0 = dup2(upper ? -other : -own), m1 = dup2(upper ? -own : -other);
-            const pair2 v0 = dup2(v.x), v1 = dup2(v.y);
-            pair2 o0 = 0, o1 = 0, f0 = 0, f1 = 0;
+                const ulonglong2 w = q[4 * V + 16 * g], k0 = q[5 * V + 16 * g], q0 = q[6 * V + 16 * g], k1 = q[7 * V + 16 * g], q1 = q[8 * V + 16 * g];
 #pragma unroll
-            for (int g = 0; g < G; ++g) {
-                const ulonglong2 w = q[DKP / 4 + 8 * g], au = q[2 * (DKP / 4) + 8 * g], k = q[3 * (DKP / 4) + 8 * g],
-                                 r = q[4 * (DKP / 4) + 8 * g];
-                S[0][g].x = fma2(w.x, S[0][g].x, fma2(au.x, m0, mul2(k.x, v0)));
-                S[0][g].y = fma2(w.y, S[0][g].y, fma2(au.y, m0, mul2(k.y, v0)));
-                S[1][g].x = fma2(w.x, S[1][g].x, fma2(au.x, m1, mul2(k.x, v1)));
-                S[1][g].y = fma2(w.y, S[1][g].y, fma2(au.y, m1, mul2(k.y, v1)));
-                o0 = fma2(r.x, S[0][g].x, o0); f0 = fma2(r.y, S[0][g].y, f0);
-                o1 = fma2(r.x, S[1][g].x, o1); f1 = fma2(r.y, S[1][g].y, f1);
+                for (int n = 0; n < 4; ++n) {
+                    S[n][g].x = fma2(q1.x, m1[n], fma2(k1.x, p1[n], fma2(q0.x, m0[n], fma2(k0.x, p0[n], mul2(w.x, S[n][g].x)))));
+                    S[n][g].y = fma2(q1.y, m1[n], fma2(k1.y, p1[n], fma2(q0.y, m0[n], fma2(k0.y, p0[n], mul2(w.y, S[n][g].y)))));
+                }
             }
-            const float ro = sum_halves(sum2(add2(o0, f0)), sum2(add2(o1, f1)), upper);
-            if (writes) o[static_cast<size_t>(ch * CT + i) * HD] = ro;
+            const float out = fmaf(f.x, pick4(v0, mine), fmaf(-f.y, pick4(d0, mine), fmaf(f.z, pick4(v1, mine), fmaf(-f.w, pick4(d1, mine), r))));
+            if (writes && t0 + 2 * i + token < p.n_tok) o[static_cast<size_t>(t0 + 2 * i) * HD] = out;
         }
         if (ch + 2 < chunks) bar_arrive(3 + b, kScanThreads);
     }
 #pragma unroll
-    for (int n = 0; n < 2; ++n)
+    for (int n = 0; n < 4; ++n)
 #pragma unroll
         for (int g = 0; g < G; ++g)
-            if (j0 + cl + n < dim) store_state4(st + static_cast<size_t>(j0 + cl + n) * dim, 4 * (l8 + 8 * g), dim, S[n][g]);
+            if (j0 + cl + n < dim) store_state4(st + static_cast<size_t>(j0 + cl + n) * dim, 4 * (l + 16 * g), dim, S[n][g]);
 }
 
 // tanh of the low-rank decay projection, in the precision's type, for the GEMM with W_w2
@@ -465,8 +543,7 @@ int launch_scan(const tbl_delta_mixer& m, DeltaParams p, int precision, int n_se
     int rc = decay_products<T>(m, p, precision, rows, static_cast<T*>(w.th), w.z, st);
     if (rc != TBL_OK) return rc;
     p.z = w.z;
-    if (p.dim <= 32) rc = launch_scan_d<32>(p, n_seq, st);
-    else if (p.dim <= 64) rc = launch_scan_d<64>(p, n_seq, st);
+    if (p.dim <= 64) rc = launch_scan_d<64>(p, n_seq, st);
     else if (p.dim <= 128) rc = launch_scan_d<128>(p, n_seq, st);
     else rc = launch_scan_d<256>(p, n_seq, st);
     if (rc != TBL_OK) return rc;

@@ -55,10 +55,12 @@ __global__ void __launch_bounds__(32 * kWarps) latent_tensor_kernel(const Latent
     const int chunks = W / 8;
     auto load_tile = [&](int stage, int t) {
         const uint32_t base = smem_u32(c_s + stage * kTile * ld);
-        for (int i = tid; i < kTile * chunks; i += 32 * kWarps) {
-            const int r = i / chunks, c = i - r * chunks;
+        // a warp takes every eighth row, its lanes the 16-byte pieces: no division per piece
+#pragma unroll
+        for (int r = warp; r < kTile; r += kWarps) {
             const bool ok = t + r < t1;
-            cp16(base + (r * ld + c * 8) * 2, cache + static_cast<size_t>(ok ? t + r : 0) * p.cw + c * 8, ok);
+            const bf16* src = cache + static_cast<size_t>(ok ? t + r : 0) * p.cw;
+            for (int c = lane; c < chunks; c += 32) cp16(base + (r * ld + c * 8) * 2, src + c * 8, ok);
         }
         asm volatile("cp.async.commit_group;" ::: "memory");
     };
@@ -105,13 +107,15 @@ __global__ void __launch_bounds__(32 * kWarps) latent_tensor_kernel(const Latent
         if (t + kTile < t1) load_tile(stage ^ 1, t + kTile);
         const bf16* ct = c_s + stage * kTile * ld;
         // scores: warp w takes tokens 8w .. 8w + 7
-        float s[MT][4];
+        float s[MT][4], s2[MT][4];                           // two sums each: half as long a chain of dependent MMAs
 #pragma unroll
-        for (int m = 0; m < MT; ++m) s[m][0] = s[m][1] = s[m][2] = s[m][3] = 0.0f;
+        for (int m = 0; m < MT; ++m)
+#pragma unroll
+            for (int e = 0; e < 4; ++e) s[m][e] = s2[m][e] = 0.0f;
         const uint32_t b_addr = smem_u32(ct + (warp * 8 + (lane & 7)) * ld + (lane >> 3) * 8);
         const uint32_t a_addr = smem_u32(q_s + (lane & 15) * ld + (lane >> 4) * 8);
         int k = 0;
-#pragma unroll 2
+#pragma unroll 3
         for (; k + 32 <= W; k += 32) {
             uint32_t b[4], a[4];
             ldsm4(b, b_addr + k * 2);
@@ -120,7 +124,7 @@ __global__ void __launch_bounds__(32 * kWarps) latent_tensor_kernel(const Latent
                 ldsm4(a, a_addr + (m * 16 * ld + k) * 2);
                 mma(s[m], a, b[0], b[1]);
                 ldsm4(a, a_addr + (m * 16 * ld + k + 16) * 2);
-                mma(s[m], a, b[2], b[3]);
+                mma(s2[m], a, b[2], b[3]);
             }
         }
         if (k < W) {
@@ -136,8 +140,8 @@ __global__ void __launch_bounds__(32 * kWarps) latent_tensor_kernel(const Latent
 #pragma unroll
         for (int m = 0; m < MT; ++m) {
             float* d = s_s + (m * 16 + (lane >> 2)) * kSLd + warp * 8 + (lane & 3) * 2;
-            *reinterpret_cast<float2*>(d) = make_float2(s[m][0], s[m][1]);
-            *reinterpret_cast<float2*>(d + 8 * kSLd) = make_float2(s[m][2], s[m][3]);
+            *reinterpret_cast<float2*>(d) = make_float2(s[m][0] + s2[m][0], s[m][1] + s2[m][1]);
+            *reinterpret_cast<float2*>(d + 8 * kSLd) = make_float2(s[m][2] + s2[m][2], s[m][3] + s2[m][3]);
         }
         __syncthreads();
         // softmax: a warp owns RPW score rows, two tokens per lane
@@ -228,37 +232,56 @@ __global__ void __launch_bounds__(32 * kWarps) latent_tensor_kernel(const Latent
         }
 }
 
-// one CTA per (row, head): the splits of the context come together
-__global__ void __launch_bounds__(128) latent_merge_kernel(const LatentParams p) {
-    __shared__ float fac[1024];
-    __shared__ float total;
+// One CTA per (row, head): the splits of the context come together.  Four groups of 128 threads take every fourth split,
+// four columns per thread.
+constexpr int kMergeThreads = 512;
+
+__global__ void __launch_bounds__(kMergeThreads) latent_merge_kernel(const LatentParams p) {
+    __shared__ float fac[1024], red[16], total_s;
+    __shared__ float4 part[4][128];
     pdl_launch_dependents();
-    const int tid = threadIdx.x;
-    const size_t unit = (static_cast<size_t>(blockIdx.x) * p.H + blockIdx.y);
+    const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, col = tid & 127, group = tid >> 7;
+    const size_t unit = static_cast<size_t>(blockIdx.x) * p.H + blockIdx.y;
     pdl_wait();
-    if (tid < 32) {
-        float m = -INFINITY, l = 0.0f;
-        for (int s = tid; s < p.splits; s += 32) m = fmaxf(m, p.part_m[unit * p.splits + s]);
-        m = warp_max(m);
-        for (int s = tid; s < p.splits; s += 32) {
-            const float f = ex2(p.part_m[unit * p.splits + s] - m);
-            fac[s] = f;
-            l = fmaf(p.part_l[unit * p.splits + s], f, l);
-        }
-        l = warp_sum(l);
-        if (tid == 0) total = 1.0f / l;
-    }
+    const float *pm = p.part_m + unit * p.splits, *pl = p.part_l + unit * p.splits;
+    float m = -INFINITY;
+    for (int s = tid; s < p.splits; s += kMergeThreads) m = fmaxf(m, pm[s]);
+    m = warp_max(m);
+    if (lane == 0) red[warp] = m;
     __syncthreads();
-    for (int e = 2 * tid; e < p.R; e += 256) {
-        const float* o = p.part_o + unit * p.splits * p.R + e;
-        float a = 0.0f, b = 0.0f;
+#pragma unroll
+    for (int w = 0; w < 16; ++w) m = fmaxf(m, red[w]);
+    float l = 0.0f;
+    for (int s = tid; s < p.splits; s += kMergeThreads) {
+        fac[s] = ex2(pm[s] - m);
+        l = fmaf(pl[s], fac[s], l);
+    }
+    l = warp_sum(l);
+    __syncthreads();
+    if (lane == 0) red[warp] = l;
+    __syncthreads();
+    if (tid == 0) {
+        float t = 0.0f;
+        for (int w = 0; w < 16; ++w) t += red[w];
+        total_s = 1.0f / t;
+    }
+    float4 a = make_float4(0.0f, 0.0f, 0.0f, 0.0f);
+    if (4 * col < p.R) {
+        const float* o = p.part_o + unit * p.splits * p.R + 4 * col;
 #pragma unroll 8
-        for (int s = 0; s < p.splits; ++s) {
-            const float2 v = *reinterpret_cast<const float2*>(o + static_cast<size_t>(s) * p.R);
-            a = fmaf(v.x, fac[s], a);
-            b = fmaf(v.y, fac[s], b);
+        for (int s = group; s < p.splits; s += 4) {
+            const float4 v = *reinterpret_cast<const float4*>(o + static_cast<size_t>(s) * p.R);
+            const float f = fac[s];
+            a.x = fmaf(v.x, f, a.x); a.y = fmaf(v.y, f, a.y); a.z = fmaf(v.z, f, a.z); a.w = fmaf(v.w, f, a.w);
         }
-        *reinterpret_cast<uint32_t*>(p.lat + unit * p.R + e) = pack_bf16(a * total, b * total);
+    }
+    part[group][col] = a;
+    __syncthreads();
+    if (group == 0 && 4 * col < p.R) {
+#pragma unroll
+        for (int g = 1; g < 4; ++g) { const float4 v = part[g][col]; a.x += v.x; a.y += v.y; a.z += v.z; a.w += v.w; }
+        const float t = total_s;
+        *reinterpret_cast<uint2*>(p.lat + unit * p.R + 4 * col) = make_uint2(pack_bf16(a.x * t, a.y * t), pack_bf16(a.z * t, a.w * t));
     }
 }
 
@@ -292,7 +315,7 @@ int launch_latent_tensor(const LatentParams& p, int rows, cudaStream_t st) {
     if (p.H > 16) e = tpw <= 1 ? launch<2, 1>(p, rows, st) : (tpw <= 2 ? launch<2, 2>(p, rows, st) : launch<2, 4>(p, rows, st));
     else e = tpw <= 1 ? launch<1, 1>(p, rows, st) : (tpw <= 2 ? launch<1, 2>(p, rows, st) : launch<1, 4>(p, rows, st));
     if (e != cudaSuccess) return TBL_ERR_CUDA;
-    if (p.splits > 1 && launch_dependent(latent_merge_kernel, dim3(rows, p.H), dim3(128), 0, st, p) != cudaSuccess) return TBL_ERR_CUDA;
+    if (p.splits > 1 && launch_dependent(latent_merge_kernel, dim3(rows, p.H), dim3(kMergeThreads), 0, st, p) != cudaSuccess) return TBL_ERR_CUDA;
     DenseCall v{};              // W_uv and the output gate
     v.x = p.lat; v.w = p.uv; v.ldx = p.H * p.R; v.M = rows; v.K = p.R; v.N = p.vd;
     v.out_b16 = static_cast<bf16*>(p.out); v.ldo = p.H * p.vd;
