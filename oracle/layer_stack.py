@@ -24,6 +24,11 @@ def silu(z):
     return z * sigmoid(z)
 
 
+def gelu_tanh(z):
+    z = np.asarray(z, F)
+    return 0.5 * z * (1.0 + np.tanh(np.sqrt(2.0 / np.pi) * (z + 0.044715 * z ** 3)))
+
+
 def linear(x, w, b=None):
     """Rows of x times W^T; W is stored [out, in]."""
     y = np.asarray(x, F) @ np.asarray(w, F).T
@@ -35,6 +40,11 @@ def rms_norm(x, w, eps):
     x = np.asarray(x, F)
     y = x / np.sqrt(np.mean(x * x, axis=-1, keepdims=True) + eps)
     return y if w is None else y * np.asarray(w, F)
+
+
+def dynamic_tanh(x, alpha, w, b):
+    """tanh(alpha x) w + b: a norm without statistics."""
+    return np.tanh(F(alpha) * np.asarray(x, F)) * np.asarray(w, F) + np.asarray(b, F)
 
 
 def embed(table, tokens, scale):
@@ -119,6 +129,54 @@ def latent_attention(h, P, p, cfg, eps, cache):
     return linear(out.reshape(T, H * vd) * sigmoid(linear(h, P[p + "g"])), P[p + "o"])
 
 
+def query_temperature(position, coef, every):
+    return 1.0 + coef * np.log(np.floor((position + 1) / every) + 1.0)
+
+
+def differential_lambda(P, p, diff):
+    dot = lambda a, b: float(np.sum(np.asarray(P[p + a], F) * np.asarray(P[p + b], F)))
+    return np.exp(dot("lq1", "lk1")) - np.exp(dot("lq2", "lk2")) + diff
+
+
+def differential_attention(h, P, p, cfg, eps, cache):
+    """Mixer: h [T, width]; cache is a list of (keys [G, 2, dim], values [G, vdim]), one entry per token of the sequence so
+    far.  A layer without a key projection finds the step's own tokens in it already."""
+    H, G, d, vd = (cfg[n] for n in ("heads", "kv_heads", "dim", "vdim"))
+    T = len(h)
+    q = linear(h, P[p + "q"], P[p + "q.b"]).reshape(T, H, 2, d)
+    if p + "k" in P:
+        k = linear(h, P[p + "k"], P[p + "k.b"]).reshape(T, G, 2, d)
+        v = linear(h, P[p + "v"], P[p + "v.b"]).reshape(T, G, vd)
+        cache.extend(zip(k, v))
+    first = len(cache) - T
+    keys, values = np.array([e[0] for e in cache]), np.array([e[1] for e in cache])
+    lam = differential_lambda(P, p, cfg["diff"])
+    o = np.zeros((T, H, vd))
+    for t in range(T):
+        n = first + t + 1
+        temp = query_temperature(first + t, cfg["q_temp"]["coef"], cfg["q_temp"]["every"])
+        for i in range(H):
+            g = i // (H // G)
+            a1, a2 = (softmax_attention(q[t, i, m] * temp, keys[:n, g, m], values[:n, g], cfg["scale"]) for m in (0, 1))
+            o[t, i] = rms_norm(a1 - lam * a2, None, eps) * (1.0 - cfg["diff"])
+    return linear(o.reshape(T, H * vd) * sigmoid(linear(h, P[p + "g"])), P[p + "o"], P[p + "o.b"])
+
+
+def streams_in(streams, weights):
+    """A sublayer's input: the weighted sum of the residual streams."""
+    return sum(F(w) * x for w, x in zip(np.asarray(weights, F), streams))
+
+
+def streams_out(streams, mix, out, y):
+    """The residual streams after a sublayer whose result is y; mix is indexed [from, to]."""
+    mix, out = np.asarray(mix, F), np.asarray(out, F)
+    return [sum(mix[s, t] * streams[s] for s in range(len(streams))) + out[t] * y for t in range(len(streams))]
+
+
+def gelu_ff(h, P, p):
+    return linear(gelu_tanh(linear(h, P[p + "gate"])) * linear(h, P[p + "up"]), P[p + "down"])
+
+
 def dense_ff(h, P, p):
     g = linear(h, P[p + "gate"], P[p + "gate.b"])
     u = linear(h, P[p + "up"], P[p + "up.b"])
@@ -154,3 +212,31 @@ class Decoder:
             if trace is not None:
                 trace.append(x.copy())
         return linear(rms_norm(x, P["final.norm"], eps), P["embed"])
+
+
+class StreamDecoder:
+    """The same for the design with several residual streams, Dynamic Tanh norms and differential attention (Goguvik)."""
+
+    def __init__(self, cfg: dict, params: Dict[str, np.ndarray]):
+        self.cfg, self.P = cfg, params
+        self.memory: List[list] = []
+        for layer in cfg["layers"]:
+            source = layer["mixer"].get("kv_from")
+            self.memory.append([] if source is None else self.memory[source])
+
+    def feed(self, tokens, trace: Optional[list] = None):
+        cfg, P, eps = self.cfg, self.P, self.cfg["norm"]["eps"]
+        norm = lambda x, name: dynamic_tanh(x, P[name + ".alpha"], P[name], P[name + ".b"])
+        xs = [embed(P["embed"], tokens, 1.0)] * cfg["streams"]
+        for i, layer in enumerate(cfg["layers"]):
+            p = f"l{i}."
+            sublayers = [lambda h: differential_attention(h, P, p + "mix.", layer["mixer"], eps, self.memory[i])]
+            if layer["mlp"] is not None:
+                sublayers.append(lambda h: gelu_ff(h, P, p + "mlp."))
+            for n, sublayer in enumerate(sublayers, 1):
+                hc = f"{p}hc{n}."
+                y = sublayer(norm(streams_in(xs, P[hc + "in"]), f"{p}norm{n}"))
+                xs = streams_out(xs, P[hc + "mix"], P[hc + "out"], y)
+            if trace is not None:
+                trace.append(sum(xs))
+        return linear(norm(sum(xs), "final.norm"), P["embed"])

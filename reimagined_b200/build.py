@@ -24,7 +24,8 @@ LIBRARIES = {
                  "edge_pack.cpp"]),
     "stack": (os.path.join(HERE, "libstack_b200.so"),
               ["runtime.cu", "stack.cu", "stack_glue.cu", "dense.cu", "dense_rows.cu", "dense_tcgen05.cu", "delta_rule.cu",
-               "latent_attention.cu", "latent_decode.cu", "latent_prefill.cu"]),
+               "latent_attention.cu", "latent_decode.cu", "latent_prefill.cu", "attention.cu", "attention_decode.cu",
+               "attention_prefill.cu"]),
 }
 LIB, SOURCES = LIBRARIES["ternary"]
 NVCC = os.environ.get("NVCC", "/usr/local/cuda/bin/nvcc")

@@ -105,11 +105,33 @@ class LatentMixer(C.Structure):
                 ("kv_rank", C.c_int), ("rope_positions", C.c_int), ("scale", C.c_float)]
 
 
+class AttentionMixer(C.Structure):
+    """tbl_attention_mixer."""
+
+    _fields_ = [("in_", DenseView), ("out", DenseView), ("temperature", C.c_void_p), ("temperature_positions", C.c_int), ("heads", C.c_int),
+                ("kv_heads", C.c_int), ("dim", C.c_int), ("vdim", C.c_int), ("maps", C.c_int), ("gated", C.c_int), ("kv_from", C.c_int),
+                ("scale", C.c_float), ("lambda_", C.c_float), ("out_scale", C.c_float)]
+
+
+class Hyper(C.Structure):
+    """tbl_hyper."""
+
+    _fields_ = [("in_", C.c_void_p), ("mix", C.c_void_p), ("out", C.c_void_p)]
+
+
+class TanhNorm(C.Structure):
+    """tbl_tanh_norm."""
+
+    _fields_ = [("bias", C.c_void_p), ("alpha", C.c_float)]
+
+
 class StackLayer(C.Structure):
     """tbl_stack_layer."""
 
     _fields_ = [("mixer", C.c_int), ("norm1", C.c_void_p), ("delta", DeltaMixer), ("latent", LatentMixer), ("ff", C.c_int),
-                ("norm2", C.c_void_p), ("gate_up", DenseView), ("down", DenseView), ("depth_weights", C.c_void_p)]
+                ("norm2", C.c_void_p), ("gate_up", DenseView), ("down", DenseView), ("depth_weights", C.c_void_p),
+                ("attention", AttentionMixer), ("tanh1", TanhNorm), ("tanh2", TanhNorm), ("hyper1", Hyper), ("hyper2", Hyper),
+                ("activation", C.c_int)]
 
 
 class StackModel(C.Structure):
@@ -117,11 +139,13 @@ class StackModel(C.Structure):
 
     _fields_ = [("width", C.c_int), ("vocab", C.c_int), ("n_layers", C.c_int), ("embedding", C.c_void_p),
                 ("embedding_scale", C.c_float), ("norm_eps", C.c_float), ("layers", C.POINTER(StackLayer)),
-                ("final_norm", C.c_void_p), ("head", DenseView)]
+                ("final_norm", C.c_void_p), ("head", DenseView), ("norm_kind", C.c_int), ("final_tanh", TanhNorm), ("streams", C.c_int)]
 
 
 F32, BF16 = 0, 1
-MIXER_GENERAL_DELTA, MIXER_LATENT_ATTENTION = 0, 1
+MIXER_GENERAL_DELTA, MIXER_LATENT_ATTENTION, MIXER_ATTENTION = 0, 1, 2
+NORM_RMS, NORM_DYNAMIC_TANH = 0, 1
+ACT_SILU, ACT_GELU_TANH = 0, 1
 PAIR_BLOCK = 32
 
 _vp = C.c_void_p
@@ -198,11 +222,18 @@ _STACK_SIGNATURES = {
                               _vp, _sz, _vp]),
     "tbl_dense_forward": (_int, [C.POINTER(DenseView), _int, _int, _vp, _int, _int, _vp, _vp, _vp]),
     "tbl_gated_dense_forward": (_int, [C.POINTER(DenseView), _int, _int, _vp, _int, _int, _int, _vp, _vp]),
+    "tbl_gated_dense_act_forward": (_int, [C.POINTER(DenseView), _int, _int, _int, _vp, _int, _int, _int, _vp, _vp]),
     "tbl_delta_workspace_bytes": (_sz, [C.POINTER(DeltaMixer), _int, _int]),
     "tbl_delta_forward": (_int, [C.POINTER(DeltaMixer), _int, _int, _float, _vp, _vp, _vp, _int, _int, _vp, _vp, _sz, _vp]),
     "tbl_latent_workspace_bytes": (_sz, [C.POINTER(LatentMixer), _int, _int, _int, _int]),
     "tbl_latent_forward": (_int, [C.POINTER(LatentMixer), _int, _int, _float, _vp, _vp, _int, _vp, _vp, _int, _int, _int, _vp,
                                   _vp, _sz, _vp]),
+    "tbl_attention_cache_width": (_int, [C.POINTER(AttentionMixer)]),
+    "tbl_attention_workspace_bytes": (_sz, [C.POINTER(AttentionMixer), _int, _int, _int, _int]),
+    "tbl_attention_forward": (_int, [C.POINTER(AttentionMixer), _int, _int, _float, _vp, _vp, _int, _int, _vp, _vp, _int, _int, _int,
+                                     _vp, _vp, _sz, _vp]),
+    "tbl_stream_norm": (_int, [_vp, _sz, _int, _vp, _vp, _vp, _int, _vp, _int, _vp, _int, _int, _int, _float, _float, _vp, _vp, _vp,
+                               _vp, _vp]),
     "tbl_depth_norm": (_int, [_vp, _sz, _int, _vp, _int, _vp, _int, _int, _float, _vp, _vp, _vp, _vp]),
 }
 STACK_SYMBOLS = tuple(_STACK_SIGNATURES)

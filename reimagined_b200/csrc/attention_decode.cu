@@ -1,0 +1,295 @@
+// Attention of a few query rows over a long cache (decode, short portions): the cache streams through shared memory once
+// per block of 16 query rows that share a key/value head.
+//
+// A CTA handles (sequence, kv head, block of rows, split of the context) in tiles of 64 tokens, brought in by cp.async a
+// few tiles ahead.  The products are warp-level MMAs (16 x 8 x 16, bf16): a warp owns one map and 16 tokens of every tile,
+// with its own maximum, sum and output, so that a tile costs one barrier; the quarters meet in shared memory at the end.
+// The scores' fragments become the weights' fragments in place, as two bf16 terms (hi + lo: 16 bits of mantissa).
+// With one split the CTA combines the maps, norms the head and gates the output itself; otherwise it leaves partial sums
+// for attention_merge_kernel.  A decode step appends its token here: the CTA whose split holds it writes it first.
+#include "attention.cuh"
+
+namespace tbl {
+namespace stack {
+namespace {
+
+constexpr int kTile = 64, kRows = 16, kQuarters = 4, kMaxStages = 4;
+
+__device__ __forceinline__ void ldsm4(uint32_t (&r)[4], uint32_t a) {
+    asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0,%1,%2,%3}, [%4];" : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(a));
+}
+__device__ __forceinline__ void ldsm4t(uint32_t (&r)[4], uint32_t a) {
+    asm volatile("ldmatrix.sync.aligned.m8n8.x4.trans.shared.b16 {%0,%1,%2,%3}, [%4];" : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(a));
+}
+__device__ __forceinline__ void mma(float (&d)[4], const uint32_t (&a)[4], uint32_t b0, uint32_t b1) {
+    mma16816(d, a[0], a[1], a[2], a[3], b0, b1);
+}
+__device__ __forceinline__ void cp16(uint32_t dst, const void* src, bool ok) {
+    asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(dst), "l"(src), "r"(ok ? 16 : 0) : "memory");
+}
+
+__host__ __device__ __forceinline__ int tile_ld(int cw) { return cw + 8; }      // an odd number of 16-byte units: conflict-free ldmatrix
+
+size_t query_smem(int maps, int dp) { return 2 * static_cast<size_t>(kRows) * maps * (dp + 8); }
+size_t tile_smem(int cw) { return 2 * static_cast<size_t>(kTile) * tile_ld(cw); }
+size_t merge_smem(int maps, int vp) { return sizeof(float) * kQuarters * maps * kRows * static_cast<size_t>(vp); }
+size_t stream_smem(int maps, int dp, int vp, int stages) {
+    const size_t tiles = stages * tile_smem(maps * dp + vp), merge = merge_smem(maps, vp);
+    return query_smem(maps, dp) + (tiles > merge ? tiles : merge);
+}
+
+// MAPS: maps per head; VN: value columns in steps of 16 a warp has room for
+template <int MAPS, int VN>
+__global__ void __launch_bounds__(32 * kQuarters * MAPS) attention_stream_kernel(const AttnParams p, const int stages) {
+    constexpr int kThreads = 32 * kQuarters * MAPS;
+    extern __shared__ __align__(16) uint8_t smem[];
+    __shared__ float m_s[kQuarters][MAPS][kRows], l_s[kQuarters][MAPS][kRows];
+    const int ld = tile_ld(p.cw), ldq = p.dp + 8;
+    bf16* q_s = reinterpret_cast<bf16*>(smem);                          // [MAPS][16][ldq]
+    bf16* t_s = q_s + MAPS * kRows * ldq;                               // [stages][64][ld]
+    float* o_s = reinterpret_cast<float*>(t_s);                         // afterwards: [quarter][MAPS][16][vp]
+    const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, map = warp % MAPS, quarter = warp / MAPS;
+    const int seq = blockIdx.x / p.G, g = blockIdx.x % p.G, first = blockIdx.y * kRows, split = blockIdx.z;
+    const int total = p.n_tok * p.group;
+    pdl_launch_dependents();
+    pdl_wait();
+    const int slot = p.slots[seq], pos0 = p.positions[slot];
+    const int n = min(pos0 + min(total - 1, first + kRows - 1) / p.group + 1, p.capacity);       // tokens the last row sees
+    const int per = ((n + p.splits - 1) / p.splits + kTile - 1) / kTile * kTile;
+    const int t0 = min(split * per, n), t1 = min(n, t0 + per);
+    bf16* cache = static_cast<bf16*>(p.cache) + cache_row(p, slot, g, 0);
+    if (p.append) {                                                     // n_tok == 1: the token at pos0
+        if (pos0 < 0 || pos0 >= p.capacity || (p.temperature && pos0 >= p.temperature_positions)) {
+            if (tid == 0 && split == 0) atomicOr(p.status, TBL_DEV_CACHE_FULL);
+        } else if (pos0 >= t0 && pos0 < t1) {
+            const float* pr = p.proj + static_cast<size_t>(seq) * p.ld;
+            for (int c = tid; c < p.cw; c += kThreads) cache[static_cast<size_t>(pos0) * p.cw + c] = __float2bfloat16_rn(cache_value(p, pr, g, c));
+            __syncthreads();                                            // the copies below read it
+        }
+    }
+    const int chunks = p.cw / 8;
+    auto load_tile = [&](int stage, int t) {
+        if (t < t1) {
+            const uint32_t base = smem_u32(t_s + stage * kTile * ld);
+            // a warp takes whole rows, its lanes the 16-byte pieces: no division per piece
+#pragma unroll 4
+            for (int r = warp; r < kTile; r += kQuarters * MAPS) {
+                const bool ok = t + r < t1;
+                const bf16* src = cache + static_cast<size_t>(ok ? t + r : 0) * p.cw;
+                for (int c = lane; c < chunks; c += 32) cp16(base + (r * ld + c * 8) * 2, src + c * 8, ok);
+            }
+        }
+        asm volatile("cp.async.commit_group;" ::: "memory");
+    };
+    for (int s = 0; s < kMaxStages - 1; ++s)
+        if (s < stages - 1) load_tile(s, t0 + s * kTile);
+    for (int i = tid; i < MAPS * kRows * p.dp; i += kThreads) {
+        const int r = i / (MAPS * p.dp), e = i - r * MAPS * p.dp, m = e / p.dp, c = e - m * p.dp, at = first + r;
+        float q = 0.0f;
+        if (at < total && c < p.d) {
+            const int t = at / p.group, head = g * p.group + at % p.group;
+            q = p.proj[(static_cast<size_t>(seq) * p.n_tok + t) * p.ld + (head * MAPS + m) * p.d + c] * temperature_of(p, pos0 + t);
+        }
+        q_s[(m * kRows + r) * ldq + c] = __float2bfloat16_rn(q);
+    }
+    float o[VN][2][4];
+#pragma unroll
+    for (int j = 0; j < VN; ++j)
+#pragma unroll
+        for (int e = 0; e < 8; ++e) o[j][e >> 2][e & 3] = 0.0f;
+    float mx[2] = {-INFINITY, -INFINITY}, sum[2] = {0.0f, 0.0f};       // rows lane / 4 and lane / 4 + 8; this lane's share of the sums
+    int last[2];                                                        // last token each of them sees
+#pragma unroll
+    for (int h = 0; h < 2; ++h) last[h] = min(pos0 + min(first + (lane >> 2) + 8 * h, total - 1) / p.group, t1 - 1);
+    const int tiles16 = p.vp / 16;
+    const uint32_t a_addr = smem_u32(q_s + (map * kRows + (lane & 15)) * ldq + (lane >> 4) * 8);
+    int stage = 0;
+    for (int t = t0; t < t1; t += kTile) {
+        if (stages == 2) asm volatile("cp.async.wait_group 0;" ::: "memory");
+        else if (stages == 3) asm volatile("cp.async.wait_group 1;" ::: "memory");
+        else asm volatile("cp.async.wait_group 2;" ::: "memory");
+        __syncthreads();                                     // the tile is there, and the one before it is no longer read
+        {
+            const int ahead = stage == 0 ? stages - 1 : stage - 1;
+            load_tile(ahead, t + (stages - 1) * kTile);
+        }
+        const bf16* tile = t_s + stage * kTile * ld + quarter * 16 * ld;
+        if (++stage == stages) stage = 0;
+        // scores: 16 rows x 16 tokens
+        float s[2][4] = {};
+        const uint32_t b_addr = smem_u32(tile + ((lane & 7) + (lane >> 4) * 8) * ld + map * p.dp + ((lane >> 3) & 1) * 8);
+#pragma unroll 4
+        for (int k = 0; k < p.dp; k += 16) {
+            uint32_t a[4], b[4];
+            ldsm4(a, a_addr + k * 2);
+            ldsm4(b, b_addr + k * 2);
+            mma(s[0], a, b[0], b[1]);
+            mma(s[1], a, b[2], b[3]);
+        }
+        const int token = t + quarter * 16 + (lane & 3) * 2;
+        uint32_t hi[4], lo[4];
+        float f[2];
+#pragma unroll
+        for (int h = 0; h < 2; ++h) {
+            float x[4];
+#pragma unroll
+            for (int e = 0; e < 4; ++e) x[e] = token + (e >> 1) * 8 + (e & 1) <= last[h] ? s[e >> 1][2 * h + (e & 1)] * p.scale_log2 : -INFINITY;
+            float top = fmaxf(fmaxf(x[0], x[1]), fmaxf(x[2], x[3]));
+            top = fmaxf(top, __shfl_xor_sync(0xffffffffu, top, 1));
+            top = fmaxf(top, __shfl_xor_sync(0xffffffffu, top, 2));
+            const float mn = fmaxf(mx[h], top), base = mn == -INFINITY ? 0.0f : mn;      // nothing seen yet: all weights zero
+            f[h] = ex2(mx[h] - base);
+            mx[h] = mn;
+#pragma unroll
+            for (int e = 0; e < 4; ++e) x[e] = ex2(x[e] - base);
+            sum[h] = fmaf(sum[h], f[h], (x[0] + x[1]) + (x[2] + x[3]));
+#pragma unroll
+            for (int e = 0; e < 2; ++e) {
+                hi[2 * e + h] = pack_bf16(x[2 * e], x[2 * e + 1]);
+                lo[2 * e + h] = pack_bf16(x[2 * e] - bf_lo(hi[2 * e + h]), x[2 * e + 1] - bf_hi(hi[2 * e + h]));
+            }
+        }
+        if (__any_sync(0xffffffffu, f[0] != 1.0f || f[1] != 1.0f)) {
+#pragma unroll
+            for (int j = 0; j < VN; ++j)
+#pragma unroll
+                for (int q = 0; q < 2; ++q) { o[j][q][0] *= f[0]; o[j][q][1] *= f[0]; o[j][q][2] *= f[1]; o[j][q][3] *= f[1]; }
+        }
+        const uint32_t v_addr = smem_u32(tile + (lane & 15) * ld + MAPS * p.dp + (lane >> 4) * 8);
+#pragma unroll
+        for (int j = 0; j < VN; ++j) {
+            if (j < tiles16) {
+                uint32_t b[4];
+                ldsm4t(b, v_addr + j * 32);
+                mma(o[j][0], hi, b[0], b[1]);
+                mma(o[j][1], hi, b[2], b[3]);
+                mma(o[j][0], lo, b[0], b[1]);
+                mma(o[j][1], lo, b[2], b[3]);
+            }
+        }
+    }
+    asm volatile("cp.async.wait_group 0;" ::: "memory");
+    __syncthreads();                                         // tiles are done with: their room takes the outputs
+#pragma unroll
+    for (int h = 0; h < 2; ++h) {
+        sum[h] += __shfl_xor_sync(0xffffffffu, sum[h], 1);
+        sum[h] += __shfl_xor_sync(0xffffffffu, sum[h], 2);
+        if ((lane & 3) == 0) { m_s[quarter][map][(lane >> 2) + 8 * h] = mx[h]; l_s[quarter][map][(lane >> 2) + 8 * h] = sum[h]; }
+    }
+    float* mine = o_s + static_cast<size_t>((quarter * MAPS + map) * kRows) * p.vp;
+#pragma unroll
+    for (int j = 0; j < VN; ++j)
+        if (j < tiles16) {
+#pragma unroll
+            for (int q = 0; q < 2; ++q)
+#pragma unroll
+                for (int h = 0; h < 2; ++h)
+                    *reinterpret_cast<float2*>(mine + ((lane >> 2) + 8 * h) * p.vp + j * 16 + q * 8 + (lane & 3) * 2) =
+                        make_float2(o[j][q][2 * h], o[j][q][2 * h + 1]);
+        }
+    __syncthreads();
+    // a warp per row
+    const size_t quarter_step = static_cast<size_t>(MAPS) * kRows * p.vp;
+    for (int r = warp; r < kRows; r += kQuarters * MAPS) {
+        const int at = first + r;
+        if (at >= total) break;
+        const int t = at / p.group, head = g * p.group + at % p.group;
+        const size_t row = static_cast<size_t>(seq) * p.n_tok + t, unit = (row * p.H + head) * MAPS;
+        float fac[MAPS][kQuarters];
+#pragma unroll
+        for (int m = 0; m < MAPS; ++m) {
+            float top = m_s[0][m][r], l = 0.0f;
+#pragma unroll
+            for (int k = 1; k < kQuarters; ++k) top = fmaxf(top, m_s[k][m][r]);
+#pragma unroll
+            for (int k = 0; k < kQuarters; ++k) {
+                fac[m][k] = m_s[k][m][r] == -INFINITY ? 0.0f : ex2(m_s[k][m][r] - top);
+                l = fmaf(l_s[k][m][r], fac[m][k], l);
+            }
+            if (p.splits > 1) {
+                if (lane == 0) { p.part_m[(unit + m) * p.splits + split] = top; p.part_l[(unit + m) * p.splits + split] = l; }
+            } else {
+                const float f = (m == 0 ? 1.0f : -p.lambda) / l;
+#pragma unroll
+                for (int k = 0; k < kQuarters; ++k) fac[m][k] *= f;
+            }
+        }
+        const float* src = o_s + static_cast<size_t>(r) * p.vp;
+        if (p.splits > 1) {
+#pragma unroll
+            for (int m = 0; m < MAPS; ++m) {
+                float* dst = p.part_o + ((unit + m) * p.splits + split) * p.vp;
+                for (int c = lane; c < p.vd; c += 32) {
+                    float v = 0.0f;
+#pragma unroll
+                    for (int k = 0; k < kQuarters; ++k) v = fmaf(src[k * quarter_step + m * kRows * p.vp + c], fac[m][k], v);
+                    dst[c] = v;
+                }
+            }
+            continue;
+        }
+        float v[VN / 2], ss = 0.0f;
+#pragma unroll
+        for (int i = 0; i < VN / 2; ++i) {
+            const int c = lane + 32 * i;
+            v[i] = 0.0f;
+            if (c < p.vd) {
+#pragma unroll
+                for (int m = 0; m < MAPS; ++m)
+#pragma unroll
+                    for (int k = 0; k < kQuarters; ++k) v[i] = fmaf(src[k * quarter_step + m * kRows * p.vp + c], fac[m][k], v[i]);
+            }
+            ss = fmaf(v[i], v[i], ss);
+        }
+        const float f = MAPS == 2 ? p.out_scale / sqrtf(warp_sum(ss) / static_cast<float>(p.vd) + p.eps) : 1.0f;
+        const float* gate = p.g_off < 0 ? nullptr : p.proj + row * p.ld + p.g_off + head * p.vd;
+        bf16* out = static_cast<bf16*>(p.out) + (row * p.H + head) * p.vd;
+#pragma unroll
+        for (int i = 0; i < VN / 2; ++i) {
+            const int c = lane + 32 * i;
+            if (c < p.vd) out[c] = __float2bfloat16_rn(v[i] * f * (gate ? sigmoid_f(gate[c]) : 1.0f));
+        }
+    }
+}
+
+int pick_stages(int maps, int dp, int vp) {
+    // two CTAs per SM where three tiles each allow it, one with what fits otherwise
+    for (int s = kMaxStages; s >= 2; --s)
+        if (stream_smem(maps, dp, vp, s) <= 110 * 1024) return s;
+    for (int s = kMaxStages; s >= 2; --s)
+        if (stream_smem(maps, dp, vp, s) <= 220 * 1024) return s;
+    return 0;
+}
+
+template <int MAPS, int VN>
+cudaError_t launch(const AttnParams& p, int n_seq, cudaStream_t st) {
+    static bool done[64] = {};
+    const int stages = pick_stages(MAPS, p.dp, p.vp);
+    const size_t smem = stream_smem(MAPS, p.dp, p.vp, stages);
+    const cudaError_t e = allow_smem(attention_stream_kernel<MAPS, VN>, smem, done);
+    if (e != cudaSuccess) return e;
+    const dim3 grid(n_seq * p.G, ceil_div(static_cast<long long>(p.n_tok) * p.group, kRows), p.splits);
+    if (grid.y > 65535) return cudaErrorInvalidValue;
+    return launch_dependent(attention_stream_kernel<MAPS, VN>, grid, dim3(32 * kQuarters * MAPS), smem, st, p, stages);
+}
+
+template <int MAPS>
+cudaError_t launch_vn(const AttnParams& p, int n_seq, cudaStream_t st) {
+    if (p.vp <= 64) return launch<MAPS, 4>(p, n_seq, st);
+    if (p.vp <= 128) return launch<MAPS, 8>(p, n_seq, st);
+    return launch<MAPS, 16>(p, n_seq, st);
+}
+
+}  // namespace
+
+bool attention_stream_supported(const tbl_attention_mixer& m) {
+    const int dp = static_cast<int>(round_up(m.dim, 16)), vp = static_cast<int>(round_up(m.vdim, 16));
+    return vp <= 256 && pick_stages(m.maps, dp, vp) > 0;
+}
+
+int launch_attention_stream(const AttnParams& p, int n_seq, cudaStream_t st) {
+    return (p.maps == 2 ? launch_vn<2>(p, n_seq, st) : launch_vn<1>(p, n_seq, st)) == cudaSuccess ? TBL_OK : TBL_ERR_CUDA;
+}
+
+}  // namespace stack
+}  // namespace tbl

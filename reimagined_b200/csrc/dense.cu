@@ -20,7 +20,7 @@ __device__ __forceinline__ void store_out(const DenseCall& c, int m, int n, floa
 // One output of a gated pair: rows g and g + 32 of the weight are the gate and up rows of output column n.
 __device__ __forceinline__ void store_pair(const DenseCall& c, int m, int n, int g, float gate, float up) {
     if (c.bias) { gate += __ldg(c.bias + g); up += __ldg(c.bias + g + TBL_PAIR_BLOCK); }
-    const float v = silu_f(gate) * up;
+    const float v = activate(activation_of(c.act), gate) * up;
     if (c.out_f32) c.out_f32[static_cast<size_t>(m) * c.ldo + n] = v;
     else c.out_b16[static_cast<size_t>(m) * c.ldo + n] = __float2bfloat16_rn(v);
 }
@@ -269,6 +269,12 @@ int tbl_dense_forward(const tbl_dense_view* view, int precision, int route, cons
 
 int tbl_gated_dense_forward(const tbl_dense_view* gate_up, int precision, int route, const void* x_dev, int ldx, int rows,
                             int ff, void* out_dev, void* stream) {
+    return tbl_gated_dense_act_forward(gate_up, precision, route, TBL_ACT_SILU, x_dev, ldx, rows, ff, out_dev, stream);
+}
+
+int tbl_gated_dense_act_forward(const tbl_dense_view* gate_up, int precision, int route, int activation, const void* x_dev, int ldx,
+                                int rows, int ff, void* out_dev, void* stream) {
+    if (activation != TBL_ACT_SILU && activation != TBL_ACT_GELU_TANH) return TBL_ERR_INVALID_ARG;
     if (!gate_up || !gate_up->weight || !x_dev || !out_dev || rows <= 0 || ff <= 0 || gate_up->inputs <= 0 ||
         ldx < gate_up->inputs || (precision != TBL_F32 && precision != TBL_BF16))
         return TBL_ERR_INVALID_ARG;
@@ -276,7 +282,7 @@ int tbl_gated_dense_forward(const tbl_dense_view* gate_up, int precision, int ro
     if (reinterpret_cast<uintptr_t>(gate_up->weight) & 15) return TBL_ERR_ALIGNMENT;
     DenseCall c{};
     c.x = x_dev; c.w = static_cast<const bf16*>(gate_up->weight); c.bias = gate_up->bias; c.ldx = ldx;
-    c.M = rows; c.K = gate_up->inputs; c.N = gate_up->outputs; c.ldo = ff; c.pair_cols = ff;
+    c.M = rows; c.K = gate_up->inputs; c.N = gate_up->outputs; c.ldo = ff; c.pair_cols = ff; c.act = activation;
     if (precision == TBL_BF16) c.out_b16 = static_cast<bf16*>(out_dev); else c.out_f32 = static_cast<float*>(out_dev);
     return launch_dense(precision, route, c, static_cast<cudaStream_t>(stream));
 }

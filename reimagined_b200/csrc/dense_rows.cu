@@ -106,7 +106,7 @@ __global__ void __launch_bounds__(32 * kWarps) dense_rows_kernel(const DenseCall
             for (int k = 0; k < wk; ++k) up += src[k * TA * 16 * LDP + 16 * LDP];
             const int gr = n / TBL_PAIR_BLOCK * 2 * TBL_PAIR_BLOCK + n % TBL_PAIR_BLOCK;
             if (c.bias) { v += __ldg(c.bias + gr); up += __ldg(c.bias + gr + TBL_PAIR_BLOCK); }
-            v = silu_f(v) * up;
+            v = activate(activation_of(c.act), v) * up;
         } else {
             if (c.bias) v += __ldg(c.bias + n);
         }

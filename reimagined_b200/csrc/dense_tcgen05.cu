@@ -8,7 +8,7 @@
 // are longer, and a tall tile cannot hide them.)
 // The epilogue adds the bias and either adds the fp32 residual and stores fp32, stores bf16, or -- for a gated
 // feed-forward, whose weight rows alternate in blocks of 32 gate and 32 up rows -- combines two neighbouring
-// 32-column blocks into silu(gate) * up and stores that.
+// 32-column blocks into act(gate) * up and stores that.
 // Every wait is bounded: on a timeout the role records the status word and falls through to the common exit, where
 // TMEM is released.
 #include <cuda.h>
@@ -194,6 +194,7 @@ dense_tcgen05_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_con
         const int half = (warp - 2) >> 2;      // which of the two warps of the quarter
         uint8_t* stage = epi_stage + (warp - 2) * 4096;
         const bool pair = p.c.pair_cols > 0;
+        const Activation act = activation_of(p.c.act);
         int local = 0, tile_row0, tn;
         bool alive = true;
         for (int tile = blockIdx.x; alive && decode_tile(p, tile, tile_row0, tn); tile += gridDim.x, ++local) {
@@ -225,7 +226,7 @@ dense_tcgen05_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_con
                     for (int i = 0; i < 32; ++i) {
                         const float g = __uint_as_float(r[i]) + __shfl_sync(0xffffffffu, bias_l, i);
                         const float u = __uint_as_float(rn[i]) + __shfl_sync(0xffffffffu, bias_u, i);
-                        v[i] = silu_f(g) * u;
+                        v[i] = activate(act, g) * u;
                     }
                     if (b + 4 < nblocks) tmem_ld32(t_row + (b + 4) * 32, r);
                     col0 = n0 >> 1;

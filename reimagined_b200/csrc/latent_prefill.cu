@@ -7,31 +7,22 @@
 //                           K-major form the second product wants
 //   latent_query_kernel     queries in bf16 with their rotated part rotated
 //   latent_prefill_kernel   256 queries of one head per CTA, two tiles of 128 that take turns on the tensor cores: while
-//                           one tile's four softmax warps work, the other tile's products run.  S = Q K^T accumulates in
-//                           TMEM; the weights go back into the columns S came from as two bf16 terms (p = hi + lo, both
-//                           multiplied: the weights keep 16 bits of mantissa and more), A operand of O += P V from TMEM.
-//                           Row maxima are only moved when they grow by 2^8 (then O and the sum are rescaled).
+//                           one tile's four softmax warps work, the other tile's products run (flash.cuh).
 // Roles: warps 0-3 and 4-7 softmax of tile 0 and 1 (a thread per query row), warp 8 TMA, warp 9 MMA issue.
 // Every wait is bounded; a role that gives up records the status word and falls through to the common exit.
 #include <cuda.h>
 
+#include "flash.cuh"
 #include "latent.cuh"
-#include "tc05.cuh"
 
 namespace tbl {
 namespace stack {
 namespace {
 
-using namespace tc05;
+using namespace flash;
 
-constexpr int kBlock = 128;                  // context tokens per block (and queries per tile)
-constexpr int kSubBytes = 128 * 128;         // a sub-tile: 128 rows x 64 bf16
 constexpr int kMaxSub = 3;                   // sub-tiles of a query or key tile: unrotated part, then rotated part
-constexpr int kSoftWarps = 8;
-constexpr int kThreads = 32 * (kSoftWarps + 2);
 constexpr int kMaxRing = 8;
-constexpr int kOCol = 256;                   // TMEM: S/P of tile w at 128 w, O of tile w at 256 + 128 w
-constexpr float kRescale = 8.0f;
 
 struct PrefillParams {
     const int32_t *slots, *positions;
@@ -41,8 +32,6 @@ struct PrefillParams {
     int ldg, H, d, rd, vd, n_tok, ctx, tiles, k_stages, v_stages;
     float scale_log2;
 };
-
-__device__ __forceinline__ float ex2(float x) { float r; asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(r) : "f"(x)); return r; }
 
 __global__ void __launch_bounds__(256) latent_gather_kernel(const bf16* __restrict__ cache, const int32_t* __restrict__ slots,
                                                             const int32_t* __restrict__ positions, int capacity, int cw, int n_tok,
@@ -106,7 +95,7 @@ latent_prefill_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_co
         fence_mbar_init();
         fence_proxy_async();
     }
-    if (warp == 9) {
+    if (warp == kMmaWarp) {
         asm volatile("tcgen05.alloc.cta_group::1.sync.aligned.shared::cta.b32 [%0], 512;" ::"r"(smem_u32(tmem_slot)) : "memory");
         asm volatile("tcgen05.relinquish_alloc_permit.cta_group::1.sync.aligned;" ::: "memory");
     }
@@ -130,7 +119,7 @@ latent_prefill_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_co
     const int nmax = max(nblk[0], nblk[1]);
     const int row_q = seq * p.n_tok + q0, row_k = seq * p.ctx;
 
-    if (warp == 8) {
+    if (warp == kTmaWarp) {
         // ---------------- TMA ----------------
         if (lane == 0) {
             const int tiles_q = nblk[1] > 0 ? 2 : 1, n = p.d + p.rd;
@@ -161,7 +150,7 @@ latent_prefill_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_co
                 }
             }
         }
-    } else if (warp == 9) {
+    } else if (warp == kMmaWarp) {
         // ---------------- MMA ----------------
         if (lane == 0) {
             const uint32_t is = idesc_bf16(kBlock), iv = idesc_bf16(p.vd);
@@ -174,15 +163,6 @@ latent_prefill_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_co
             const int nd = p.d / 16, nr = p.rd / 16;
             int ks = 0, v0 = 0, v1 = 1;       // ring slots of the next key block and of this block's value halves
             uint32_t kp = 0, vp0 = 0, vp1 = 0;
-            auto products = [&](uint32_t d_tmem, uint64_t a, uint64_t b, int n, uint32_t acc) {
-                for (; n >= 4; n -= 4, a += kSubBytes / 16, b += kSubBytes / 16, acc = 1) {
-                    umma_f16(d_tmem, a, b, is, acc);
-                    umma_f16(d_tmem, a + 2, b + 2, is, 1);
-                    umma_f16(d_tmem, a + 4, b + 4, is, 1);
-                    umma_f16(d_tmem, a + 6, b + 6, is, 1);
-                }
-                for (; n > 0; --n, a += 2, b += 2, acc = 1) umma_f16(d_tmem, a, b, is, acc);
-            };
             // The order S0(0) S1(0) | PV0(j) S0(j+1) PV1(j) S1(j+1) | ...: each softmax runs under the other tile's products.
             for (int j = -1; alive && j < nmax; ++j) {
 #pragma unroll
@@ -221,8 +201,8 @@ latent_prefill_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_co
                         }
                         const uint64_t a = q_desc + static_cast<uint64_t>(w) * (q_bytes / 16), b = k_desc + static_cast<uint64_t>(ks) * (k_bytes / 16);
                         const uint64_t rot = static_cast<uint64_t>(sub_d) * (kSubBytes / 16);
-                        products(tmem + w * kBlock, a, b, nd, 0);
-                        products(tmem + w * kBlock, a + rot, b + rot, nr, 1);
+                        products(tmem + w * kBlock, a, b, nd, is, 0);
+                        products(tmem + w * kBlock, a + rot, b + rot, nr, is, 1);
                         umma_commit(&s_full[w]);
                         if (w == 1 || jn >= nblk[1]) umma_commit(&k_empty[ks]);
                     }
@@ -252,63 +232,7 @@ latent_prefill_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_co
             alive = __all_sync(0xffffffffu, alive);
             if (!alive) break;
             tc_fence_after();
-            const int last = pos - j * kBlock;                 // last visible column of the block
-            const bool edge = __any_sync(0xffffffffu, last < kBlock - 1);
-            // the whole row at once: 128 scores in registers
-            uint32_t x[4][32];
-#pragma unroll
-            for (int ch = 0; ch < 4; ++ch) tmem_ld32(s_col + ch * 32, x[ch]);
-            tmem_ld_wait();
-            if (edge) {
-#pragma unroll
-                for (int ch = 0; ch < 4; ++ch)
-#pragma unroll
-                    for (int i = 0; i < 32; ++i)
-                        if (ch * 32 + i > last) x[ch][i] = 0xff800000u;         // -inf
-            }
-            float mx[4];
-#pragma unroll
-            for (int ch = 0; ch < 4; ++ch) {
-                mx[ch] = __uint_as_float(x[ch][0]);
-#pragma unroll
-                for (int i = 1; i < 32; ++i) mx[ch] = fmaxf(mx[ch], __uint_as_float(x[ch][i]));
-            }
-            const float top = fmaxf(fmaxf(mx[0], mx[1]), fmaxf(mx[2], mx[3])) * c;
-            if (j == 0) {
-                m = top;
-            } else if (__any_sync(0xffffffffu, top > m + kRescale)) {
-                const float mn = fmaxf(m, top), f = ex2(m - mn);
-                m = mn;
-                l *= f;
-#pragma unroll 1
-                for (int ch = 0; ch * 32 < p.vd; ++ch) {       // columns past vd are unused tensor memory
-                    uint32_t y[32];
-                    tmem_ld32(o_col + ch * 32, y);
-                    tmem_ld_wait();
-#pragma unroll
-                    for (int i = 0; i < 32; ++i) y[i] = __float_as_uint(__uint_as_float(y[i]) * f);
-                    tmem_st32(o_col + ch * 32, y);
-                }
-            }
-            float sum = 0.0f;
-#pragma unroll
-            for (int ch = 0; ch < 4; ++ch) {
-                float a0 = 0.0f, a1 = 0.0f;
-                uint32_t y[32];
-#pragma unroll
-                for (int i = 0; i < 16; ++i) {
-                    const float p0 = ex2(fmaf(__uint_as_float(x[ch][2 * i]), c, -m)), p1 = ex2(fmaf(__uint_as_float(x[ch][2 * i + 1]), c, -m));
-                    a0 += p0;
-                    a1 += p1;
-                    const uint32_t hi = pack_bf16(p0, p1);
-                    y[i] = hi;
-                    y[16 + i] = pack_bf16(p0 - bf_lo(hi), p1 - bf_hi(hi));
-                }
-                sum += a0 + a1;
-                tmem_st32(s_col + ch * 32, y);
-            }
-            l += sum;
-            tmem_st_wait();
+            softmax_block(s_col, o_col, p.vd, pos - j * kBlock, c, j == 0, m, l);
             tc_fence_before();
             __syncwarp();
             if (lane == 0) mbar_arrive(&p_full[w]);
@@ -350,7 +274,7 @@ latent_prefill_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_co
 
     tc_fence_before();
     __syncthreads();
-    if (warp == 9) {
+    if (warp == kMmaWarp) {
         tc_fence_after();
         asm volatile("tcgen05.dealloc.cta_group::1.sync.aligned.b32 %0, 512;" ::"r"(tmem) : "memory");
     }

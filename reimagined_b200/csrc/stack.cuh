@@ -25,7 +25,14 @@ template <> __device__ __forceinline__ float from_f<float>(float v) { return v; 
 template <> __device__ __forceinline__ bf16 from_f<bf16>(float v) { return __float2bfloat16_rn(v); }
 
 __device__ __forceinline__ float sigmoid_f(float z) { return 1.0f / (1.0f + expf(-z)); }
-__device__ __forceinline__ float silu_f(float z) { return z * sigmoid_f(z); }
+
+// Activation of a gated feed-forward, TBL_ACT_*: z sigmoid(z (lin + cubic z^2)).  With (1, 0) that is silu; the tanh form
+// of gelu is z (1 + tanh(a)) / 2 = z sigmoid(2 a), a = sqrt(2/pi) (z + 0.044715 z^3).
+struct Activation { float lin, cubic; };
+__device__ __forceinline__ Activation activation_of(int act) {
+    return act == TBL_ACT_GELU_TANH ? Activation{1.5957691216f, 0.0713548163f} : Activation{1.0f, 0.0f};
+}
+__device__ __forceinline__ float activate(const Activation& a, float z) { return z * sigmoid_f(z * fmaf(z * z, a.cubic, a.lin)); }
 
 // the two bf16 halves of a 32-bit word, widened
 __device__ __forceinline__ float bf_lo(uint32_t w) { return __uint_as_float(w << 16); }
@@ -67,14 +74,17 @@ cudaError_t launch_dependent(void (*kernel)(Params...), dim3 grid, dim3 block, s
     return e;
 }
 
-// Raises a kernel's dynamic shared memory limit once per device.
+// Raises a kernel's dynamic shared memory limit once per device, to what its static shared memory leaves.
 template <typename Kernel>
 cudaError_t allow_smem(Kernel kernel, size_t bytes, bool (&done)[64]) {
     if (bytes <= 48 * 1024) return cudaSuccess;
     int dev = 0;
     cudaGetDevice(&dev);
     if (dev >= 0 && dev < 64 && done[dev]) return cudaSuccess;
-    const cudaError_t e = cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, 227 * 1024);
+    cudaFuncAttributes attr{};
+    cudaError_t e = cudaFuncGetAttributes(&attr, kernel);
+    if (e == cudaSuccess)
+        e = cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, 227 * 1024 - static_cast<int>(attr.sharedSizeBytes));
     if (e == cudaSuccess && dev >= 0 && dev < 64) done[dev] = true;
     return e;
 }
@@ -89,8 +99,9 @@ struct DenseCall {
     bf16* out_b16;
     int ldo;
     const float* residual;   // fp32, ld = ldo, added to out_f32 (may alias it); null: none
-    int pair_cols;           // > 0: rows of w alternate in blocks of 32 gate / 32 up rows, out = silu(gate) * up,
+    int pair_cols;           // > 0: rows of w alternate in blocks of 32 gate / 32 up rows, out = act(gate) * up,
                              //      clipped at this many columns
+    int act;                 // TBL_ACT_*
     // row-streaming kernel only: `batch` products of one launch (0: one), their strides in elements, and an output
     // gate: out *= sigmoid(gate[m * ldg + n])
     int batch, ldg, batch_gate;
@@ -117,6 +128,14 @@ struct DepthNorm {
     const int32_t* row_index;
     int rows, width;
     float eps;
+    // streams > 0: the source are this many residual streams instead, updated with the last sublayer's result first;
+    // `weights` then make the sublayer input out of them (null: ones) and `trace` receives their plain sum
+    int streams, store;      // store: write the updated streams back (embedding: write them)
+    float* stream;           // [streams] arrays at `stride`
+    const float *y, *mix, *out_weights;      // y null: no update
+    int norm_kind;           // TBL_NORM_*
+    float alpha;
+    const float* norm_bias;
     const float* norm;       // null: no h
     float* x;
     float* trace;
@@ -138,6 +157,14 @@ int launch_latent(const tbl_latent_mixer& m, int precision, int route, float eps
                   int capacity, const int32_t* slots, const int32_t* positions, int n_seq, int n_tok, int context,
                   void* out, void* ws, cudaStream_t st);
 int latent_cache_width(const tbl_latent_mixer& m);     // cached numbers per token, padded to 16 bytes of bf16
+// ---- attention.cu --------------------------------------------------------------------------------------------------
+size_t attention_workspace(const tbl_attention_mixer& m, int precision, int n_seq, int n_tok, int context);
+int launch_attention(const tbl_attention_mixer& m, int precision, int route, float eps, const float* proj, void* cache, int n_slots,
+                     int capacity, const int32_t* slots, const int32_t* positions, int n_seq, int n_tok, int context, void* out,
+                     void* ws, cudaStream_t st);
+int attention_cache_width(const tbl_attention_mixer& m);      // cached numbers per token and key/value head
+int check_attention(const tbl_attention_mixer& m, int width);
+
 int check_delta(const tbl_delta_mixer& m, int width);
 int check_latent(const tbl_latent_mixer& m, int width);
 

@@ -33,6 +33,7 @@ def _load_hybrid(folder, cfg, dtype, slots, capacity):
 
 MODELS: Dict[str, Entry] = {
     "Guselix": Entry("stack", ("bfloat16", "float32"), _load_stack),
+    "Goguvik": Entry("stack", ("bfloat16", "float32"), _load_stack),
     # the Mamba-2 / attention hybrid on ternary weights: params.npz holds DecodeEngine's parameter set
     "JambaHybrid": Entry("ternary", ("bfloat16",), _load_hybrid),
 }

@@ -6,19 +6,22 @@ A design is a list of layers in its configuration; every layer names its mixer a
      "layers": [{"type": <mixer>, "mixer": {sizes and constants}, "mlp": {"kind": "dense", "ff": ..} or null}, ...]}
 
 `MIXERS` maps a mixer's name to the code that says which tensors it has and how they become the library's descriptor,
-so another design that uses the same mixers in another order needs no new code.  `StackEngine` owns the device state of
-a number of sequences (slots) and runs steps: portions of prompts and decode steps of several sequences, the latter
-replayed from CUDA graphs.  torch owns device memory and streams only.
+and `DESIGNS` an architecture to what surrounds its mixers (norm, residual, feed-forward), so another design that uses the
+same mechanisms in another order needs no new code.  `StackEngine` owns the device state of a number of sequences (slots)
+and runs steps: portions of prompts and decode steps of several sequences, the latter replayed from CUDA graphs.  torch
+owns device memory and streams only.
 
 Guselix is this family with the mixers `general_delta` (delta rule with per-channel decay and removal rate) and
-`latent_attention`, and a learned average over the depth after every layer.
+`latent_attention`, RMS norms and a learned average over the depth after every layer.  Goguvik has the mixer `attention`
+(differential, grouped key/value heads, query temperature, layers that read an earlier layer's cache), Dynamic Tanh norms
+and several residual streams ("streams") joined by hyper-connections.
 """
 from __future__ import annotations
 
 import ctypes as C
 import math
 import os
-from typing import Callable, Dict, Iterable, List, NamedTuple, Optional, Sequence, Tuple
+from typing import Callable, Dict, Iterable, List, NamedTuple, Optional, Sequence, Set, Tuple
 
 import numpy as np
 import torch
@@ -79,39 +82,113 @@ def _fill_latent(e: "StackEngine", layer: capi.StackLayer, p: str, m: dict) -> N
     a.rope_cos, a.rope_sin = e.rotation(float(m["rot"]["base"]), m["rot_dim"])
 
 
+def _attention_shapes(m: dict, width: int, rank: int) -> Shapes:
+    h, g, d, vd = (m[n] for n in ("heads", "kv_heads", "dim", "vdim"))
+    rows = {"q": h * 2 * d}
+    if m.get("kv_from") is None:
+        rows.update(k=g * 2 * d, v=g * vd)
+    out = {name: (n, width) for name, n in rows.items()}
+    out.update({name + ".b": (n,) for name, n in rows.items()})
+    out.update({name: (d,) for name in ("lq1", "lk1", "lq2", "lk2")})
+    return {**out, "g": (h * vd, width), "o": (width, h * vd), "o.b": (width,)}
+
+
+def _fill_attention(e: "StackEngine", layer: capi.StackLayer, p: str, m: dict) -> None:
+    a, w, source = layer.attention, e.weights, m.get("kv_from")
+    layer.mixer = capi.MIXER_ATTENTION
+    a.heads, a.kv_heads, a.dim, a.vdim, a.maps, a.gated = m["heads"], m["kv_heads"], m["dim"], m["vdim"], 2, 1
+    a.scale, a.kv_from = float(m["scale"]), -1 if source is None else source
+    names = ["q"] if source is not None else ["q", "k", "v"]
+    bias = torch.cat([w[p + n + ".b"].float() for n in names] + [torch.zeros(m["heads"] * m["vdim"])])
+    a.in_ = e.dense([p + n for n in names + ["g"]], bias)
+    a.out = e.dense([p + "o"], w[p + "o.b"])
+    dot = lambda x, y: float((w[p + x].double() * w[p + y].double()).sum())
+    a.lambda_ = math.exp(dot("lq1", "lk1")) - math.exp(dot("lq2", "lk2")) + float(m["diff"])
+    a.out_scale = 1.0 - float(m["diff"])
+    if m.get("q_temp") is not None:
+        a.temperature, a.temperature_positions = e.query_temperature(float(m["q_temp"]["coef"]), m["q_temp"]["every"]), e.capacity
+
+
 MIXERS: Dict[str, Mixer] = {
     "general_delta": Mixer(_delta_shapes, _fill_delta),
     "latent_attention": Mixer(_latent_shapes, _fill_latent),
+    "attention": Mixer(_attention_shapes, _fill_attention),
 }
+
+
+class Design(NamedTuple):
+    """What an architecture fixes around its mixers."""
+    norm: int                     # capi.NORM_*
+    activation: int               # capi.ACT_* of the feed-forward
+    ff_bias: bool
+    depth_average: bool           # learned average over the depth after every layer
+    streams: bool                 # several residual streams with hyper-connections; their number is in the configuration
+
+
+DESIGNS: Dict[str, Design] = {
+    "Guselix": Design(capi.NORM_RMS, capi.ACT_SILU, ff_bias=True, depth_average=True, streams=False),
+    "Goguvik": Design(capi.NORM_DYNAMIC_TANH, capi.ACT_GELU_TANH, ff_bias=False, depth_average=False, streams=True),
+}
+
+
+def design_of(cfg: dict) -> Design:
+    if cfg["architecture"] not in DESIGNS:
+        raise ValueError(f"no layer-stack design named {cfg['architecture']!r}")
+    return DESIGNS[cfg["architecture"]]
+
+
+def _sublayer_shapes(design: Design, cfg: dict, p: str, n: int) -> Shapes:
+    """The tensors around sublayer n (1: mixer, 2: feed-forward) of a layer."""
+    out = _norm_shapes(design, f"{p}norm{n}", cfg["width"])
+    if design.streams:
+        s = cfg["streams"]
+        out.update({f"{p}hc{n}.in": (s,), f"{p}hc{n}.out": (s,), f"{p}hc{n}.mix": (s, s)})
+    return out
+
+
+def _norm_shapes(design: Design, name: str, width: int) -> Shapes:
+    out = {name: (width,)}
+    if design.norm == capi.NORM_DYNAMIC_TANH:
+        out.update({name + ".b": (width,), name + ".alpha": ()})
+    return out
 
 
 def tensor_shapes(cfg: dict, ranks: Sequence[int]) -> Shapes:
     """Every tensor of a configuration; ranks[i] is the rank of layer i's low-rank decay (it is not in the
     configuration: the tensor's shape gives it)."""
-    width, out = cfg["width"], {"embed": (cfg["vocab"], cfg["width"]), "final.norm": (cfg["width"],)}
+    design, width = design_of(cfg), cfg["width"]
+    out = {"embed": (cfg["vocab"], width), **_norm_shapes(design, "final.norm", width)}
     for i, layer in enumerate(cfg["layers"]):
         p = f"l{i}."
         if layer["type"] not in MIXERS:
             raise ValueError(f"layer {i}: no mixer named {layer['type']!r}")
-        out[p + "norm1"] = (width,)
+        out.update(_sublayer_shapes(design, cfg, p, 1))
         for name, shape in MIXERS[layer["type"]].shapes(layer["mixer"], width, ranks[i]).items():
             out[p + "mix." + name] = shape
         if layer["mlp"] is not None:
             if layer["mlp"]["kind"] != "dense":
                 raise ValueError(f"layer {i}: no feed-forward of the kind {layer['mlp']['kind']!r}")
             ff = layer["mlp"]["ff"]
-            out[p + "norm2"] = (width,)
+            out.update(_sublayer_shapes(design, cfg, p, 2))
             for name, shape in (("gate", (ff, width)), ("up", (ff, width)), ("down", (width, ff))):
                 out[p + "mlp." + name] = shape
-                out[p + "mlp." + name + ".b"] = shape[:1]
-        out[p + "dwa"] = (i + 2,)
+                if design.ff_bias:
+                    out[p + "mlp." + name + ".b"] = shape[:1]
+        if design.depth_average:
+            out[p + "dwa"] = (i + 2,)
     return out
+
+
+def _unused_tensors(cfg: dict) -> Set[str]:
+    """Tensors that a checkpoint may hold although nothing reads them: around the feed-forward a layer does not have."""
+    design = design_of(cfg)
+    return {name for i, layer in enumerate(cfg["layers"]) if layer["mlp"] is None for name in _sublayer_shapes(design, cfg, f"l{i}.", 2)}
 
 
 def check_weights(cfg: dict, weights: Dict[str, torch.Tensor]) -> None:
     ranks = [weights[f"l{i}.mix.w1"].shape[0] if f"l{i}.mix.w1" in weights else 0 for i in range(len(cfg["layers"]))]
     want = tensor_shapes(cfg, ranks)
-    missing, extra = sorted(set(want) - set(weights)), sorted(set(weights) - set(want))
+    missing, extra = sorted(set(want) - set(weights)), sorted(set(weights) - set(want) - _unused_tensors(cfg))
     if missing or extra:
         raise ValueError(f"weights do not fit the configuration: missing {missing[:5]}, unknown {extra[:5]}")
     for name, shape in want.items():
@@ -128,6 +205,14 @@ def synthetic_weights(cfg: dict, seed: int = 1, rank: int = 16, device: str = "c
         if name.endswith("dwa"):
             w = 0.1 * w
             w[-1] += 1.0
+        elif ".hc" in name:
+            w = 0.2 * w + (torch.eye(shape[0], device=device) if name.endswith(".mix") else 1.0 / shape[0] if name.endswith(".in") else 1.0)
+        elif name.endswith(".alpha"):
+            w = 0.5 + 0.1 * w.clamp(-3.0, 3.0)
+        elif name.endswith(".b"):
+            w = 0.1 * w
+        elif ".mix.l" in name:
+            w = 0.5 * shape[0] ** -0.5 * w
         elif name.endswith("norm") or ".norm" in name:
             w = 1.0 + 0.1 * w
         elif len(shape) == 2 and name != "embed":
@@ -150,12 +235,13 @@ class StackEngine:
             raise RuntimeError("layer-stack models run on CUDA devices only (no CPU fallback)")
         check_weights(cfg, weights)
         self.L = capi.stack_lib()
-        self.cfg, self.weights = cfg, weights
+        self.cfg, self.weights, self.design = cfg, weights, design_of(cfg)
         self.precision = {"float32": capi.F32, "bfloat16": capi.BF16}[dtype]
         self.slots, self.capacity, self.graphs = int(slots), int(capacity), graphs
         self.vocab, self.width, self.n_layers = cfg["vocab"], cfg["width"], len(cfg["layers"])
         self._keep: List[torch.Tensor] = []
         self._rotations: Dict[Tuple[float, int], Tuple[int, int]] = {}
+        self._temperatures: Dict[tuple, int] = {}
         self._build()
         del self.weights
         m = C.byref(self.model)
@@ -194,6 +280,25 @@ class StackEngine:
             self._rotations[base, dims] = self.f32(torch.from_numpy(np.cos(ang))), self.f32(torch.from_numpy(np.sin(ang)))
         return self._rotations[base, dims]
 
+    def query_temperature(self, coef: float, every) -> int:
+        """1 + coef * ln(floor((position + 1) / every) + 1), worked out in double precision."""
+        if (coef, every) not in self._temperatures:
+            steps = np.floor_divide(np.arange(1, self.capacity + 1), every)
+            self._temperatures[coef, every] = self.f32(torch.from_numpy(1.0 + coef * np.log(steps + 1.0)))
+        return self._temperatures[coef, every]
+
+    def norm(self, name: str) -> Tuple[int, capi.TanhNorm]:
+        """A norm's weight, and what Dynamic Tanh has beside it."""
+        extra = capi.TanhNorm()
+        if self.design.norm == capi.NORM_DYNAMIC_TANH:
+            extra.bias, extra.alpha = self.f32(self.weights[name + ".b"]), float(self.weights[name + ".alpha"])
+        return self.f32(self.weights[name]), extra
+
+    def hyper(self, prefix: str) -> capi.Hyper:
+        if not self.design.streams:
+            return capi.Hyper()
+        return capi.Hyper(*(self.f32(self.weights[prefix + n]) for n in ("in", "mix", "out")))
+
     def _paired(self, gate: torch.Tensor, up: torch.Tensor) -> torch.Tensor:
         """Gate and up rows in alternating blocks, the last block filled with zero rows."""
         b = capi.PAIR_BLOCK
@@ -210,23 +315,27 @@ class StackEngine:
         self._layers = (capi.StackLayer * self.n_layers)()
         for i, c in enumerate(cfg["layers"]):
             layer, p = self._layers[i], f"l{i}."
-            layer.norm1 = self.f32(w[p + "norm1"])
+            layer.norm1, layer.tanh1 = self.norm(p + "norm1")
+            layer.hyper1 = self.hyper(p + "hc1.")
             MIXERS[c["type"]].fill(self, layer, p + "mix.", c["mixer"])
             if c["mlp"] is not None:
-                layer.ff = c["mlp"]["ff"]
-                layer.norm2 = self.f32(w[p + "norm2"])
+                layer.ff, layer.activation = c["mlp"]["ff"], self.design.activation
+                layer.norm2, layer.tanh2 = self.norm(p + "norm2")
+                layer.hyper2 = self.hyper(p + "hc2.")
                 gu = self._bf16(self._paired(w[p + "mlp.gate"], w[p + "mlp.up"]))
-                bias = self._paired(w[p + "mlp.gate.b"], w[p + "mlp.up.b"])
-                layer.gate_up = capi.DenseView(gu.data_ptr(), self.f32(bias), gu.shape[1], gu.shape[0])
-                layer.down = self.dense([p + "mlp.down"], w[p + "mlp.down.b"])
-            layer.depth_weights = self.f32(w[p + "dwa"])
+                bias = self.f32(self._paired(w[p + "mlp.gate.b"], w[p + "mlp.up.b"])) if self.design.ff_bias else None
+                layer.gate_up = capi.DenseView(gu.data_ptr(), bias, gu.shape[1], gu.shape[0])
+                layer.down = self.dense([p + "mlp.down"], w[p + "mlp.down.b"] if self.design.ff_bias else None)
+            if self.design.depth_average:
+                layer.depth_weights = self.f32(w[p + "dwa"])
         model = capi.StackModel()
         model.width, model.vocab, model.n_layers = self.width, self.vocab, self.n_layers
         embed = self._bf16(w["embed"])
-        model.embedding, model.embedding_scale = embed.data_ptr(), float(cfg["embedding"]["scale"])
-        model.norm_eps = float(cfg["norm"]["eps"])
+        model.embedding, model.embedding_scale = embed.data_ptr(), float(cfg.get("embedding", {}).get("scale", 1.0))
+        model.norm_kind, model.norm_eps = self.design.norm, float(cfg["norm"]["eps"])
+        model.streams = cfg["streams"] if self.design.streams else 0
         model.layers = C.cast(self._layers, C.POINTER(capi.StackLayer))
-        model.final_norm = self.f32(w["final.norm"])
+        model.final_norm, model.final_tanh = self.norm("final.norm")
         model.head = capi.DenseView(embed.data_ptr(), None, self.width, self.vocab)
         self.model = model
 
