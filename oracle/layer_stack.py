@@ -138,28 +138,35 @@ def differential_lambda(P, p, diff):
     return np.exp(dot("lq1", "lk1")) - np.exp(dot("lq2", "lk2")) + diff
 
 
-def differential_attention(h, P, p, cfg, eps, cache):
-    """Mixer: h [T, width]; cache is a list of (keys [G, 2, dim], values [G, vdim]), one entry per token of the sequence so
-    far.  A layer without a key projection finds the step's own tokens in it already."""
+def differential_output(a1, a2, lam, diff, eps):
+    return rms_norm(a1 - lam * a2, None, eps) * (1.0 - diff)
+
+
+def grouped_attention(h, P, p, cfg, eps, cache):
+    """Mixer: h [T, width]; cache is a list of (keys [G, maps, dim], values [G, vdim]), one entry per token of the sequence
+    so far.  A layer without a key projection finds the step's own tokens in it already.  With "diff" in the configuration
+    every head has two maps, whose difference is normed (differential attention)."""
     H, G, d, vd = (cfg[n] for n in ("heads", "kv_heads", "dim", "vdim"))
-    T = len(h)
-    q = linear(h, P[p + "q"], P[p + "q.b"]).reshape(T, H, 2, d)
+    T, maps = len(h), 2 if "diff" in cfg else 1
+    project = lambda name: linear(h, P[p + name], P.get(p + name + ".b"))
+    q = project("q").reshape(T, H, maps, d)
     if p + "k" in P:
-        k = linear(h, P[p + "k"], P[p + "k.b"]).reshape(T, G, 2, d)
-        v = linear(h, P[p + "v"], P[p + "v.b"]).reshape(T, G, vd)
-        cache.extend(zip(k, v))
+        cache.extend(zip(project("k").reshape(T, G, maps, d), project("v").reshape(T, G, vd)))
     first = len(cache) - T
     keys, values = np.array([e[0] for e in cache]), np.array([e[1] for e in cache])
-    lam = differential_lambda(P, p, cfg["diff"])
     o = np.zeros((T, H, vd))
     for t in range(T):
-        n = first + t + 1
-        temp = query_temperature(first + t, cfg["q_temp"]["coef"], cfg["q_temp"]["every"])
+        n, temp = first + t + 1, 1.0
+        if "q_temp" in cfg:
+            temp = query_temperature(first + t, cfg["q_temp"]["coef"], cfg["q_temp"]["every"])
         for i in range(H):
             g = i // (H // G)
-            a1, a2 = (softmax_attention(q[t, i, m] * temp, keys[:n, g, m], values[:n, g], cfg["scale"]) for m in (0, 1))
-            o[t, i] = rms_norm(a1 - lam * a2, None, eps) * (1.0 - cfg["diff"])
-    return linear(o.reshape(T, H * vd) * sigmoid(linear(h, P[p + "g"])), P[p + "o"], P[p + "o.b"])
+            a = [softmax_attention(q[t, i, m] * temp, keys[:n, g, m], values[:n, g], cfg["scale"]) for m in range(maps)]
+            o[t, i] = a[0] if maps == 1 else differential_output(a[0], a[1], differential_lambda(P, p, cfg["diff"]), cfg["diff"], eps)
+    o = o.reshape(T, H * vd)
+    if p + "g" in P:
+        o = o * sigmoid(linear(h, P[p + "g"]))
+    return linear(o, P[p + "o"], P.get(p + "o.b"))
 
 
 def streams_in(streams, weights):
@@ -230,7 +237,7 @@ class StreamDecoder:
         xs = [embed(P["embed"], tokens, 1.0)] * cfg["streams"]
         for i, layer in enumerate(cfg["layers"]):
             p = f"l{i}."
-            sublayers = [lambda h: differential_attention(h, P, p + "mix.", layer["mixer"], eps, self.memory[i])]
+            sublayers = [lambda h: grouped_attention(h, P, p + "mix.", layer["mixer"], eps, self.memory[i])]
             if layer["mlp"] is not None:
                 sublayers.append(lambda h: gelu_ff(h, P, p + "mlp."))
             for n, sublayer in enumerate(sublayers, 1):
@@ -240,3 +247,7 @@ class StreamDecoder:
             if trace is not None:
                 trace.append(sum(xs))
         return linear(norm(sum(xs), "final.norm"), P["embed"])
+
+
+def decoder(cfg: dict, params: Dict[str, np.ndarray]):
+    return (StreamDecoder if "streams" in cfg else Decoder)(cfg, params)

@@ -97,11 +97,10 @@ struct DenseCall {
     int ldx, M, K, N, ldw;
     float* out_f32;          // exactly one of the two outputs
     bf16* out_b16;
-    int ldo;
+    int ldo, act;            // act: TBL_ACT_* of a gated pair
     const float* residual;   // fp32, ld = ldo, added to out_f32 (may alias it); null: none
     int pair_cols;           // > 0: rows of w alternate in blocks of 32 gate / 32 up rows, out = act(gate) * up,
                              //      clipped at this many columns
-    int act;                 // TBL_ACT_*
     // row-streaming kernel only: `batch` products of one launch (0: one), their strides in elements, and an output
     // gate: out *= sigmoid(gate[m * ldg + n])
     int batch, ldg, batch_gate;

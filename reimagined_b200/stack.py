@@ -99,7 +99,7 @@ def _fill_attention(e: "StackEngine", layer: capi.StackLayer, p: str, m: dict) -
     a.heads, a.kv_heads, a.dim, a.vdim, a.maps, a.gated = m["heads"], m["kv_heads"], m["dim"], m["vdim"], 2, 1
     a.scale, a.kv_from = float(m["scale"]), -1 if source is None else source
     names = ["q"] if source is not None else ["q", "k", "v"]
-    bias = torch.cat([w[p + n + ".b"].float() for n in names] + [torch.zeros(m["heads"] * m["vdim"])])
+    bias = torch.cat([w[p + n + ".b"].float() for n in names] + [w[p + "q.b"].new_zeros(m["heads"] * m["vdim"]).float()])
     a.in_ = e.dense([p + n for n in names + ["g"]], bias)
     a.out = e.dense([p + "o"], w[p + "o.b"])
     dot = lambda x, y: float((w[p + x].double() * w[p + y].double()).sum())

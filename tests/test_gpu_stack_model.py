@@ -54,12 +54,12 @@ def test_prompt_matches_oracle(name, dtype):
     S.close(run(e, ids, [len(ids)]), want, dtype)
 
 
-@pytest.mark.parametrize("name", ["odd", "even"])
+@pytest.mark.parametrize("name", ["odd", "even", "diff_odd", "diff_even"])
 def test_residual_stream_after_every_layer(name):
-    from oracle.layer_stack import Decoder
+    from oracle.layer_stack import decoder
     e, p = S.engine(name)
     ids, layers = S.tokens(name, 30, 4), []
-    Decoder(S.CONFIGS[name], p).feed(ids, layers)
+    decoder(S.CONFIGS[name], p).feed(ids, layers)
     slot = e.open()
     _, hidden = e.step([slot], [ids], trace=True)
     for got, want in zip(hidden.cpu().numpy(), layers):
@@ -75,7 +75,7 @@ def test_token_by_token_matches_oracle(name, dtype):
 
 
 @pytest.mark.parametrize("dtype", DTYPES)
-@pytest.mark.parametrize("name", ["odd", "even", "wide"])
+@pytest.mark.parametrize("name", ["odd", "even", "wide", "diff_odd", "diff_even", "diff_wide"])
 @pytest.mark.parametrize("cuts", [[2] * 75, [37, 2, 3, 1, 64, 2, 41], [3, 48, 47, 49, 3], [16, 1, 15, 17, 1, 100], [128, 2, 20], [149, 1]])
 def test_portions_match_oracle(name, dtype, cuts):
     e, ids, want = setup(name, dtype)
@@ -83,8 +83,9 @@ def test_portions_match_oracle(name, dtype, cuts):
 
 
 @pytest.mark.parametrize("dtype", DTYPES)
-def test_long_prompt_in_engine_portions_and_the_order_of_wanted_places(dtype):
-    e, ids, want = setup("even", dtype)
+@pytest.mark.parametrize("name", ["even", "diff_even"])
+def test_long_prompt_in_engine_portions_and_the_order_of_wanted_places(name, dtype):
+    e, ids, want = setup(name, dtype)
     e.PORTION = 48
     try:
         slot, places = e.open(), [149, 3, 47, 48, 3, 96, 0]
@@ -96,7 +97,7 @@ def test_long_prompt_in_engine_portions_and_the_order_of_wanted_places(dtype):
 
 
 @pytest.mark.parametrize("dtype", DTYPES)
-@pytest.mark.parametrize("name", ["odd", "even"])
+@pytest.mark.parametrize("name", ["odd", "even", "diff_odd", "diff_even"])
 def test_unequal_sequences_decoded_together_match_each_alone(name, dtype):
     import torch
     e, p = S.engine(name, dtype)
@@ -117,18 +118,19 @@ def test_unequal_sequences_decoded_together_match_each_alone(name, dtype):
 
 
 @pytest.mark.parametrize("dtype", DTYPES)
-def test_prompts_in_lockstep_match_each_alone(dtype):
-    e, p = S.engine("even", dtype)
-    a, b = S.tokens("even", 120, 1), S.tokens("even", 120, 2)
+@pytest.mark.parametrize("name", ["even", "diff_even"])
+def test_prompts_in_lockstep_match_each_alone(name, dtype):
+    e, p = S.engine(name, dtype)
+    a, b = S.tokens(name, 120, 1), S.tokens(name, 120, 2)
     slots = [e.open(), e.open()]
     e.feed(slots[1], b[:20])
     got = e.step(slots, [a[:60], b[20:80]], list(range(120)))
-    S.close(got[:60], S.oracle_logits("even", p, a[:60]), dtype)
-    S.close(got[60:], S.oracle_logits("even", p, b[:80])[20:], dtype)
+    S.close(got[:60], S.oracle_logits(name, p, a[:60]), dtype)
+    S.close(got[60:], S.oracle_logits(name, p, b[:80])[20:], dtype)
 
 
 @pytest.mark.parametrize("dtype", DTYPES)
-@pytest.mark.parametrize("name", ["odd", "even"])
+@pytest.mark.parametrize("name", ["odd", "even", "diff_odd", "diff_even"])
 def test_slots_used_again_start_empty(name, dtype):
     e, ids, want = setup(name, dtype)
     run(e, S.tokens(name, 390, 77), [390])
@@ -141,27 +143,30 @@ def test_slots_used_again_start_empty(name, dtype):
     e.close(other)
 
 
-def test_the_same_bits_whatever_else_is_live():
-    e, ids, _ = setup("even", "bfloat16")
+@pytest.mark.parametrize("name", ["even", "diff_even"])
+def test_the_same_bits_whatever_else_is_live(name):
+    e, ids, _ = setup(name, "bfloat16")
     first = run(e, ids, [100] + [1] * 50)
     other = e.open()
-    e.feed(other, S.tokens("even", 217, 5))
+    e.feed(other, S.tokens(name, 217, 5))
     assert (run(e, ids, [100] + [1] * 50) == first).all()
     e.close(other)
 
 
 @pytest.mark.parametrize("dtype", DTYPES)
-def test_long_decode(dtype):
-    e, p = S.engine("even", dtype, slots=1, capacity=700)
-    ids = S.tokens("even", 640, 11)
-    want = S.oracle_logits("even", p, ids)
+@pytest.mark.parametrize("name", ["even", "diff_even"])
+def test_long_decode(name, dtype):
+    e, p = S.engine(name, dtype, slots=1, capacity=700)
+    ids = S.tokens(name, 640, 11)
+    want = S.oracle_logits(name, p, ids)
     S.close(run(e, ids, [20] + [1] * 620), want, dtype)
 
 
-def test_graphs_and_eager_steps_agree():
-    a, _ = S.engine("even", "bfloat16")
-    b, _ = S.engine("even", "bfloat16", graphs=False)
-    ids = S.tokens("even", 80, 3)
+@pytest.mark.parametrize("name", ["even", "diff_even"])
+def test_graphs_and_eager_steps_agree(name):
+    a, _ = S.engine(name, "bfloat16")
+    b, _ = S.engine(name, "bfloat16", graphs=False)
+    ids = S.tokens(name, 80, 3)
     x, y = run(a, ids, [60] + [1] * 20), run(b, ids, [60] + [1] * 20)
     assert a._graphs and not b._graphs
     # the split of the context follows the context class of the graph, so only rounding may differ
@@ -184,8 +189,8 @@ def test_steps_are_checked():
 
 
 def greedy(name, params, prompt, n):
-    from oracle.layer_stack import Decoder
-    d, new = Decoder(S.CONFIGS[name], params), []
+    from oracle.layer_stack import decoder
+    d, new = decoder(S.CONFIGS[name], params), []
     logits = d.feed(prompt)[-1]
     for _ in range(n):
         new.append(int(np.argmax(logits)))
@@ -193,7 +198,7 @@ def greedy(name, params, prompt, n):
     return new
 
 
-@pytest.mark.parametrize("name", ["odd", "even"])
+@pytest.mark.parametrize("name", ["odd", "even", "diff_odd", "diff_even"])
 def test_greedy_generation_through_the_scheduler(name):
     """Five prompts over three slots, in fp32: the token ids of the oracle."""
     from reimagined_b200.generate import generate
@@ -211,23 +216,25 @@ def save_model(folder, name):
     return p
 
 
-def test_generation_from_the_command_line(tmp_path):
-    p = save_model(tmp_path, "even")
+@pytest.mark.parametrize("name", ["even", "diff_even"])
+def test_generation_from_the_command_line(tmp_path, name):
+    p = save_model(tmp_path, name)
     prompts = [[3, 200, 17], [9]]
     r = subprocess.run([sys.executable, "-m", "reimagined_b200.generate", "--model", str(tmp_path), "--dtype", "float32", "--tokens", "5",
                         *sum((["--prompt", ",".join(map(str, ids))] for ids in prompts), [])], cwd=ROOT, capture_output=True, text=True, timeout=300)
     assert r.returncode == 0, r.stderr
     got = [json.loads(x) for x in r.stdout.splitlines() if x.startswith("{")]
-    assert got == [{"prompt": ids, "tokens": greedy("even", p, ids, 5)} for ids in prompts]
+    assert got == [{"prompt": ids, "tokens": greedy(name, p, ids, 5)} for ids in prompts]
 
 
+@pytest.mark.parametrize("name", ["odd", "diff_odd"])
 @pytest.mark.parametrize("dtype", DTYPES)
-def test_trace_replay(tmp_path, dtype):
+def test_trace_replay(tmp_path, name, dtype):
     model, out = tmp_path / "m", tmp_path / "o"
     model.mkdir()
     out.mkdir()
-    p = save_model(model, "odd")
-    a, b = S.tokens("odd", 40, 1), S.tokens("odd", 9, 2)
+    p = save_model(model, name)
+    a, b = S.tokens(name, 40, 1), S.tokens(name, 9, 2)
     steps = [{"step": 0, "entries": [{"id": "a", "tokens": a[:30], "want": [0, 29]}], "end": []},
              {"step": 1, "entries": [{"id": "a", "tokens": a[30:32], "want": []}], "end": []},
              {"step": 2, "entries": [{"id": "a", "tokens": a[32:], "want": [7, 2]}], "end": ["a"]},
@@ -236,7 +243,7 @@ def test_trace_replay(tmp_path, dtype):
                        input="".join(json.dumps(s) + "\n" for s in steps), cwd=str(tmp_path), capture_output=True, text=True, timeout=300)
     assert r.returncode == 0, r.stderr
     assert [x for x in r.stdout.splitlines() if x.startswith("done")] == [f"done {i}" for i in range(4)]
-    la, lb = S.oracle_logits("odd", p, a), S.oracle_logits("odd", p, b)
+    la, lb = S.oracle_logits(name, p, a), S.oracle_logits(name, p, b)
     for step, want in ((0, la[[0, 29]]), (2, la[[39, 34]]), (3, lb[[8]])):
         S.close(np.fromfile(out / f"{step}.f32", "<f4").reshape(len(want), -1), want, dtype)
     assert not (out / "1.f32").exists()

@@ -353,3 +353,247 @@ def test_latent_attention_reports_a_full_cache(cuda, stack_lib):
                                         out.data_ptr(), ws.data_ptr(), size, stream(cuda)) == 0
     assert stack_lib.tbl_device_status(stream(cuda)) == 4
     assert cuda.equal(before, a.cache[1:])
+
+
+# ---- residual streams and Dynamic Tanh ------------------------------------------------------------------------------------------
+@pytest.mark.parametrize("precision", [0, 1])
+@pytest.mark.parametrize("rows,width,streams", [(1, 512, 2), (3, 1000, 1), (40, 90, 3), (2, 4100, 4), (33, 516, 8), (5, 37, 5), (70, 64, 6), (32, 2048, 7)])
+def test_stream_norm(cuda, stack_lib, precision, rows, width, streams):
+    """Update, store, sum, next input and both norms; then rows picked out without a store."""
+    torch, rng = cuda, np.random.default_rng(width)
+    b = Buf(torch)
+    xs, y = rng.standard_normal((streams, rows, width)).astype(np.float32), rng.standard_normal((rows, width)).astype(np.float32)
+    mix, out_w, in_w = rng.standard_normal((streams, streams)), rng.standard_normal(streams), rng.standard_normal(streams)
+    norm, bias, alpha, eps = rng.standard_normal(width), rng.standard_normal(width), 0.7, 0.3
+    index = rng.integers(0, rows, max(1, rows // 2))
+    tol = 4e-3 if precision else 2e-6
+    for kind in (0, 1):
+        for update, store, weights, idx in ((True, 1, in_w, None), (False, 0, in_w, None), (True, 0, None, index), (True, 0, in_w, None)):
+            n = rows if idx is None else len(idx)
+            x = torch.as_tensor(xs).cuda()
+            total = torch.full((n, width), float("nan"), device="cuda")
+            h = torch.zeros((n, width), device="cuda", dtype=torch.bfloat16 if precision else torch.float32)
+            rc = stack_lib.tbl_stream_norm(x.data_ptr(), rows * width, streams, b.f32(y) if update else None, b.f32(mix), b.f32(out_w), store,
+                                           None if weights is None else b.f32(weights), precision, None if idx is None else b.i32(idx), n, width, kind,
+                                           eps, alpha, b.f32(norm), b.f32(bias), total.data_ptr(), h.data_ptr(), stream(torch))
+            assert rc == 0
+            f32 = lambda a: np.float32(a).astype(np.float64)
+            new = O.streams_out(list(xs.astype(np.float64)), f32(mix), f32(out_w), y) if update else list(xs.astype(np.float64))
+            pick = slice(None) if idx is None else idx
+            assert_close(f64(total), sum(new)[pick], 3e-6, "sum")
+            u = O.streams_in(new, np.ones(streams) if weights is None else f32(weights))[pick]
+            want = O.rms_norm(u, f32(norm), eps) if kind == 0 else O.dynamic_tanh(u, np.float32(alpha), f32(norm), f32(bias))
+            assert_close(f64(h), want, tol, "h")
+            for got, a in zip(f64(x), new if store else xs):
+                assert_close(got, a, 3e-6 if store else 0, "streams")
+
+
+@pytest.mark.parametrize("route,precision", [(SIMT, 0), (GEMV, 0), (GEMV, 1), (SIMT, 1), (TENSOR, 1), (ROWS, 1)])
+@pytest.mark.parametrize("m,k,ff", [(9, 512, 70), (1, 64, 32), (3, 40, 37), (150, 72, 100)])
+def test_gated_dense_with_gelu(cuda, stack_lib, route, precision, m, k, ff):
+    from reimagined_b200.stack import StackEngine
+    torch, rng = cuda, np.random.default_rng(ff + 1)
+    if route == GEMV and m > 4:
+        return
+    b = Buf(torch)
+    gate, up = (torch.as_tensor(2.0 * rng.standard_normal((ff, k)) * k ** -0.5, dtype=torch.float32).bfloat16() for _ in range(2))
+    v = b.view(StackEngine._paired(None, gate, up))
+    x = act(torch, rng.standard_normal((m, k)), precision)
+    out = torch.zeros((m, ff), device="cuda", dtype=x.dtype)
+    assert stack_lib.tbl_gated_dense_act_forward(C.byref(v), precision, route, 1, x.data_ptr(), k, m, ff, out.data_ptr(), stream(torch)) == 0
+    want = O.gelu_tanh(O.linear(f64(x), f64(gate))) * O.linear(f64(x), f64(up))
+    assert_close(f64(out), want, 4e-3 if precision else 3e-6)
+
+
+# ---- attention with grouped heads and one or two maps ---------------------------------------------------------------------------
+A_SIMT, A_STREAM, A_FLASH = 1, 2, 3
+
+
+class Attention:
+    """An attention mixer on given projections, its cache, and the same in the oracle."""
+
+    def __init__(self, torch, lib, cfg, precision, slots=3, capacity=420, eps=1e-2, lam=0.6, gated=True, owner=None):
+        from reimagined_b200 import capi
+        self.torch, self.lib, self.cfg, self.precision, self.capacity, self.eps, self.gated = torch, lib, cfg, precision, capacity, eps, gated
+        self.b, self.owner, self.n_slots = Buf(torch), owner, slots
+        H, G, d, vd = (cfg[n] for n in ("heads", "kv_heads", "dim", "vdim"))
+        self.maps = maps = 2 if "diff" in cfg else 1
+        self.sizes = [("q", H * maps * d)] + ([("k", G * maps * d), ("v", G * vd)] if owner is None else []) + ([("g", H * vd)] if gated else [])
+        self.cols = sum(n for _, n in self.sizes)
+        dummy = self.b.view(torch.zeros(1, 8).bfloat16()).weight
+        m = self.m = capi.AttentionMixer()
+        m.in_, m.out = capi.DenseView(dummy, None, 8, self.cols), capi.DenseView(dummy, None, H * vd, 8)
+        m.heads, m.kv_heads, m.dim, m.vdim, m.maps, m.gated, m.kv_from, m.scale = H, G, d, vd, maps, int(gated), -1 if owner is None else 0, cfg["scale"]
+        m.lambda_, m.out_scale = lam, 1.0 - cfg.get("diff", 0.0)
+        # lambda = exp(lq1 . lk1) - exp(lq2 . lk2) + diff
+        self.P = {n: np.eye(d)[0] for n in ("lq1", "lk1", "lk2")}
+        self.P["lq2"] = np.eye(d)[0] * np.log(np.e - lam + cfg.get("diff", 0.0))
+        if "q_temp" in cfg:
+            m.temperature = self.b.f32(O.query_temperature(np.arange(capacity), cfg["q_temp"]["coef"], cfg["q_temp"]["every"]))
+            m.temperature_positions = capacity
+        cw = lib.tbl_attention_cache_width(C.byref(m))
+        dtype = torch.bfloat16 if precision else torch.float32
+        self.cache = torch.zeros((slots, G, capacity, cw), device="cuda", dtype=dtype) if owner is None else owner.cache
+        self.positions = torch.zeros(slots, dtype=torch.int32, device="cuda") if owner is None else owner.positions
+        self.ocache = {} if owner is None else owner.ocache
+
+    def forward(self, route, slots, proj, check_rc=0, advance=True):
+        torch, n_seq = self.torch, len(slots)
+        n = len(proj) // n_seq
+        context = int(self.positions[slots].max()) + n
+        out = torch.zeros((n_seq * n, self.cfg["heads"] * self.cfg["vdim"]), device="cuda", dtype=self.cache.dtype)
+        size = self.lib.tbl_attention_workspace_bytes(C.byref(self.m), self.precision, n_seq, n, context)
+        ws = torch.full((size,), 255, dtype=torch.uint8, device="cuda")          # NaN patterns: nothing unwritten may be used
+        pd = torch.as_tensor(np.asarray(proj, np.float32)).cuda()
+        rc = self.lib.tbl_attention_forward(C.byref(self.m), self.precision, route, self.eps, pd.data_ptr(), self.cache.data_ptr(), self.n_slots,
+                                            self.capacity, self.b.i32(slots), self.positions.data_ptr(), n_seq, n, context, out.data_ptr(),
+                                            ws.data_ptr(), size, stream(torch))
+        assert rc == check_rc
+        if rc == 0 and advance:
+            self.positions[slots] += n
+        return f64(out)
+
+    def oracle(self, slots, proj):
+        """The oracle's mixer reads h; identity projections turn the stacked products into that."""
+        eye, at, P = np.eye(self.cols), 0, dict(self.P)
+        for name, n in self.sizes:
+            P[name], at = eye[at:at + n], at + n
+        P["o"] = np.eye(self.cfg["heads"] * self.cfg["vdim"])
+        n = len(proj) // len(slots)
+        return np.concatenate([O.grouped_attention(np.asarray(proj[i * n:(i + 1) * n], np.float64), P, "", self.cfg, self.eps, self.ocache.setdefault(s, []))
+                               for i, s in enumerate(slots)])
+
+
+def att(*args, diff=True, temp=True):
+    m = dict(S.attention(*args)["mixer"])
+    for name, keep in (("diff", diff), ("q_temp", temp)):
+        if not keep:
+            del m[name]
+    return m
+
+
+ATT = {
+    "odd": att(6, 3, 10, 28, 0.8, 0.3, 0.5, 7),
+    "tiny": att(2, 1, 3, 5, 0.4, 0.0, 0.5, 2),
+    "small": att(4, 2, 48, 80, 0.3, 0.6, 0.4, 32),
+    "group12": att(12, 1, 16, 32, 0.5, 0.2, 0.3, 100),
+    "group20": att(40, 2, 32, 64, 0.3, 0.5, 0.2, 50),
+    "wide": att(2, 1, 128, 256, 0.15, 0.4, 0.5, 40),
+    "values144": att(3, 3, 24, 144, 0.4, 0.5, 0.4, 64),
+    "plain": att(6, 2, 64, 64, 0.2, 0, 0.5, 20, diff=False),
+    "plain_odd": att(5, 1, 20, 36, 0.4, 0, 0, 1, diff=False, temp=False),
+    "plain_wide": att(2, 2, 192, 200, 0.1, 0, 0, 1, diff=False, temp=False),
+    "keys300": att(2, 1, 300, 512, 0.1, 0.3, 0.5, 64),
+}
+A_ROUTES = {A_SIMT: list(ATT), A_STREAM: [s for s in ATT if s != "keys300"], A_FLASH: [s for s in ATT if s != "keys300"]}
+
+
+def rows_close(got, want, tol, what):
+    """Every row by itself: its error against the rows' usual size."""
+    err = np.sqrt(((got - want) ** 2).mean(axis=1)) / np.sqrt((want ** 2).mean())
+    assert np.isfinite(got).all() and err.max() < tol, (what, int(err.argmax()), err.max())
+
+
+@pytest.mark.parametrize("precision,route,size", [(0, A_SIMT, s) for s in ATT] + [(1, r, s) for r in A_ROUTES for s in A_ROUTES[r]] +
+                         [(0, 0, "small"), (1, 0, "small"), (1, 0, "odd"), (1, 0, "keys300"), (1, 0, "plain_wide")])
+def test_attention(cuda, stack_lib, precision, route, size):
+    """A prompt in portions (two tokens among them), then single tokens, on two slots at different places."""
+    # (heads of five values come close to zero as a whole: a larger eps, so that their norm does not blow up the rounding)
+    a = Attention(cuda, stack_lib, ATT[size], precision, gated=size not in ("plain", "tiny"), eps=0.5 if size == "tiny" else 1e-2)
+    rng, tol = np.random.default_rng(5), 3e-2 if precision else 2e-5
+    for slots, n in [([1], 130), ([1], 2), ([2], 61), ([1, 2], 3), ([1, 2], 1), ([2, 1], 1), ([1, 2], 140), ([2], 1)]:
+        proj = rng.standard_normal((len(slots) * n, a.cols)).astype(np.float32)
+        rows_close(a.forward(route, slots, proj), a.oracle(slots, proj), tol, f"slots {slots} n {n}")
+    assert not a.cache[0].any()                   # nobody touched the first slot
+
+
+@pytest.mark.parametrize("precision,route", [(0, A_SIMT), (1, A_SIMT), (1, A_STREAM), (1, A_FLASH)])
+def test_attention_over_another_layers_cache(cuda, stack_lib, precision, route):
+    """The second mixer has queries, scale, temperature and maps' weights of its own, and leaves the cache alone."""
+    first = Attention(cuda, stack_lib, ATT["small"], precision)
+    second = Attention(cuda, stack_lib, {**ATT["small"], "scale": 0.5, "diff": 0.1, "q_temp": {"coef": 0.9, "every": 10}}, precision, lam=-0.4, owner=first)
+    rng, tol = np.random.default_rng(7), 3e-2 if precision else 2e-5
+    for slots, n in [([1], 131), ([2], 2), ([1, 2], 1), ([2, 1], 37)]:
+        proj, own = (rng.standard_normal((len(slots) * n, x.cols)).astype(np.float32) for x in (first, second))
+        rows_close(first.forward(route, slots, proj, advance=False), first.oracle(slots, proj), tol, "first")
+        before = first.cache.clone()
+        rows_close(second.forward(route, slots, own), second.oracle(slots, own), tol, "second")
+        assert cuda.equal(before, first.cache)
+
+
+@pytest.mark.parametrize("route,size", [(A_STREAM, "keys300"), (A_FLASH, "keys300")])
+def test_attention_routes_refuse_sizes_they_do_not_take(cuda, stack_lib, route, size):
+    a = Attention(cuda, stack_lib, ATT[size], 1)
+    a.forward(route, [0], np.zeros((2, a.cols)), check_rc=-2)
+    a = Attention(cuda, stack_lib, ATT["small"], 0)
+    a.forward(route, [0], np.zeros((2, a.cols)), check_rc=-2)
+
+
+@pytest.mark.parametrize("precision,route,size", [(0, A_SIMT, "odd")] + [(1, r, s) for r in (A_SIMT, A_STREAM, A_FLASH)
+                                                                         for s in ("odd", "small", "group12", "wide", "plain")])
+@pytest.mark.parametrize("aimed", [0, 1])
+def test_attention_finds_one_key(cuda, stack_lib, precision, route, size, aimed):
+    """One map's queries aim at a single cached token: the first ones, both sides of tile and block borders, the latest,
+    itself.  The other map spreads out.  A key that is missing or off by one replaces the output."""
+    cfg = {**ATT[size], "q_temp": {"coef": 0.1, "every": 50}}
+    maps = 2 if "diff" in cfg else 1
+    if aimed >= maps:
+        return
+    a = Attention(cuda, stack_lib, cfg, precision, lam=1.5)
+    rng, n = np.random.default_rng(6), 400
+    H, G, d, vd = (cfg[k] for k in ("heads", "kv_heads", "dim", "vdim"))
+    proj = rng.standard_normal((n, a.cols)).astype(np.float32)
+    borders = [0, 1, 2, 15, 16, 31, 32, 63, 64, 65, 126, 127, 128, 129, 191, 192, 255, 256, 257, 383, 384]
+    target = np.array([borders[t % len(borders)] if borders[t % len(borders)] <= t else t for t in range(n)])
+    target[::7] = np.arange(n)[::7]                # itself
+    target[3::11] = np.maximum(np.arange(n)[3::11] - 1, 0)
+    q = proj[:, :H * maps * d].reshape(n, H, maps, d)
+    k = proj[:, H * maps * d:(H + G) * maps * d].reshape(n, G, maps, d)
+    k /= np.sqrt((k ** 2).sum(-1, keepdims=True))
+    aim = 45.0 / cfg["scale"]                      # the target's score; the others follow from the angle to it
+    for h in range(H):
+        q[:, h] *= 0.1
+        q[:, h, aimed] = aim * k[target, h // (H // G), aimed]
+    cuts = [300, 60, 1, 2, 37] if route != A_STREAM else [300] + [1] * 40 + [2, 58]
+    got, at = [], 0
+    for c in cuts:
+        got.append(a.forward(route, [0], proj[at:at + c]))
+        at += c
+    got, want = np.concatenate(got), a.oracle([0], proj)
+    if maps == 1:                                  # the construction works
+        v = np.array([e[1] for e in a.ocache[0]])[target].repeat(H // G, axis=1).reshape(n, -1)
+        gate = O.sigmoid(proj[:, -H * vd:])
+        assert np.median(np.abs(want - v * gate).max(axis=1) / np.abs(v).max(axis=1)) < 0.2
+    rows_close(got, want, 6e-2 if precision else 1e-4, "aimed")
+
+
+def test_attention_does_not_depend_on_what_else_is_in_the_batch_or_on_slots(cuda, stack_lib):
+    """The same rows alone, and in other slots beside longer sequences, prompt and decode."""
+    rng = np.random.default_rng(8)
+    for n, route in ((100, A_FLASH), (1, A_STREAM), (5, A_STREAM)):
+        a, b = (Attention(cuda, stack_lib, ATT["small"], 1) for _ in range(2))
+        history, other = rng.standard_normal((150, a.cols)), rng.standard_normal((260, a.cols))
+        a.forward(A_FLASH, [0], history)
+        b.forward(A_FLASH, [1], other)
+        b.forward(A_FLASH, [2], history)
+        x, y = rng.standard_normal((n, a.cols)), rng.standard_normal((n, a.cols))
+        alone, beside = a.forward(route, [0], x), b.forward(route, [1, 2], np.concatenate([y, x]))[n:]
+        # the split of the cache may differ: rounding only
+        assert np.abs(alone - beside).max() <= (0 if route == A_FLASH else 1e-2) * np.abs(alone).max() + 1e-6
+
+
+def test_attention_reports_a_full_cache(cuda, stack_lib):
+    a = Attention(cuda, stack_lib, ATT["small"], 1, capacity=16)
+    stack_lib.tbl_device_status(stream(cuda))
+    a.forward(0, [0], np.zeros((10, a.cols)))
+    assert stack_lib.tbl_device_status(stream(cuda)) == 0
+    for n, pos in ((2, 15), (1, 16)):               # the step's context claims less than the device holds
+        a.positions[0] = pos
+        size = stack_lib.tbl_attention_workspace_bytes(C.byref(a.m), 1, 1, n, 16)
+        ws, pd = cuda.empty(size, dtype=cuda.uint8, device="cuda"), cuda.ones((n, a.cols), device="cuda")
+        out = cuda.zeros((n, 4 * 80), device="cuda", dtype=cuda.bfloat16)
+        before = a.cache[1:].clone()
+        assert stack_lib.tbl_attention_forward(C.byref(a.m), 1, 0, 1e-4, pd.data_ptr(), a.cache.data_ptr(), 3, 16, a.b.i32([0]), a.positions.data_ptr(), 1,
+                                               n, 16, out.data_ptr(), ws.data_ptr(), size, stream(cuda)) == 0
+        assert stack_lib.tbl_device_status(stream(cuda)) == 4
+        assert cuda.equal(before, a.cache[1:])

@@ -14,12 +14,12 @@ from oracle import layer_stack as O
 ROOT = os.path.dirname(os.path.dirname(os.path.abspath(__file__)))
 
 
-@pytest.mark.parametrize("name", ["odd", "only_delta", "only_latent"])
+@pytest.mark.parametrize("name", ["odd", "only_delta", "only_latent", "diff_odd", "diff_wide"])
 def test_oracle_does_not_depend_on_the_cut(name):
     _, p = S.weights(name)
     ids = S.tokens(name, 23)
-    whole = O.Decoder(S.CONFIGS[name], p).feed(ids)
-    d = O.Decoder(S.CONFIGS[name], p)
+    whole = O.decoder(S.CONFIGS[name], p).feed(ids)
+    d = O.decoder(S.CONFIGS[name], p)
     parts, at = [], 0
     for n in (1, 2, 7, 1, 12):
         parts.append(d.feed(ids[at:at + n]))
@@ -45,6 +45,35 @@ def test_oracle_rotation_pairs_and_angle():
     np.testing.assert_allclose(y[0, 1], 2 * np.cos(a) - 5 * np.sin(a))
     np.testing.assert_allclose(y[0, 4], 5 * np.cos(a) + 2 * np.sin(a))
     np.testing.assert_allclose(y[0, 6:], x[0, 6:])
+
+
+def test_oracle_streams_and_norm_by_hand():
+    xs, y = [np.array([[1.0, 2.0]]), np.array([[-3.0, 0.5]])], np.array([[10.0, 20.0]])
+    np.testing.assert_allclose(O.streams_in(xs, [2.0, 3.0]), [[-7.0, 5.5]])
+    got = O.streams_out(xs, [[1.0, 0.5], [0.25, 2.0]], [0.1, 0.2], y)              # mix[from][to]
+    np.testing.assert_allclose(got[0], [[1.0 - 0.75 + 1.0, 2.0 + 0.125 + 2.0]])
+    np.testing.assert_allclose(got[1], [[0.5 - 6.0 + 2.0, 1.0 + 1.0 + 4.0]])
+    np.testing.assert_allclose(O.dynamic_tanh([2.0], 0.25, [3.0], [1.0]), [3 * np.tanh(0.5) + 1])
+    np.testing.assert_allclose(O.gelu_tanh([1.0, -2.0]), [0.841192, -0.045402], atol=1e-6)
+
+
+def test_oracle_query_temperature_steps():
+    assert [round(float(O.query_temperature(p, 2.0, 4)), 6) for p in (0, 2, 3, 6, 7)] == [
+        1.0, 1.0, round(1 + 2 * np.log(2), 6), round(1 + 2 * np.log(2), 6), round(1 + 2 * np.log(3), 6)]
+
+
+def test_oracle_differential_attention_by_hand():
+    """One head, one-dimensional keys, two tokens."""
+    cfg = {"heads": 1, "kv_heads": 1, "dim": 1, "vdim": 2, "scale": 0.5, "diff": 0.25, "q_temp": {"coef": 1.0, "every": 2}}
+    P = {"q": [[1.0], [2.0]], "q.b": [0.0, 0.5], "k": [[1.0], [-1.0]], "k.b": [0.25, 0.0], "v": [[1.0], [0.0]], "v.b": [0.0, 3.0],
+         "lq1": [0.5], "lk1": [1.0], "lq2": [0.0], "lk2": [1.0], "g": np.zeros((2, 1)), "o": np.eye(2), "o.b": [0.0, 1.0]}
+    h = np.array([[1.0], [2.0]])
+    t = 1 + np.log(2)                                                               # the second token: (1 + 1) / 2 = 1
+    s1, s2 = 0.5 * t * 2.0 * np.array([1.25, 2.25]), 0.5 * t * 4.5 * np.array([-1.0, -2.0])
+    a1, a2 = (np.exp(s) / np.exp(s).sum() @ np.array([[1.0, 3.0], [2.0, 3.0]]) for s in (s1, s2))
+    o = a1 - (np.exp(0.5) - 1 + 0.25) * a2
+    o = o / np.sqrt((o ** 2).mean() + 1e-3) * 0.75
+    np.testing.assert_allclose(O.grouped_attention(h, P, "", cfg, 1e-3, [])[1], 0.5 * o + [0.0, 1.0])
 
 
 def test_safetensors_round_trip_at_any_offset(tmp_path):
@@ -87,11 +116,38 @@ def test_weights_must_fit_the_configuration():
             check_weights(cfg, w)
 
 
+def test_weights_of_layers_that_share_a_cache():
+    from reimagined_b200.stack import check_weights
+    w, _ = S.weights("diff_odd")
+    assert "l0.mix.k.b" in w and "l1.mix.k" not in w and "l1.mix.v.b" not in w and "l1.hc2.mix" not in w and "l3.hc1.mix" in w
+    check_weights(S.DIFF_ODD, w)
+    # tensors around a feed-forward that is not there may be in the file
+    check_weights(S.DIFF_ODD, {**w, "l1.norm2": w["l0.norm2"], "l1.hc2.in": w["l0.hc2.in"]})
+    for name, value in (("l1.mix.k", w["l0.mix.k"]), ("l0.dwa", torch.ones(2)), ("l0.mlp.gate.b", torch.zeros(50)), ("l0.hc1.mix", torch.zeros(3, 2)),
+                        ("l2.norm1.alpha", torch.zeros(1)), ("final.norm.b", None)):
+        d = {**w, name: value}
+        if value is None:
+            del d[name]
+        with pytest.raises(ValueError):
+            check_weights(S.DIFF_ODD, d)
+
+
+def test_query_temperature_table():
+    from reimagined_b200.stack import StackEngine
+
+    class Stub:
+        capacity, _temperatures, f32 = 300, {}, staticmethod(lambda t: t.numpy())
+    for coef, every in ((0.7, 7), (1.5, 1), (0.3, 64), (0.4, 2.5)):
+        np.testing.assert_allclose(StackEngine.query_temperature(Stub, coef, every), O.query_temperature(np.arange(300), coef, every))
+
+
 def test_registry_knows_its_models(tmp_path):
     from reimagined_b200 import registry
     (tmp_path / "config.json").write_text(json.dumps(S.ODD))
     e, cfg = registry.entry(str(tmp_path))
     assert e.library == "stack" and "float32" in e.dtypes and cfg == S.ODD
+    (tmp_path / "config.json").write_text(json.dumps(S.DIFF_ODD))
+    assert registry.entry(str(tmp_path))[0].dtypes == ("bfloat16", "float32")
     (tmp_path / "config.json").write_text(json.dumps({"architecture": "Nonesuch"}))
     with pytest.raises(ValueError):
         registry.entry(str(tmp_path))
@@ -198,3 +254,60 @@ def test_entry_points_refuse_before_they_touch_a_device(stack_lib):
     assert L.tbl_gated_dense_forward(C.byref(v), 1, 0, 4096, 64, 1, 8, 4096, None) == -2
     v.weight = 4100
     assert L.tbl_dense_forward(C.byref(v), 1, 0, 4096, 64, 1, None, 4096, None) == -6
+
+
+def test_models_with_streams_are_checked(stack_lib):
+    import ctypes as C
+    from reimagined_b200 import capi
+    L = stack_lib
+
+    def layer(kv_from=-1, heads=4, kv_heads=2, dim=16, vdim=24):
+        a, l = capi.AttentionMixer(), capi.StackLayer()
+        kv = kv_heads * (2 * dim + vdim) if kv_from < 0 else 0
+        a.in_, a.out = capi.DenseView(4096, 4096, 64, heads * (2 * dim + vdim) + kv), capi.DenseView(4096, 4096, heads * vdim, 64)
+        a.heads, a.kv_heads, a.dim, a.vdim, a.maps, a.gated, a.kv_from, a.scale, a.out_scale = heads, kv_heads, dim, vdim, 2, 1, kv_from, 0.1, 0.5
+        l.mixer, l.norm1, l.attention, l.tanh1, l.hyper1 = capi.MIXER_ATTENTION, 4096, a, capi.TanhNorm(4096, 0.5), capi.Hyper(4096, 4096, 4096)
+        return l
+
+    def state_bytes(layers, precision=capi.BF16, norm=capi.NORM_DYNAMIC_TANH, streams=2):
+        arr = (capi.StackLayer * len(layers))(*layers)
+        m = capi.StackModel(64, 100, len(layers), 4096, 1.0, 1e-5, arr, 4096, capi.DenseView(4096, None, 64, 100), norm, capi.TanhNorm(4096, 0.5), streams)
+        return L.tbl_stack_state_bytes(C.byref(m), precision, 3, 50)
+
+    one = state_bytes([layer()])
+    # a token's row: two keys of 16 and values of 24, padded to 32, for every key/value head
+    assert one == 256 + -(-3 * 50 * 2 * 64 * 2 // 256) * 256
+    assert state_bytes([layer(), layer(0)]) == one                        # no cache of its own
+    assert state_bytes([layer(), layer(0), layer()]) == 2 * one - 256
+    assert state_bytes([layer()], capi.F32) == 2 * one - 256
+    assert state_bytes([layer()], streams=8) and not state_bytes([layer()], streams=9) and not state_bytes([layer()], norm=5)
+    assert not state_bytes([layer(0)])                                    # itself
+    assert not state_bytes([layer(1), layer()])                           # a later layer
+    assert not state_bytes([layer(), layer(0), layer(1)])                 # a layer that shares
+    assert not state_bytes([layer(), layer(0, kv_heads=4)]) and not state_bytes([layer(), layer(0, vdim=16)])
+    assert not state_bytes([layer(heads=5)]) and not state_bytes([layer(dim=600)])
+    bare = layer()
+    bare.hyper1.mix = None
+    assert not state_bytes([bare])
+    averaged = layer()
+    averaged.depth_weights = 4096
+    assert not state_bytes([averaged])
+
+
+def test_attention_entry_points_refuse_before_they_touch_a_device(stack_lib):
+    import ctypes as C
+    from reimagined_b200 import capi
+    L, a = stack_lib, capi.AttentionMixer()
+    a.in_, a.out = capi.DenseView(4096, None, 8, 4 * 32 + 2 * 56), capi.DenseView(4096, None, 4 * 24, 8)
+    a.heads, a.kv_heads, a.dim, a.vdim, a.maps, a.kv_from, a.scale, a.out_scale = 4, 2, 16, 24, 2, -1, 0.1, 1.0
+    assert L.tbl_attention_cache_width(C.byref(a)) == 64
+    run = lambda **k: L.tbl_attention_forward(C.byref(a), k.get("precision", 1), k.get("route", 0), 1e-5, 4096, k.get("cache", 4096), k.get("slots", 2), 16, 4096,
+                                              4096, k.get("n_seq", 1), k.get("n_tok", 1), k.get("context", 16), 4096, k.get("ws", 4096), k.get("bytes", 1 << 40), None)
+    assert run(precision=3) == -1 and run(context=17) == -1 and run(n_tok=9, context=8) == -1 and run(cache=None) == -1 and run(n_seq=3) == -1
+    assert run(bytes=0) == -7 and run(ws=4096 + 16) == -6 and run(cache=4096 + 8) == -6
+    a.kv_heads = 3
+    assert run() == -2 and L.tbl_attention_cache_width(C.byref(a)) == 0
+    norm = lambda **k: L.tbl_stream_norm(4096, k.get("stride", 64), k.get("streams", 2), k.get("y", 4096), 4096, k.get("out", 4096), k.get("store", 0), 4096, 1,
+                                         k.get("index"), 1, 64, k.get("kind", 1), 1e-5, 0.5, 4096, k.get("bias", 4096), None, 4096, None)
+    assert norm(streams=0) == -1 and norm(streams=9) == -10 and norm(out=None) == -1 and norm(kind=2) == -1 and norm(bias=None) == -1
+    assert norm(index=4096, store=1) == -1 and norm(stride=66) == -6 and norm(y=4100) == -6
