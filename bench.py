@@ -684,8 +684,13 @@ def run_ours(args):
         dist.destroy_process_group()
 
 
-def run_guselix(args):
-    """One JSON line: tokens/s of Guselix (prefill, decode) and of the hybrid at equal width and depth, one GPU."""
+STACK_MODELS = {"guselix": "Guselix, every 4th layer latent attention, random weights; weights exceed L2",
+                "goguvik": "Goguvik, every other layer over an earlier layer's cache, two residual streams, random weights; weights exceed L2"}
+
+
+def run_stack(args):
+    """One JSON line: tokens/s of a layer-stack model (prefill, decode), one GPU, and at equal width and depth of the model
+    that was there before it: the hybrid beside Guselix, Guselix beside Goguvik."""
     import torch
     from reimagined_b200 import build as tbl_build, stack_shapes
     if int(os.environ.get("RANK", "0")) != 0:
@@ -699,13 +704,15 @@ def run_guselix(args):
     sampler.start()
     records = []
     for width, layers in ((2048, 8), (4096, 4)):
-        records += stack_shapes.time_guselix(width, layers, iters=args.steps)
-        records += stack_shapes.time_hybrid(width, layers, iters=args.steps)
-    best = max(r["tokens_per_s"] for r in records if r["model"] == "Guselix" and r["phase"] == "decode")
-    print(json.dumps({"metric": "guselix_decode_tokens_per_s", "value": best, "unit": "tokens/s", "n_gpus": 1, "steps": args.steps,
+        records += stack_shapes.time_stack(args.model, width, layers, iters=args.steps)
+        if args.model == "guselix":
+            records += stack_shapes.time_hybrid(width, layers, iters=args.steps)
+        else:
+            records += stack_shapes.time_stack("guselix", width, layers, iters=args.steps)
+    best = max(r["tokens_per_s"] for r in records if r["model"].lower() == args.model and r["phase"] == "decode")
+    print(json.dumps({"metric": f"{args.model}_decode_tokens_per_s", "value": best, "unit": "tokens/s", "n_gpus": 1, "steps": args.steps,
                       "higher_is_better": True, "vs_baseline": None, "dtype": "bf16", "data": "synthetic", "clocks": sampler.stop(),
-                      "config": {"model": "Guselix, every 4th layer latent attention, random weights; weights exceed L2"},
-                      "records": records}))
+                      "config": {"model": STACK_MODELS[args.model]}, "records": records}))
 
 
 def main():
@@ -716,12 +723,12 @@ def main():
     ap.add_argument("--impl", default="ours", choices=["ours", "reference"])
     ap.add_argument("--headline-only", action="store_true",
                     help="skip the gemm / decode / colsplit sections (used for profiler captures of the headline kernel)")
-    ap.add_argument("--model", default="ternary", choices=["ternary", "guselix"],
-                    help="guselix: prefill and decode of the layer-stack model at real layer sizes (random weights) beside the "
-                         "hybrid of the same width and depth, instead of the headline")
+    ap.add_argument("--model", default="ternary", choices=["ternary", *STACK_MODELS],
+                    help="guselix, goguvik: prefill and decode of a layer-stack model at real layer sizes (random weights) beside "
+                         "an older model of the same width and depth, instead of the headline")
     args = ap.parse_args()
-    if args.model == "guselix":
-        run_guselix(args)
+    if args.model in STACK_MODELS:
+        run_stack(args)
     elif args.impl == "reference":
         run_reference(args)
     else:

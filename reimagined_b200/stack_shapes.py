@@ -1,6 +1,6 @@
 """Time the layer-stack operators and models, each beside the like operator of the ternary hybrid at the same size.
 
-    python -m reimagined_b200.stack_shapes --width 4096 [--only dense,delta,latent,norm,model]
+    python -m reimagined_b200.stack_shapes --width 4096 [--only dense,delta,latent,attention,norm,model] [--model guselix,goguvik]
 
 One JSON line per record.  Every operator runs from a CUDA graph over several copies of its weights, states or caches, so
 that a call never finds them in L2.  `roofline` is the share of min(bytes / copy bandwidth, FLOPs / bf16 GEMM rate) that
@@ -85,14 +85,14 @@ def dense(m: int, k: int, n: int, residual: bool = False) -> dict:
                   rows=m, k=k, n=n)
 
 
-def gated(m: int, k: int, ff: int) -> dict:
+def gated(m: int, k: int, ff: int, activation: int = capi.ACT_SILU) -> dict:
     L = capi.stack_lib()
     ws = [bf16(2 * ff, k) for _ in range(copies(4.0 * ff * k))]
     x, out, bias = bf16(m, k, scale=1.0), torch.empty(m, ff, device="cuda", dtype=torch.bfloat16), torch.zeros(2 * ff, device="cuda")
     views = [capi.DenseView(w.data_ptr(), bias.data_ptr(), k, 2 * ff) for w in ws]
-    us = time_calls([lambda v=v: check(L.tbl_gated_dense_forward(C.byref(v), capi.BF16, 0, x.data_ptr(), k, m, ff, out.data_ptr(), stream()),
-                                       "tbl_gated_dense_forward") for v in views])
-    return record("gated dense", us, 2.0 * (2 * ff * k + m * k + m * ff), 4.0 * m * ff * k, rows=m, k=k, n=ff)
+    us = time_calls([lambda v=v: check(L.tbl_gated_dense_act_forward(C.byref(v), capi.BF16, 0, activation, x.data_ptr(), k, m, ff, out.data_ptr(), stream()),
+                                       "tbl_gated_dense_act_forward") for v in views])
+    return record("gated dense, gelu" if activation == capi.ACT_GELU_TANH else "gated dense", us, 2.0 * (2 * ff * k + m * k + m * ff), 4.0 * m * ff * k, rows=m, k=k, n=ff)
 
 
 def ternary(m: int, k: int, n: int) -> dict:
@@ -190,6 +190,33 @@ def latent(n_seq: int, n_tok: int, context: int, heads: int, dim: int = 128, rot
     return record("latent attention", us, cache + weights + 4.0 * rows * cols, flops, sequences=n_seq, tokens=n_tok, context=context, heads=heads)
 
 
+def differential(n_seq: int, n_tok: int, context: int, heads: int, kv_heads: int, dim: int = 64, vdim: int = 128, maps: int = 2) -> dict:
+    """The whole mixer between its stacked projection and W_o: cache append, attention, combination of the maps, head norm, gate."""
+    L, rows = capi.stack_lib(), n_seq * n_tok
+    cols = heads * (maps * dim + vdim) + kv_heads * (maps * dim + vdim)
+    some, zeros = bf16(1, 8), torch.zeros(cols, device="cuda")
+    m = capi.AttentionMixer()
+    m.in_, m.out = capi.DenseView(some.data_ptr(), zeros.data_ptr(), 8, cols), capi.DenseView(some.data_ptr(), None, heads * vdim, 8)
+    table = torch.ones(context, device="cuda")
+    m.temperature, m.temperature_positions, m.heads, m.kv_heads, m.dim, m.vdim, m.maps, m.gated = table.data_ptr(), context, heads, kv_heads, dim, vdim, maps, 1
+    m.kv_from, m.scale, m.lambda_, m.out_scale = -1, dim ** -0.5, 0.5, 0.5
+    per_token = kv_heads * L.tbl_attention_cache_width(C.byref(m))
+    cache = 2.0 * n_seq * context * per_token
+    caches = [bf16(n_seq, context * per_token, scale=1.0) for _ in range(copies(cache, 16) if n_tok == 1 else 1)]
+    pos = torch.full((n_seq,), context - n_tok, dtype=torch.int32, device="cuda")
+    slots = torch.arange(n_seq, dtype=torch.int32, device="cuda")
+    proj, out = torch.randn(rows, cols, device="cuda"), torch.empty(rows, heads * vdim, device="cuda", dtype=torch.bfloat16)
+    size = L.tbl_attention_workspace_bytes(C.byref(m), capi.BF16, n_seq, n_tok, context)
+    ws = torch.empty(size, dtype=torch.uint8, device="cuda")
+    us = time_calls([lambda c=c: check(L.tbl_attention_forward(C.byref(m), capi.BF16, 0, 1e-6, proj.data_ptr(), c.data_ptr(), n_seq, context, slots.data_ptr(),
+                                                               pos.data_ptr(), n_seq, n_tok, context, out.data_ptr(), ws.data_ptr(), size, stream()),
+                                       "tbl_attention_forward") for c in caches], 16 if n_tok <= 8 else 4)
+    pairs = n_seq * sum(range(context - n_tok + 1, context + 1))
+    name = "differential attention" if maps == 2 else "attention"
+    return record(name, us, cache + 4.0 * rows * cols + 2.0 * rows * heads * vdim, 2.0 * heads * maps * pairs * (dim + vdim), sequences=n_seq, tokens=n_tok,
+                  context=context, heads=heads, kv_heads=kv_heads)
+
+
 def attention(n_seq: int, context: int, heads: int, dim: int) -> dict:
     """The hybrid's attention for one token (its kernel's shared memory bounds the context)."""
     L, kv = capi.lib(), heads * dim
@@ -215,6 +242,19 @@ def depth(rows: int, width: int, count: int) -> dict:
     return record("depth average + norm", us, rows * width * (4.0 * count + 6), rows=rows, width=width, arrays=count)
 
 
+def streams(rows: int, width: int, count: int) -> dict:
+    """A boundary between sublayers: the streams updated in place, the next input, Dynamic Tanh."""
+    L = capi.stack_lib()
+    xs = [torch.randn(count, rows, width, device="cuda") for _ in range(copies(4.0 * count * rows * width, 8))]
+    y, norm = torch.randn(rows, width, device="cuda"), torch.ones(width, device="cuda")
+    mix, w = torch.eye(count, device="cuda"), torch.ones(count, device="cuda")
+    out = torch.empty(rows, width, device="cuda", dtype=torch.bfloat16)
+    us = time_calls([lambda a=a: check(L.tbl_stream_norm(a.data_ptr(), rows * width, count, y.data_ptr(), mix.data_ptr(), w.data_ptr(), 1, w.data_ptr(),
+                                                         capi.BF16, None, rows, width, capi.NORM_DYNAMIC_TANH, 1e-6, 0.5, norm.data_ptr(), norm.data_ptr(),
+                                                         None, out.data_ptr(), stream()), "tbl_stream_norm") for a in xs])
+    return record("stream update + norm", us, rows * width * (8.0 * count + 6), rows=rows, width=width, streams=count)
+
+
 def row_norm(rows: int, width: int) -> dict:
     L = capi.lib()
     xs = [torch.randn(rows, width, device="cuda") for _ in range(copies(4.0 * rows * width, 8))]
@@ -236,16 +276,32 @@ def guselix_config(width: int, layers: int, vocab: int = 32000) -> dict:
             "layers": [att if i % 4 == 3 else mix for i in range(layers)]}
 
 
-def time_guselix(width: int, layers: int, batches=(1, 8, 64), context: int = 512, prompts=(512, 8192), iters: int = 50) -> List[dict]:
+def goguvik_config(width: int, layers: int, vocab: int = 32000) -> dict:
+    """Sizes like a real model's: heads of two maps of 64 over values of 128, four query heads to a key/value head, every
+    other layer over the cache of the one before it; random weights."""
+    heads = width // 128
+    out = []
+    for i in range(layers):
+        m = {"heads": heads, "kv_heads": max(1, heads // 4), "dim": 64, "vdim": 128, "scale": 0.125, "diff": 0.4, "q_temp": {"coef": 0.1, "every": 8192}}
+        if i % 2:
+            m["kv_from"] = i - 1
+        out.append({"type": "attention", "mixer": m, "mlp": {"kind": "dense", "ff": 3 * width}})
+    return {"architecture": "Goguvik", "layers": out, "norm": {"eps": 1e-6}, "streams": 2, "vocab": vocab, "width": width}
+
+
+CONFIGS = {"guselix": guselix_config, "goguvik": goguvik_config}
+
+
+def time_stack(name: str, width: int, layers: int, batches=(1, 8, 64), context: int = 512, prompts=(512, 8192), iters: int = 50) -> List[dict]:
     from .stack import StackEngine, synthetic_weights
-    cfg = guselix_config(width, layers)
+    cfg = CONFIGS[name](width, layers)
     weights = synthetic_weights(cfg, 1, rank=width // 32, device="cuda")
     params, out = sum(w.numel() for w in weights.values()), []
     for batch, prompt in [(b, 0) for b in batches] + [(1, p) for p in prompts]:
         eng = StackEngine(cfg, weights, slots=batch, capacity=max(prompt, context + iters + 8))
         slots = [eng.open() for _ in range(batch)]
         a, b = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
-        rec = {"model": "Guselix", "width": width, "layers": layers, "parameters": params}
+        rec = {"model": cfg["architecture"], "width": width, "layers": layers, "parameters": params}
         if prompt:
             ids, times = torch.randint(0, cfg["vocab"], (prompt,)).tolist(), []
             for _ in range(4):
@@ -297,7 +353,7 @@ def time_hybrid(width: int, layers: int, batches=(1, 8, 64), context: int = 512,
     return out
 
 
-def operators(width: int, only=("dense", "delta", "latent", "norm")):
+def operators(width: int, only=("dense", "delta", "latent", "attention", "norm")):
     """Generator of records at one model width."""
     heads, ff = width // 128, 3 * width
     if "dense" in only:
@@ -307,6 +363,7 @@ def operators(width: int, only=("dense", "delta", "latent", "norm")):
             yield dense(m, width, width, residual=True)
             yield ternary(m, width, width)
             yield gated(m, width, ff)
+            yield gated(m, width, ff, capi.ACT_GELU_TANH)
             yield dense(m, ff, width, residual=True)
             yield ternary(m, ff, width)
     if "delta" in only:
@@ -322,8 +379,17 @@ def operators(width: int, only=("dense", "delta", "latent", "norm")):
                 yield attention(n_seq, context, heads, 128)
         for n_tok in (512, 2048, 8192):
             yield latent(1, n_tok, n_tok, heads, q_rank=3 * width // 8)
+    if "attention" in only:
+        for n_seq, context in ((1, 1024), (1, 8192), (8, 8192), (64, 4096)):
+            yield differential(n_seq, 1, context, heads, max(1, heads // 4))
+            if n_seq <= 8 and "latent" not in only:
+                yield attention(n_seq, context, heads, 128)
+        for n_tok in (512, 2048, 8192):
+            yield differential(1, n_tok, n_tok, heads, max(1, heads // 4))
     if "norm" in only:
         for rows in (1, 64, 8192):
+            yield streams(rows, width, 2)
+            yield streams(rows, width, 4)
             yield depth(rows, width, 9)
             yield row_norm(rows, width)
 
@@ -332,14 +398,18 @@ def main() -> None:
     ap = argparse.ArgumentParser(description=__doc__, formatter_class=argparse.RawDescriptionHelpFormatter)
     ap.add_argument("--width", type=int, default=4096)
     ap.add_argument("--layers", type=int, default=4, help="layers of the whole-model timings")
-    ap.add_argument("--only", default="dense,delta,latent,norm,model")
+    ap.add_argument("--only", default="dense,delta,latent,attention,norm,model")
+    ap.add_argument("--model", default="guselix,goguvik", help="layer-stack models of the whole-model timings")
     args = ap.parse_args()
     use_measured_peaks()
     only = args.only.split(",")
     for r in operators(args.width, only):
         print(json.dumps(r), flush=True)
     if "model" in only:
-        for r in time_guselix(args.width, args.layers) + time_hybrid(args.width, args.layers):
+        for name in args.model.split(","):
+            for r in time_stack(name, args.width, args.layers):
+                print(json.dumps(r), flush=True)
+        for r in time_hybrid(args.width, args.layers):
             print(json.dumps(r), flush=True)
 
 
