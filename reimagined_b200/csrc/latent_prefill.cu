@@ -87,7 +87,7 @@ latent_prefill_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_co
              *s_full = v_empty + kMaxRing, *p_full = s_full + 2, *o_full = p_full + 2;
     uint32_t* tmem_slot = reinterpret_cast<uint32_t*>(o_full + 2);
 
-    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+    const int warp = uniform_warp(), lane = threadIdx.x & 31;
     if (threadIdx.x == 0) {
         mbar_init(q_full, 1);
         for (int s = 0; s < kMaxRing; ++s) { mbar_init(&k_full[s], 1); mbar_init(&k_empty[s], 1); mbar_init(&v_full[s], 1); mbar_init(&v_empty[s], 1); }
@@ -110,19 +110,18 @@ latent_prefill_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_co
     const int tile = p.tiles - 1 - blockIdx.x, head = blockIdx.y, seq = blockIdx.z;
     const int q0 = tile * 2 * kBlock;                          // first query of the CTA within its sequence's portion
     const int pos0 = p.positions[p.slots[seq]] + q0;           // and its position
-    int nblk[2];                                               // blocks each tile sees
-#pragma unroll
-    for (int w = 0; w < 2; ++w) {
+    auto blocks_of = [&](int w) {                              // blocks a tile sees
         const int rows = min(kBlock, p.n_tok - q0 - w * kBlock);
-        nblk[w] = rows > 0 ? min(pos0 + w * kBlock + rows - 1, p.ctx - 1) / kBlock + 1 : 0;
-    }
-    const int nmax = max(nblk[0], nblk[1]);
+        return rows > 0 ? min(pos0 + w * kBlock + rows - 1, p.ctx - 1) / kBlock + 1 : 0;
+    };
+    const int nblk0 = blocks_of(0), nblk1 = blocks_of(1);
+    const int nmax = max(nblk0, nblk1);
     const int row_q = seq * p.n_tok + q0, row_k = seq * p.ctx;
 
     if (warp == kTmaWarp) {
         // ---------------- TMA ----------------
-        if (lane == 0) {
-            const int tiles_q = nblk[1] > 0 ? 2 : 1, n = p.d + p.rd;
+        if (elect_one()) {
+            const int tiles_q = nblk1 > 0 ? 2 : 1, n = p.d + p.rd;
             mbar_arrive_expect_tx(q_full, tiles_q * q_bytes);
             for (int w = 0; w < tiles_q; ++w) {
                 for (int s = 0; s < sub_d; ++s)
@@ -152,7 +151,7 @@ latent_prefill_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_co
         }
     } else if (warp == kMmaWarp) {
         // ---------------- MMA ----------------
-        if (lane == 0) {
+        if (elect_one()) {
             const uint32_t is = idesc_bf16(kBlock), iv = idesc_bf16(p.vd);
             bool alive = mbar_wait_bounded(q_full, 0, p.status);
             tc_fence_after();
@@ -167,7 +166,7 @@ latent_prefill_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_co
             for (int j = -1; alive && j < nmax; ++j) {
 #pragma unroll
                 for (int w = 0; w < 2; ++w) {
-                    if (j >= 0 && j < nblk[w]) {
+                    if (j >= 0 && j < (w ? nblk1 : nblk0)) {
                         alive = mbar_wait_bounded(&p_full[w], j & 1, p.status);
                         if (!alive) break;
                         tc_fence_after();
@@ -186,15 +185,15 @@ latent_prefill_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_co
                                 umma_f16_ta(o, pc + (k >> 1) * 32 + (k & 1) * 8 + 16, bd + 2 * k, iv, 1);
                             }
                             // the entry is free once the last tile that uses it has read it
-                            if (w == 1 || j >= nblk[1]) umma_commit(&v_empty[vs]);
+                            if (w == 1 || j >= nblk1) umma_commit(&v_empty[vs]);
                         }
                         if (!alive) break;
-                        if (j == nblk[w] - 1) umma_commit(&o_full[w]);
+                        if (j == (w ? nblk1 : nblk0) - 1) umma_commit(&o_full[w]);
                     }
                     const int jn = j + 1;
-                    if (jn < nblk[w]) {
+                    if (jn < (w ? nblk1 : nblk0)) {
                         // first use of a key block waits for it
-                        if (w == 0 || jn >= nblk[0]) {
+                        if (w == 0 || jn >= nblk0) {
                             alive = mbar_wait_bounded(&k_full[ks], kp, p.status);
                             if (!alive) break;
                             tc_fence_after();
@@ -204,7 +203,7 @@ latent_prefill_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_co
                         products(tmem + w * kBlock, a, b, nd, is, 0);
                         products(tmem + w * kBlock, a + rot, b + rot, nr, is, 1);
                         umma_commit(&s_full[w]);
-                        if (w == 1 || jn >= nblk[1]) umma_commit(&k_empty[ks]);
+                        if (w == 1 || jn >= nblk1) umma_commit(&k_empty[ks]);
                     }
                 }
                 if (++ks == p.k_stages) { ks = 0; kp ^= 1; }
@@ -226,7 +225,7 @@ latent_prefill_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_co
         const float c = p.scale_log2;
         float m = -INFINITY, l = 0.0f;
         bool alive = true;
-        const int n = w == 0 ? nblk[0] : nblk[1];
+        const int n = w == 0 ? nblk0 : nblk1;
         for (int j = 0; j < n; ++j) {
             alive = mbar_wait_bounded(&s_full[w], j & 1, p.status);
             alive = __all_sync(0xffffffffu, alive);

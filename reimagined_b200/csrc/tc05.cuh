@@ -10,6 +10,21 @@
 namespace tbl {
 namespace tc05 {
 
+// The warp's index as a value the compiler knows to be the same in all lanes, and one elected lane of a converged warp: code
+// under both keeps addresses and descriptors in uniform registers, which is where tcgen05 and TMA instructions take them from.
+__device__ __forceinline__ int uniform_warp() { return __shfl_sync(0xffffffffu, static_cast<int>(threadIdx.x >> 5), 0); }
+__device__ __forceinline__ bool elect_one() {
+    uint32_t p;
+    asm volatile(
+        "{\n"
+        ".reg .pred q;\n"
+        "elect.sync _|q, 0xffffffff;\n"
+        "selp.u32 %0, 1, 0, q;\n"
+        "}\n"
+        : "=r"(p));
+    return p != 0;
+}
+
 __device__ __forceinline__ void tma_load_2d(void* dst, const CUtensorMap* map, int c0, int c1, uint64_t* bar) {
     asm volatile(
         "cp.async.bulk.tensor.2d.shared::cluster.global.mbarrier::complete_tx::bytes [%0], [%1, {%2, %3}], [%4];"
