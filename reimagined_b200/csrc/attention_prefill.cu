@@ -83,14 +83,14 @@ attention_flash_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_c
     uint8_t* v_smem = k_smem + p.k_stages * k_bytes;           // ring of half blocks of values
     uint64_t* bars = reinterpret_cast<uint64_t*>(v_smem + p.v_stages * v_bytes);
     uint64_t *q_full = bars, *k_full = bars + 1, *k_empty = k_full + kMaxRing, *v_full = k_empty + kMaxRing, *v_empty = v_full + kMaxRing,
-             *s_full = v_empty + kMaxRing, *p_full = s_full + 2, *o_full = p_full + 2;
+             *s_full = v_empty + kMaxRing, *p_full = s_full + 2, *o_full = p_full + 4;
     uint32_t* tmem_slot = reinterpret_cast<uint32_t*>(o_full + 2);
 
     const int warp = uniform_warp(), lane = threadIdx.x & 31;
     if (threadIdx.x == 0) {
         mbar_init(q_full, 1);
         for (int s = 0; s < kMaxRing; ++s) { mbar_init(&k_full[s], 1); mbar_init(&k_empty[s], 1); mbar_init(&v_full[s], 1); mbar_init(&v_empty[s], 1); }
-        for (int w = 0; w < 2; ++w) { mbar_init(&s_full[w], 1); mbar_init(&p_full[w], 4); mbar_init(&o_full[w], 1); }
+        for (int w = 0; w < 2; ++w) { mbar_init(&s_full[w], 1); mbar_init(&p_full[2 * w], 4); mbar_init(&p_full[2 * w + 1], 4); mbar_init(&o_full[w], 1); }
         fence_mbar_init();
         fence_proxy_async();
     }
@@ -164,13 +164,12 @@ attention_flash_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_c
 #pragma unroll
                 for (int w = 0; w < 2; ++w) {
                     if (j >= 0 && j < (w ? nblk1 : nblk0)) {
-                        alive = mbar_wait_bounded(&p_full[w], j & 1, p.status);
-                        if (!alive) break;
-                        tc_fence_after();
                         const uint32_t o = tmem + kOCol + w * 128;
 #pragma unroll
                         for (int h = 0; h < 2; ++h) {
                             const int vs = h ? v1 : v0;
+                            alive = mbar_wait_bounded(&p_full[2 * w + h], j & 1, p.status);
+                            if (!alive) break;
                             alive = mbar_wait_bounded(&v_full[vs], h ? vp1 : vp0, p.status);
                             if (!alive) break;
                             tc_fence_after();
@@ -227,10 +226,7 @@ attention_flash_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_c
             alive = __all_sync(0xffffffffu, alive);
             if (!alive) break;
             tc_fence_after();
-            softmax_block(s_col, o_col, vcols, pos - j * kBlock, p.scale_log2, j == 0, m, l);
-            tc_fence_before();
-            __syncwarp();
-            if (lane == 0) mbar_arrive(&p_full[w]);
+            softmax_block(s_col, o_col, vcols, pos - j * kBlock, p.scale_log2, j == 0, m, l, p_full + 2 * w, lane);
         }
         const int q = q0 + in_cta;
         const bool ok = q < p.n_tok;
@@ -323,7 +319,7 @@ attention_flash_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_c
     }
 }
 
-constexpr size_t kFixedSmem = 1024 + 8 * (1 + 4 * kMaxRing + 6) + 16;
+constexpr size_t kFixedSmem = 1024 + 8 * (1 + 4 * kMaxRing + 8) + 16;
 constexpr size_t kRoom = 227 * 1024 - kFixedSmem;
 
 struct Rings { int k, v; size_t smem; };
