@@ -259,6 +259,8 @@ int pick_splits(const tbl_attention_mixer& m, int route, int n_seq, int n_tok, i
     const int tokens = ceil_div(context, 64);                       // a split is worth at least a tile of tokens
     long long s = 2LL * kNumSm / units;
     if (s > tokens) s = tokens;
+    // a cluster's worth is enough when that keeps most of the SMs busy, or leaves a CTA little to read
+    if (route == kStream && s > kClusterSplits && (units * kClusterSplits >= kNumSm / 2 || tokens <= 4 * kClusterSplits)) s = kClusterSplits;
     return s < 1 ? 1 : (s > kMergeMaxSplits ? kMergeMaxSplits : static_cast<int>(s));
 }
 
@@ -280,7 +282,7 @@ Plan make_plan(const tbl_attention_mixer& m, int precision, int route, int n_seq
     auto take = [&](size_t bytes) { const size_t at = off; off += round_up(bytes, 256); return at; };
     const size_t units = rows * m.heads * m.maps * w.splits;
     w.q16 = take(w.route == kFlash ? 2 * rows * m.heads * m.maps * padded(m.dim) : 0);
-    const bool parts = w.route == kSimt || (w.route == kStream && w.splits > 1) || (w.route == kFlash && !attention_flash_whole(m));
+    const bool parts = w.route == kSimt || (w.route == kStream && w.splits > kClusterSplits) || (w.route == kFlash && !attention_flash_whole(m));
     w.pm = take(parts ? sizeof(float) * units : 0);
     w.pl = take(parts ? sizeof(float) * units : 0);
     w.po = take(parts ? sizeof(float) * units * padded(m.vdim) : 0);
@@ -300,7 +302,7 @@ int run(const tbl_attention_mixer& m, AttnParams p, const Plan& w, int n_seq, in
     }
     p.append = append && w.fused_append;
     int rc;
-    bool merge = w.splits > 1 || w.route == kSimt;
+    bool merge = w.route == kSimt || w.splits > kClusterSplits;
     if (w.route == kFlash) {
         rc = launch_attention_flash(p, n_seq, context, st);
         merge = !attention_flash_whole(m);

@@ -44,7 +44,9 @@ __device__ __forceinline__ float cache_value(const AttnParams& p, const float* p
     return e < p.vd ? proj_row[p.v_off + g * p.vd + e] : 0.0f;
 }
 
-// attention_decode.cu: streams the cache, warp-level MMAs
+// attention_decode.cu: streams the cache, warp-level MMAs.  Up to kClusterSplits splits of the context are a cluster that
+// finishes the rows itself, more leave partial sums.
+constexpr int kClusterSplits = 8;
 bool attention_stream_supported(const tbl_attention_mixer& m);
 int launch_attention_stream(const AttnParams& p, int n_seq, cudaStream_t st);
 

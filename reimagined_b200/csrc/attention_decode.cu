@@ -5,13 +5,19 @@
 // few tiles ahead.  The products are warp-level MMAs (16 x 8 x 16, bf16): a warp owns one map and 16 tokens of every tile,
 // with its own maximum, sum and output, so that a tile costs one barrier; the quarters meet in shared memory at the end.
 // The scores' fragments become the weights' fragments in place, as two bf16 terms (hi + lo: 16 bits of mantissa).
-// With one split the CTA combines the maps, norms the head and gates the output itself; otherwise it leaves partial sums
-// for attention_merge_kernel.  A decode step appends its token here: the CTA whose split holds it writes it first.
+// The splits of the context are a cluster: its CTAs read each other's sums through distributed shared memory, combine the
+// maps, norm the heads and gate the output, a row at a time each.  Only a context that wants more CTAs than a cluster has
+// leaves partial sums for attention_merge_kernel.  A decode step appends its token here: the CTA whose split holds it
+// takes it from the projections and writes it to the cache.
+#include <cooperative_groups.h>
+
 #include "attention.cuh"
 
 namespace tbl {
 namespace stack {
 namespace {
+
+namespace cg = cooperative_groups;
 
 constexpr int kTile = 64, kRows = 16, kQuarters = 4, kMaxStages = 4;
 
@@ -38,12 +44,13 @@ size_t stream_smem(int maps, int dp, int vp, int stages) {
     return query_smem(maps, dp) + (tiles > merge ? tiles : merge);
 }
 
-// MAPS: maps per head; VN: value columns in steps of 16 a warp has room for
+// MAPS: maps per head; VN: value columns in steps of 16 a warp has room for.  clustered: the splits are a cluster
 template <int MAPS, int VN>
-__global__ void __launch_bounds__(32 * kQuarters * MAPS) attention_stream_kernel(const AttnParams p, const int stages) {
+__global__ void __launch_bounds__(32 * kQuarters * MAPS) attention_stream_kernel(const AttnParams p, const int stages, const int clustered) {
     constexpr int kThreads = 32 * kQuarters * MAPS;
     extern __shared__ __align__(16) uint8_t smem[];
-    __shared__ float m_s[kQuarters][MAPS][kRows], l_s[kQuarters][MAPS][kRows];
+    __shared__ float m_s[kQuarters][MAPS][kRows], l_s[kQuarters][MAPS][kRows], top_s[MAPS][kRows], sum_s[MAPS][kRows], red_s[kQuarters * MAPS];
+    __shared__ float fac_s[MAPS][kClusterSplits];
     const int ld = tile_ld(p.cw), ldq = p.dp + 8;
     bf16* q_s = reinterpret_cast<bf16*>(smem);                          // [MAPS][16][ldq]
     bf16* t_s = q_s + MAPS * kRows * ldq;                               // [stages][64][ld]
@@ -51,20 +58,19 @@ __global__ void __launch_bounds__(32 * kQuarters * MAPS) attention_stream_kernel
     const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, map = warp % MAPS, quarter = warp / MAPS;
     const int seq = blockIdx.x / p.G, g = blockIdx.x % p.G, first = blockIdx.y * kRows, split = blockIdx.z;
     const int total = p.n_tok * p.group;
-    pdl_launch_dependents();
     pdl_wait();
     const int slot = p.slots[seq], pos0 = p.positions[slot];
     const int n = min(pos0 + min(total - 1, first + kRows - 1) / p.group + 1, p.capacity);       // tokens the last row sees
     const int per = ((n + p.splits - 1) / p.splits + kTile - 1) / kTile * kTile;
     const int t0 = min(split * per, n), t1 = min(n, t0 + per);
     bf16* cache = static_cast<bf16*>(p.cache) + cache_row(p, slot, g, 0);
-    if (p.append) {                                                     // n_tok == 1: the token at pos0
+    // a decode step's token (n_tok == 1, at pos0) comes from the projections, not from the cache
+    int fresh = -1;
+    if (p.append) {
         if (pos0 < 0 || pos0 >= p.capacity || (p.temperature && pos0 >= p.temperature_positions)) {
             if (tid == 0 && split == 0) atomicOr(p.status, TBL_DEV_CACHE_FULL);
-        } else if (pos0 >= t0 && pos0 < t1) {
-            const float* pr = p.proj + static_cast<size_t>(seq) * p.ld;
-            for (int c = tid; c < p.cw; c += kThreads) cache[static_cast<size_t>(pos0) * p.cw + c] = __float2bfloat16_rn(cache_value(p, pr, g, c));
-            __syncthreads();                                            // the copies below read it
+        } else {
+            if (pos0 >= t0 && pos0 < t1) fresh = pos0;
         }
     }
     const int chunks = p.cw / 8;
@@ -112,6 +118,15 @@ __global__ void __launch_bounds__(32 * kQuarters * MAPS) attention_stream_kernel
         {
             const int ahead = stage == 0 ? stages - 1 : stage - 1;
             load_tile(ahead, t + (stages - 1) * kTile);
+        }
+        if (fresh >= t && fresh < t + kTile) {               // in the last tile of one split
+            const float* pr = p.proj + static_cast<size_t>(seq) * p.ld;
+            for (int c = tid; c < p.cw; c += kThreads) {
+                const bf16 v = __float2bfloat16_rn(cache_value(p, pr, g, c));
+                t_s[(stage * kTile + fresh - t) * ld + c] = v;
+                cache[static_cast<size_t>(fresh) * p.cw + c] = v;
+            }
+            __syncthreads();
         }
         const bf16* tile = t_s + stage * kTile * ld + quarter * 16 * ld;
         if (++stage == stages) stage = 0;
@@ -188,89 +203,132 @@ __global__ void __launch_bounds__(32 * kQuarters * MAPS) attention_stream_kernel
                         make_float2(o[j][q][2 * h], o[j][q][2 * h + 1]);
         }
     __syncthreads();
-    // a warp per row
+    pdl_launch_dependents();
+    // the quarters come together: sums of this split, a warp per row
     const size_t quarter_step = static_cast<size_t>(MAPS) * kRows * p.vp;
-    for (int r = warp; r < kRows; r += kQuarters * MAPS) {
-        const int at = first + r;
-        if (at >= total) break;
-        const int t = at / p.group, head = g * p.group + at % p.group;
-        const size_t row = static_cast<size_t>(seq) * p.n_tok + t, unit = (row * p.H + head) * MAPS;
-        float fac[MAPS][kQuarters];
+    const int rows = min(kRows, total - first);
+    for (int r = warp; r < rows; r += kQuarters * MAPS) {
 #pragma unroll
         for (int m = 0; m < MAPS; ++m) {
-            float top = m_s[0][m][r], l = 0.0f;
+            float fac[kQuarters], top = m_s[0][m][r], l = 0.0f;
 #pragma unroll
             for (int k = 1; k < kQuarters; ++k) top = fmaxf(top, m_s[k][m][r]);
 #pragma unroll
             for (int k = 0; k < kQuarters; ++k) {
-                fac[m][k] = m_s[k][m][r] == -INFINITY ? 0.0f : ex2(m_s[k][m][r] - top);
-                l = fmaf(l_s[k][m][r], fac[m][k], l);
+                fac[k] = m_s[k][m][r] == -INFINITY ? 0.0f : ex2(m_s[k][m][r] - top);
+                l = fmaf(l_s[k][m][r], fac[k], l);
             }
-            if (p.splits > 1) {
-                if (lane == 0) { p.part_m[(unit + m) * p.splits + split] = top; p.part_l[(unit + m) * p.splits + split] = l; }
-            } else {
-                const float f = (m == 0 ? 1.0f : -p.lambda) / l;
+            if (lane == 0) { top_s[m][r] = top; sum_s[m][r] = l; }
+            float* src = o_s + static_cast<size_t>(m * kRows + r) * p.vp;
+            for (int c = lane; c < p.vd; c += 32) {
+                float v = 0.0f;
 #pragma unroll
-                for (int k = 0; k < kQuarters; ++k) fac[m][k] *= f;
+                for (int k = 0; k < kQuarters; ++k) v = fmaf(src[k * quarter_step + c], fac[k], v);
+                src[c] = v;                                  // over the first quarter, which only this lane reads
             }
         }
-        const float* src = o_s + static_cast<size_t>(r) * p.vp;
-        if (p.splits > 1) {
+    }
+    if (p.splits > 1 && !clustered) {
+        __syncwarp();
+        for (int r = warp; r < rows; r += kQuarters * MAPS) {
+            const int t = (first + r) / p.group, head = g * p.group + (first + r) % p.group;
+            const size_t unit = ((static_cast<size_t>(seq) * p.n_tok + t) * p.H + head) * MAPS;
 #pragma unroll
             for (int m = 0; m < MAPS; ++m) {
-                float* dst = p.part_o + ((unit + m) * p.splits + split) * p.vp;
-                for (int c = lane; c < p.vd; c += 32) {
-                    float v = 0.0f;
-#pragma unroll
-                    for (int k = 0; k < kQuarters; ++k) v = fmaf(src[k * quarter_step + m * kRows * p.vp + c], fac[m][k], v);
-                    dst[c] = v;
-                }
+                const size_t u = (unit + m) * p.splits + split;
+                if (lane == 0) { p.part_m[u] = top_s[m][r]; p.part_l[u] = sum_s[m][r]; }
+                for (int c = lane; c < p.vd; c += 32) p.part_o[u * p.vp + c] = o_s[static_cast<size_t>(m * kRows + r) * p.vp + c];
             }
-            continue;
         }
-        float v[VN / 2], ss = 0.0f;
-#pragma unroll
-        for (int i = 0; i < VN / 2; ++i) {
-            const int c = lane + 32 * i;
-            v[i] = 0.0f;
-            if (c < p.vd) {
-#pragma unroll
-                for (int m = 0; m < MAPS; ++m)
-#pragma unroll
-                    for (int k = 0; k < kQuarters; ++k) v[i] = fmaf(src[k * quarter_step + m * kRows * p.vp + c], fac[m][k], v[i]);
-            }
-            ss = fmaf(v[i], v[i], ss);
+        return;
+    }
+    cg::cluster_group cluster = cg::this_cluster();
+    if (p.splits > 1) cluster.sync();
+    else __syncthreads();
+    // a row at a time: row r is finished by split r mod splits.  v_s (the second quarter's room, read by nobody else): the
+    // maps' weighted averages.
+    float* v_s = o_s + quarter_step;
+    for (int r = split; r < rows; r += p.splits) {
+        if (warp < MAPS) {                                   // a lane per split
+            const float top = lane < p.splits ? *cluster.map_shared_rank(&top_s[warp][r], lane) : -INFINITY;
+            const float l = lane < p.splits ? *cluster.map_shared_rank(&sum_s[warp][r], lane) : 0.0f;
+            const float most = warp_max(top), f = top == -INFINITY ? 0.0f : ex2(top - most);
+            const float total_l = warp_sum(l * f);
+            if (lane < kClusterSplits) fac_s[warp][lane] = f * ((warp == 0 ? 1.0f : -p.lambda) / total_l);
         }
-        const float f = MAPS == 2 ? p.out_scale / sqrtf(warp_sum(ss) / static_cast<float>(p.vd) + p.eps) : 1.0f;
+        __syncthreads();
+        for (int i = tid; i < MAPS * p.vp; i += kThreads) {
+            const int m = MAPS == 2 && i >= p.vp, c = i - m * p.vp;
+            const float* src = o_s + static_cast<size_t>(m * kRows + r) * p.vp + (c < p.vd ? c : 0);
+            float v = 0.0f;
+#pragma unroll
+            for (int k = 0; k < kClusterSplits; ++k)
+                if (k < p.splits) v = fmaf(*cluster.map_shared_rank(src, k), fac_s[m][k], v);
+            v_s[i] = v;
+        }
+        __syncthreads();
+        float x[VN * 16 / kThreads + 1], ss = 0.0f;
+#pragma unroll
+        for (int i = 0; i < VN * 16 / kThreads + 1; ++i) {
+            const int c = tid + i * kThreads;
+            x[i] = c < p.vd ? v_s[c] + (MAPS == 2 ? v_s[p.vp + c] : 0.0f) : 0.0f;
+            ss = fmaf(x[i], x[i], ss);
+        }
+        float f = 1.0f;
+        if (MAPS == 2) {
+            ss = warp_sum(ss);
+            if (lane == 0) red_s[warp] = ss;
+            __syncthreads();
+            ss = 0.0f;
+#pragma unroll
+            for (int k = 0; k < kQuarters * MAPS; ++k) ss += red_s[k];
+            f = p.out_scale / sqrtf(ss / static_cast<float>(p.vd) + p.eps);
+        }
+        const int t = (first + r) / p.group, head = g * p.group + (first + r) % p.group;
+        const size_t row = static_cast<size_t>(seq) * p.n_tok + t;
         const float* gate = p.g_off < 0 ? nullptr : p.proj + row * p.ld + p.g_off + head * p.vd;
         bf16* out = static_cast<bf16*>(p.out) + (row * p.H + head) * p.vd;
 #pragma unroll
-        for (int i = 0; i < VN / 2; ++i) {
-            const int c = lane + 32 * i;
-            if (c < p.vd) out[c] = __float2bfloat16_rn(v[i] * f * (gate ? sigmoid_f(gate[c]) : 1.0f));
+        for (int i = 0; i < VN * 16 / kThreads + 1; ++i) {
+            const int c = tid + i * kThreads;
+            if (c < p.vd) out[c] = __float2bfloat16_rn(x[i] * f * (gate ? sigmoid_f(gate[c]) : 1.0f));
         }
+        __syncthreads();                                     // v_s, red_s and fac_s are free again
     }
+    if (p.splits > 1) cluster.sync();                        // nobody leaves while a neighbour may still read its sums
 }
 
+// Tiles in shared memory: two CTAs of an SM take no more than kShare together.  Shared memory comes off the SM's first-level
+// cache, and the linear layers on either side, whose CTAs share the SM with this kernel's, read their activations through that.
+constexpr size_t kShare = 160 * 1024;
+
 int pick_stages(int maps, int dp, int vp) {
-    // two CTAs per SM where three tiles each allow it, one with what fits otherwise
-    for (int s = kMaxStages; s >= 2; --s)
-        if (stream_smem(maps, dp, vp, s) <= 110 * 1024) return s;
-    for (int s = kMaxStages; s >= 2; --s)
-        if (stream_smem(maps, dp, vp, s) <= 220 * 1024) return s;
-    return 0;
+    for (int s = kMaxStages; s > 2; --s)
+        if (stream_smem(maps, dp, vp, s) <= kShare / 2) return s;
+    return stream_smem(maps, dp, vp, 2) <= 220 * 1024 ? 2 : 0;
 }
 
 template <int MAPS, int VN>
 cudaError_t launch(const AttnParams& p, int n_seq, cudaStream_t st) {
     static bool done[64] = {};
+    const dim3 grid(n_seq * p.G, ceil_div(static_cast<long long>(p.n_tok) * p.group, kRows), p.splits);
     const int stages = pick_stages(MAPS, p.dp, p.vp);
     const size_t smem = stream_smem(MAPS, p.dp, p.vp, stages);
     const cudaError_t e = allow_smem(attention_stream_kernel<MAPS, VN>, smem, done);
     if (e != cudaSuccess) return e;
-    const dim3 grid(n_seq * p.G, ceil_div(static_cast<long long>(p.n_tok) * p.group, kRows), p.splits);
     if (grid.y > 65535) return cudaErrorInvalidValue;
-    return launch_dependent(attention_stream_kernel<MAPS, VN>, grid, dim3(32 * kQuarters * MAPS), smem, st, p, stages);
+    const bool clustered = p.splits > 1 && p.splits <= kClusterSplits;
+    cudaLaunchConfig_t cfg{};
+    cfg.gridDim = grid; cfg.blockDim = dim3(32 * kQuarters * MAPS); cfg.dynamicSmemBytes = smem; cfg.stream = st;
+    cudaLaunchAttribute attr[2];
+    attr[0].id = cudaLaunchAttributeProgrammaticStreamSerialization;
+    attr[0].val.programmaticStreamSerializationAllowed = 1;
+    attr[1].id = cudaLaunchAttributeClusterDimension;
+    attr[1].val.clusterDim.x = 1; attr[1].val.clusterDim.y = 1; attr[1].val.clusterDim.z = p.splits;
+    cfg.attrs = attr; cfg.numAttrs = clustered ? 2 : 1;
+    const cudaError_t r = cudaLaunchKernelEx(&cfg, attention_stream_kernel<MAPS, VN>, p, stages, static_cast<int>(clustered));
+    note_launch();
+    return r;
 }
 
 template <int MAPS>
