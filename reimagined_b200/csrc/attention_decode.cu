@@ -1,8 +1,8 @@
 // Attention of a few query rows over a long cache (decode, short portions): the cache streams through shared memory once
 // per block of 16 query rows that share a key/value head.
 //
-// A CTA handles (sequence, kv head, block of rows, split of the context) in tiles of 64 tokens, brought in by cp.async a
-// few tiles ahead.  The products are warp-level MMAs (16 x 8 x 16, bf16): a warp owns one map and 16 tokens of every tile,
+// A CTA handles (sequence, kv head, block of rows, split of the context) in tiles of 64 tokens, brought in by TMA
+// ahead of their use as sub-tiles of 64 columns with the 128-byte swizzle (conflict-free for ldmatrix).  The products are warp-level MMAs (16 x 8 x 16, bf16): a warp owns one map and 16 tokens of every tile,
 // with its own maximum, sum and output, so that a tile costs one barrier; the quarters meet in shared memory at the end.
 // The scores' fragments become the weights' fragments in place, as two bf16 terms (hi + lo: 16 bits of mantissa).
 // The splits of the context are a cluster: its CTAs read each other's sums through distributed shared memory, combine the
@@ -10,8 +10,10 @@
 // leaves partial sums for attention_merge_kernel.  A decode step appends its token here: the CTA whose split holds it
 // takes it from the projections and writes it to the cache.
 #include <cooperative_groups.h>
+#include <cuda.h>
 
 #include "attention.cuh"
+#include "tc05.cuh"
 
 namespace tbl {
 namespace stack {
@@ -20,6 +22,7 @@ namespace {
 namespace cg = cooperative_groups;
 
 constexpr int kTile = 64, kRows = 16, kQuarters = 4, kMaxStages = 4;
+constexpr float kRescale = 8.0f;
 
 __device__ __forceinline__ void ldsm4(uint32_t (&r)[4], uint32_t a) {
     asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0,%1,%2,%3}, [%4];" : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(a));
@@ -30,34 +33,40 @@ __device__ __forceinline__ void ldsm4t(uint32_t (&r)[4], uint32_t a) {
 __device__ __forceinline__ void mma(float (&d)[4], const uint32_t (&a)[4], uint32_t b0, uint32_t b1) {
     mma16816(d, a[0], a[1], a[2], a[3], b0, b1);
 }
-__device__ __forceinline__ void cp16(uint32_t dst, const void* src, bool ok) {
-    asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(dst), "l"(src), "r"(ok ? 16 : 0) : "memory");
-}
-
-__host__ __device__ __forceinline__ int tile_ld(int cw) { return cw + 8; }      // an odd number of 16-byte units: conflict-free ldmatrix
+constexpr int kSub = kTile * 128;               // bytes of a sub-tile: 64 tokens x 64 columns
+__host__ __device__ __forceinline__ int sub_tiles(int cw) { return (cw + 63) / 64; }
 
 size_t query_smem(int maps, int dp) { return 2 * static_cast<size_t>(kRows) * maps * (dp + 8); }
-size_t tile_smem(int cw) { return 2 * static_cast<size_t>(kTile) * tile_ld(cw); }
 size_t merge_smem(int maps, int vp) { return sizeof(float) * kQuarters * maps * kRows * static_cast<size_t>(vp); }
-size_t stream_smem(int maps, int dp, int vp, int stages) {
-    const size_t tiles = stages * tile_smem(maps * dp + vp), merge = merge_smem(maps, vp);
-    return query_smem(maps, dp) + (tiles > merge ? tiles : merge);
+size_t tiles_smem(int maps, int dp, int vp, int stages) {
+    const size_t tiles = static_cast<size_t>(stages) * sub_tiles(maps * dp + vp) * kSub, merge = merge_smem(maps, vp);
+    return tiles > merge ? tiles : merge;
 }
+size_t stream_smem(int maps, int dp, int vp, int stages) { return 1024 + tiles_smem(maps, dp, vp, stages) + query_smem(maps, dp); }
 
 // MAPS: maps per head; VN: value columns in steps of 16 a warp has room for.  clustered: the splits are a cluster
 template <int MAPS, int VN>
-__global__ void __launch_bounds__(32 * kQuarters * MAPS) attention_stream_kernel(const AttnParams p, const int stages, const int clustered) {
+__global__ void __launch_bounds__(32 * kQuarters * MAPS) attention_stream_kernel(const __grid_constant__ CUtensorMap map_c, const AttnParams p,
+                                                                               const int stages, const int q_at, const int clustered) {
     constexpr int kThreads = 32 * kQuarters * MAPS;
-    extern __shared__ __align__(16) uint8_t smem[];
+    extern __shared__ __align__(1024) uint8_t smem_raw[];
+    uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~uintptr_t(1023));
     __shared__ float m_s[kQuarters][MAPS][kRows], l_s[kQuarters][MAPS][kRows], top_s[MAPS][kRows], sum_s[MAPS][kRows], red_s[kQuarters * MAPS];
     __shared__ float fac_s[MAPS][kClusterSplits];
-    const int ld = tile_ld(p.cw), ldq = p.dp + 8;
-    bf16* q_s = reinterpret_cast<bf16*>(smem);                          // [MAPS][16][ldq]
-    bf16* t_s = q_s + MAPS * kRows * ldq;                               // [stages][64][ld]
-    float* o_s = reinterpret_cast<float*>(t_s);                         // afterwards: [quarter][MAPS][16][vp]
-    const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, map = warp % MAPS, quarter = warp / MAPS;
+    __shared__ __align__(8) uint64_t full[kMaxStages];
+    const int ldq = p.dp + 8, tile_bytes = sub_tiles(p.cw) * kSub;
+    uint8_t* t_s = smem;                                                // [stages][sub-tile][64 tokens][128 bytes]
+    float* o_s = reinterpret_cast<float*>(smem);                        // afterwards: [quarter][MAPS][16][vp]
+    bf16* q_s = reinterpret_cast<bf16*>(smem + q_at);                   // [MAPS][16][ldq]
+    const int tid = threadIdx.x, warp = tc05::uniform_warp(), lane = tid & 31, map = warp % MAPS, quarter = warp / MAPS;
     const int seq = blockIdx.x / p.G, g = blockIdx.x % p.G, first = blockIdx.y * kRows, split = blockIdx.z;
     const int total = p.n_tok * p.group;
+    if (tid == 0) {
+        for (int s = 0; s < kMaxStages; ++s) mbar_init(&full[s], 1);
+        fence_mbar_init();
+        fence_proxy_async();
+    }
+    __syncthreads();
     pdl_wait();
     const int slot = p.slots[seq], pos0 = p.positions[slot];
     const int n = min(pos0 + min(total - 1, first + kRows - 1) / p.group + 1, p.capacity);       // tokens the last row sees
@@ -73,19 +82,13 @@ __global__ void __launch_bounds__(32 * kQuarters * MAPS) attention_stream_kernel
             if (pos0 >= t0 && pos0 < t1) fresh = pos0;
         }
     }
-    const int chunks = p.cw / 8;
+    // Rows past the split's end come along: their tokens are masked, and a weight of zero only needs a finite value beside it.
+    const int row0 = (slot * p.G + g) * p.capacity;
     auto load_tile = [&](int stage, int t) {
-        if (t < t1) {
-            const uint32_t base = smem_u32(t_s + stage * kTile * ld);
-            // a warp takes whole rows, its lanes the 16-byte pieces: no division per piece
-#pragma unroll 4
-            for (int r = warp; r < kTile; r += kQuarters * MAPS) {
-                const bool ok = t + r < t1;
-                const bf16* src = cache + static_cast<size_t>(ok ? t + r : 0) * p.cw;
-                for (int c = lane; c < chunks; c += 32) cp16(base + (r * ld + c * 8) * 2, src + c * 8, ok);
-            }
+        if (warp == 0 && t < t1 && tc05::elect_one()) {
+            mbar_arrive_expect_tx(&full[stage], tile_bytes);
+            for (int c = 0; c * 64 < p.cw; ++c) tc05::tma_load_2d(t_s + stage * tile_bytes + c * kSub, &map_c, c * 64, row0 + t, &full[stage]);
         }
-        asm volatile("cp.async.commit_group;" ::: "memory");
     };
     for (int s = 0; s < kMaxStages - 1; ++s)
         if (s < stages - 1) load_tile(s, t0 + s * kTile);
@@ -109,51 +112,65 @@ __global__ void __launch_bounds__(32 * kQuarters * MAPS) attention_stream_kernel
     for (int h = 0; h < 2; ++h) last[h] = min(pos0 + min(first + (lane >> 2) + 8 * h, total - 1) / p.group, t1 - 1);
     const int tiles16 = p.vp / 16;
     const uint32_t a_addr = smem_u32(q_s + (map * kRows + (lane & 15)) * ldq + (lane >> 4) * 8);
+    const bool upper = total - first > kRows / 2;                      // rows 8 .. 15 in use
+    const int all_see = min(pos0 + first / p.group, t1 - 1);            // the last token that every row sees
+    bool alive = true;
+    uint32_t phase = 0;
     int stage = 0;
     for (int t = t0; t < t1; t += kTile) {
-        if (stages == 2) asm volatile("cp.async.wait_group 0;" ::: "memory");
-        else if (stages == 3) asm volatile("cp.async.wait_group 1;" ::: "memory");
-        else asm volatile("cp.async.wait_group 2;" ::: "memory");
+        // (after a wait that gave up nothing more is asked for, and what is on its way gets a short time)
+        alive = __all_sync(0xffffffffu, mbar_wait_bounded(&full[stage], phase, p.status, alive ? kWaitSpinLimit : 1024)) && alive;
         __syncthreads();                                     // the tile is there, and the one before it is no longer read
         {
             const int ahead = stage == 0 ? stages - 1 : stage - 1;
-            load_tile(ahead, t + (stages - 1) * kTile);
+            if (alive) load_tile(ahead, t + (stages - 1) * kTile);
         }
         if (fresh >= t && fresh < t + kTile) {               // in the last tile of one split
             const float* pr = p.proj + static_cast<size_t>(seq) * p.ld;
             for (int c = tid; c < p.cw; c += kThreads) {
                 const bf16 v = __float2bfloat16_rn(cache_value(p, pr, g, c));
-                t_s[(stage * kTile + fresh - t) * ld + c] = v;
+                const int r = fresh - t;
+                reinterpret_cast<bf16*>(t_s + stage * tile_bytes + (c >> 6) * kSub + r * 128 + ((((c >> 3) & 7) ^ (r & 7)) << 4))[c & 7] = v;
                 cache[static_cast<size_t>(fresh) * p.cw + c] = v;
             }
             __syncthreads();
         }
-        const bf16* tile = t_s + stage * kTile * ld + quarter * 16 * ld;
-        if (++stage == stages) stage = 0;
+        const uint32_t tile = smem_u32(t_s + stage * tile_bytes) + quarter * 16 * 128;
+        if (++stage == stages) { stage = 0; phase ^= 1; }
         // scores: 16 rows x 16 tokens
         float s[2][4] = {};
-        const uint32_t b_addr = smem_u32(tile + ((lane & 7) + (lane >> 4) * 8) * ld + map * p.dp + ((lane >> 3) & 1) * 8);
+        const uint32_t k_row = tile + ((lane & 7) + (lane >> 4) * 8) * 128;
+        const uint32_t k_mix = ((lane >> 3) & 1) ^ (lane & 7);            // 16-byte piece c of a row r lies at c ^ (r & 7)
 #pragma unroll 4
         for (int k = 0; k < p.dp; k += 16) {
             uint32_t a[4], b[4];
+            const int piece = (map * p.dp + k) >> 3;
             ldsm4(a, a_addr + k * 2);
-            ldsm4(b, b_addr + k * 2);
+            ldsm4(b, k_row + (piece >> 3) * kSub + (((piece & 7) ^ k_mix) << 4));
             mma(s[0], a, b[0], b[1]);
             mma(s[1], a, b[2], b[3]);
         }
         const int token = t + quarter * 16 + (lane & 3) * 2;
-        uint32_t hi[4], lo[4];
-        float f[2];
+        const bool whole = t + kTile - 1 <= all_see;         // nothing of the tile is masked
+        uint32_t hi[4] = {}, lo[4] = {};
+        float f[2] = {1.0f, 1.0f};
 #pragma unroll
         for (int h = 0; h < 2; ++h) {
+            if (h == 1 && !upper) break;
             float x[4];
 #pragma unroll
-            for (int e = 0; e < 4; ++e) x[e] = token + (e >> 1) * 8 + (e & 1) <= last[h] ? s[e >> 1][2 * h + (e & 1)] * p.scale_log2 : -INFINITY;
+            for (int e = 0; e < 4; ++e) x[e] = s[e >> 1][2 * h + (e & 1)] * p.scale_log2;
+            if (!whole) {
+#pragma unroll
+                for (int e = 0; e < 4; ++e)
+                    if (token + (e >> 1) * 8 + (e & 1) > last[h]) x[e] = -INFINITY;
+            }
             float top = fmaxf(fmaxf(x[0], x[1]), fmaxf(x[2], x[3]));
             top = fmaxf(top, __shfl_xor_sync(0xffffffffu, top, 1));
             top = fmaxf(top, __shfl_xor_sync(0xffffffffu, top, 2));
-            const float mn = fmaxf(mx[h], top), base = mn == -INFINITY ? 0.0f : mn;      // nothing seen yet: all weights zero
-            f[h] = ex2(mx[h] - base);
+            // the maximum only moves when it grows by 2^8: then output and sum are rescaled
+            const float mn = top > mx[h] + kRescale ? top : mx[h], base = mn == -INFINITY ? 0.0f : mn;   // nothing seen yet: all weights zero
+            f[h] = mn == mx[h] ? 1.0f : ex2(mx[h] - base);
             mx[h] = mn;
 #pragma unroll
             for (int e = 0; e < 4; ++e) x[e] = ex2(x[e] - base);
@@ -170,12 +187,13 @@ __global__ void __launch_bounds__(32 * kQuarters * MAPS) attention_stream_kernel
 #pragma unroll
                 for (int q = 0; q < 2; ++q) { o[j][q][0] *= f[0]; o[j][q][1] *= f[0]; o[j][q][2] *= f[1]; o[j][q][3] *= f[1]; }
         }
-        const uint32_t v_addr = smem_u32(tile + (lane & 15) * ld + MAPS * p.dp + (lane >> 4) * 8);
+        const uint32_t v_row = tile + (lane & 15) * 128, v_mix = (lane >> 4) ^ (lane & 7);
 #pragma unroll
         for (int j = 0; j < VN; ++j) {
             if (j < tiles16) {
                 uint32_t b[4];
-                ldsm4t(b, v_addr + j * 32);
+                const int piece = (MAPS * p.dp >> 3) + 2 * j;
+                ldsm4t(b, v_row + (piece >> 3) * kSub + (((piece & 7) ^ v_mix) << 4));
                 mma(o[j][0], hi, b[0], b[1]);
                 mma(o[j][1], hi, b[2], b[3]);
                 mma(o[j][0], lo, b[0], b[1]);
@@ -183,7 +201,6 @@ __global__ void __launch_bounds__(32 * kQuarters * MAPS) attention_stream_kernel
             }
         }
     }
-    asm volatile("cp.async.wait_group 0;" ::: "memory");
     __syncthreads();                                         // tiles are done with: their room takes the outputs
 #pragma unroll
     for (int h = 0; h < 2; ++h) {
@@ -318,6 +335,10 @@ cudaError_t launch(const AttnParams& p, int n_seq, cudaStream_t st) {
     if (e != cudaSuccess) return e;
     if (grid.y > 65535) return cudaErrorInvalidValue;
     const bool clustered = p.splits > 1 && p.splits <= kClusterSplits;
+    const long long cached = static_cast<long long>(p.n_slots) * p.G * p.capacity;
+    CUtensorMap map_c;
+    if (cached > 2147483647LL || !tc05::make_map(&map_c, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, p.cache, cached, p.cw, 64, kTile))
+        return cudaErrorInvalidValue;
     cudaLaunchConfig_t cfg{};
     cfg.gridDim = grid; cfg.blockDim = dim3(32 * kQuarters * MAPS); cfg.dynamicSmemBytes = smem; cfg.stream = st;
     cudaLaunchAttribute attr[2];
@@ -326,7 +347,8 @@ cudaError_t launch(const AttnParams& p, int n_seq, cudaStream_t st) {
     attr[1].id = cudaLaunchAttributeClusterDimension;
     attr[1].val.clusterDim.x = 1; attr[1].val.clusterDim.y = 1; attr[1].val.clusterDim.z = p.splits;
     cfg.attrs = attr; cfg.numAttrs = clustered ? 2 : 1;
-    const cudaError_t r = cudaLaunchKernelEx(&cfg, attention_stream_kernel<MAPS, VN>, p, stages, static_cast<int>(clustered));
+    const cudaError_t r = cudaLaunchKernelEx(&cfg, attention_stream_kernel<MAPS, VN>, map_c, p, stages,
+                                             static_cast<int>(tiles_smem(MAPS, p.dp, p.vp, stages)), static_cast<int>(clustered));
     note_launch();
     return r;
 }
