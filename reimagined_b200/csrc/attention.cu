@@ -260,7 +260,7 @@ int pick_splits(const tbl_attention_mixer& m, int route, int n_seq, int n_tok, i
     long long s = 2LL * kNumSm / units;
     if (s > tokens) s = tokens;
     // a cluster's worth is enough when that keeps most of the SMs busy, or leaves a CTA little to read
-    if (route == kStream && s > kClusterSplits && (units * kClusterSplits >= kNumSm / 2 || tokens <= 4 * kClusterSplits)) s = kClusterSplits;
+    if (route == kStream && s > kClusterSplits && (units * kClusterSplits >= kNumSm / 2 || tokens <= 8 * kClusterSplits)) s = kClusterSplits;
     return s < 1 ? 1 : (s > kMergeMaxSplits ? kMergeMaxSplits : static_cast<int>(s));
 }
 

@@ -26,7 +26,6 @@ struct AttnParams {
     float scale_log2, lambda, out_scale, eps;
 };
 
-__device__ __forceinline__ float ex2(float x) { float r; asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(r) : "f"(x)); return r; }
 __device__ __forceinline__ float temperature_of(const AttnParams& p, int pos) {
     return p.temperature ? __ldg(p.temperature + min(max(pos, 0), p.temperature_positions - 1)) : 1.0f;
 }

@@ -24,15 +24,6 @@ namespace cg = cooperative_groups;
 constexpr int kTile = 64, kRows = 16, kQuarters = 4, kMaxStages = 4;
 constexpr float kRescale = 8.0f;
 
-__device__ __forceinline__ void ldsm4(uint32_t (&r)[4], uint32_t a) {
-    asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0,%1,%2,%3}, [%4];" : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(a));
-}
-__device__ __forceinline__ void ldsm4t(uint32_t (&r)[4], uint32_t a) {
-    asm volatile("ldmatrix.sync.aligned.m8n8.x4.trans.shared.b16 {%0,%1,%2,%3}, [%4];" : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(a));
-}
-__device__ __forceinline__ void mma(float (&d)[4], const uint32_t (&a)[4], uint32_t b0, uint32_t b1) {
-    mma16816(d, a[0], a[1], a[2], a[3], b0, b1);
-}
 constexpr int kSub = kTile * 128;               // bytes of a sub-tile: 64 tokens x 64 columns
 __host__ __device__ __forceinline__ int sub_tiles(int cw) { return (cw + 63) / 64; }
 

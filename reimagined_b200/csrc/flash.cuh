@@ -23,8 +23,6 @@ constexpr int kThreads = 32 * (kSoftWarps + 2);
 constexpr int kOCol = 256;
 constexpr float kRescale = 8.0f;
 
-__device__ __forceinline__ float pow2(float x) { float r; asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(r) : "f"(x)); return r; }
-
 // two fp32 numbers per instruction
 __device__ __forceinline__ uint64_t pair_of(float a, float b) {
     uint64_t r;
@@ -88,7 +86,7 @@ __device__ __forceinline__ void softmax_block(uint32_t s_col, uint32_t o_col, in
     if (first) {
         m = top;
     } else if (__any_sync(0xffffffffu, top > m + kRescale)) {
-        const float mn = fmaxf(m, top), f = pow2(m - mn);
+        const float mn = fmaxf(m, top), f = ex2(m - mn);
         m = mn;
         l *= f;
 #pragma unroll 1
@@ -110,8 +108,8 @@ __device__ __forceinline__ void softmax_block(uint32_t s_col, uint32_t o_col, in
         for (int i = 0; i < 16; ++i) {
             float p0, p1;
             unpair(fma2(pair_of(__uint_as_float(x[ch][2 * i]), __uint_as_float(x[ch][2 * i + 1])), cc, mm), p0, p1);
-            p0 = pow2(p0);
-            p1 = pow2(p1);
+            p0 = ex2(p0);
+            p1 = ex2(p1);
             const uint64_t p = pair_of(p0, p1);
             sums[i & 1] = add2(sums[i & 1], p);
             // the high term cut off, the low term the (exact) rest rounded

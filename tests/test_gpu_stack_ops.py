@@ -597,3 +597,29 @@ def test_attention_reports_a_full_cache(cuda, stack_lib):
                                                n, 16, out.data_ptr(), ws.data_ptr(), size, stream(cuda)) == 0
         assert stack_lib.tbl_device_status(stream(cuda)) == 4
         assert cuda.equal(before, a.cache[1:])
+
+
+@pytest.mark.parametrize("precision,route", [(0, A_SIMT), (1, A_STREAM), (1, A_FLASH)])
+def test_attention_finds_keys_far_back_in_a_long_cache(cuda, stack_lib, precision, route):
+    """More splits of the context than a cluster has: single tokens and a short portion behind a long prompt, the first
+    map's queries aimed at keys at its start, at tile and block borders and at its end."""
+    cfg = {**ATT["small"], "heads": 2, "kv_heads": 1, "q_temp": {"coef": 0.05, "every": 1000}}
+    a = Attention(cuda, stack_lib, cfg, precision, slots=2, capacity=4800, lam=1.2)
+    H, d, vd, n = 2, cfg["dim"], cfg["vdim"], 4700
+    rng = np.random.default_rng(3)
+    proj = rng.standard_normal((n + 28, a.cols)).astype(np.float32)
+    k = proj[:, H * 2 * d:(H + 1) * 2 * d].reshape(-1, 2, d)
+    k /= np.sqrt((k ** 2).sum(-1, keepdims=True))
+    v = proj[:, (H + 1) * 2 * d:(H + 1) * 2 * d + vd]
+    target = [0, 1, 63, 64, 127, 128, 2047, 2048, 4095, 4096, 4607, 4608, 4699, 4700] * 2
+    q = proj[:, :H * 2 * d].reshape(-1, H, 2, d)
+    q *= 0.1
+    for i, t in enumerate(target):
+        q[n + i, :, 0] = 45.0 / cfg["scale"] * k[t, 0]
+    a.forward(0, [1], proj[:n])
+    a.ocache[1] = [(k[t][None].astype(np.float64), v[t][None].astype(np.float64)) for t in range(n)]
+    at = n
+    for c in [1] * 14 + [3, 2, 9]:
+        got, want = a.forward(route, [1], proj[at:at + c]), a.oracle([1], proj[at:at + c])
+        rows_close(got, want, 6e-2 if precision else 1e-4, at)
+        at += c
