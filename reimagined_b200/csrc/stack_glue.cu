@@ -212,12 +212,12 @@ int launch_depth_norm_cl(const DepthNorm& p, cudaStream_t st) {
     if (allow_smem(depth_norm_kernel<T, CL, S>, smem, done) != cudaSuccess) return TBL_ERR_CUDA;
     cudaLaunchConfig_t cfg{};
     cfg.gridDim = dim3(p.rows * CL); cfg.blockDim = dim3(kRowThreads); cfg.dynamicSmemBytes = smem; cfg.stream = st;
-    // Not a programmatic dependent of the kernel before it: between two kernels that overlap an SM cannot change its split of
-    // first-level cache and shared memory, and the linear layers after an attention kernel would run with what that left.
-    cudaLaunchAttribute attr[1];
-    attr[0].id = cudaLaunchAttributeClusterDimension;
-    attr[0].val.clusterDim.x = CL; attr[0].val.clusterDim.y = 1; attr[0].val.clusterDim.z = 1;
-    cfg.attrs = attr; cfg.numAttrs = CL > 1 ? 1 : 0;
+    cudaLaunchAttribute attr[2];
+    attr[0].id = cudaLaunchAttributeProgrammaticStreamSerialization;
+    attr[0].val.programmaticStreamSerializationAllowed = 1;
+    attr[1].id = cudaLaunchAttributeClusterDimension;
+    attr[1].val.clusterDim.x = CL; attr[1].val.clusterDim.y = 1; attr[1].val.clusterDim.z = 1;
+    cfg.attrs = attr; cfg.numAttrs = CL > 1 ? 2 : 1;
     const cudaError_t e = cudaLaunchKernelEx(&cfg, depth_norm_kernel<T, CL, S>, p);
     note_launch();
     return e == cudaSuccess ? TBL_OK : TBL_ERR_CUDA;
