@@ -291,7 +291,7 @@ Plan make_plan(const tbl_attention_mixer& m, int precision, int route, int n_seq
 }
 
 template <typename T>
-int run(const tbl_attention_mixer& m, AttnParams p, const Plan& w, int n_seq, int context, cudaStream_t st) {
+int run(const tbl_attention_mixer& m, AttnParams p, const Plan& w, int n_seq, cudaStream_t st) {
     const int rows = n_seq * p.n_tok;
     const bool append = m.kv_from < 0;
     bf16* q16 = p.q16;
@@ -304,7 +304,7 @@ int run(const tbl_attention_mixer& m, AttnParams p, const Plan& w, int n_seq, in
     int rc;
     bool merge = w.route == kSimt || w.splits > kClusterSplits;
     if (w.route == kFlash) {
-        rc = launch_attention_flash(p, n_seq, context, st);
+        rc = launch_attention_flash(p, n_seq, st);
         merge = !attention_flash_whole(m);
     } else if (w.route == kStream) {
         rc = launch_attention_stream(p, n_seq, st);
@@ -359,7 +359,7 @@ int launch_attention(const tbl_attention_mixer& m, int precision, int route, flo
     p.n_slots = n_slots; p.capacity = capacity; p.n_tok = n_tok; p.splits = w.splits;
     p.vec = (p.ld | m.dim | m.vdim) % 4 == 0 && (reinterpret_cast<uintptr_t>(proj) & 15) == 0;
     p.scale_log2 = static_cast<float>(static_cast<double>(m.scale) * 1.4426950408889634); p.lambda = m.lambda; p.out_scale = m.out_scale; p.eps = eps;
-    return precision == TBL_BF16 ? run<bf16>(m, p, w, n_seq, context, st) : run<float>(m, p, w, n_seq, context, st);
+    return precision == TBL_BF16 ? run<bf16>(m, p, w, n_seq, st) : run<float>(m, p, w, n_seq, st);
 }
 
 }  // namespace stack

@@ -52,7 +52,7 @@ int launch_attention_stream(const AttnParams& p, int n_seq, cudaStream_t st);
 // attention_prefill.cu: flash attention on tcgen05
 bool attention_flash_supported(const tbl_attention_mixer& m);
 bool attention_flash_whole(const tbl_attention_mixer& m);    // a CTA holds a head's whole output (otherwise it leaves partial sums)
-int launch_attention_flash(const AttnParams& p, int n_seq, int context, cudaStream_t st);
+int launch_attention_flash(const AttnParams& p, int n_seq, cudaStream_t st);
 
 }  // namespace stack
 }  // namespace tbl

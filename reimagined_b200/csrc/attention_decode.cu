@@ -1,9 +1,10 @@
 // Attention of a few query rows over a long cache (decode, short portions): the cache streams through shared memory once
 // per block of 16 query rows that share a key/value head.
 //
-// A CTA handles (sequence, kv head, block of rows, split of the context) in tiles of 64 tokens, brought in by TMA
-// ahead of their use as sub-tiles of 64 columns with the 128-byte swizzle (conflict-free for ldmatrix).  The products are warp-level MMAs (16 x 8 x 16, bf16): a warp owns one map and 16 tokens of every tile,
-// with its own maximum, sum and output, so that a tile costs one barrier; the quarters meet in shared memory at the end.
+// A CTA handles (sequence, kv head, block of rows, split of the context) in tiles of 64 tokens, brought in by TMA ahead of
+// their use as sub-tiles of 64 columns with the 128-byte swizzle (conflict-free for ldmatrix).  The products are warp-level
+// MMAs (16 x 8 x 16, bf16): a warp owns one map and 16 tokens of every tile, with its own maximum, sum and output, so that
+// a tile costs one barrier; the quarters meet in shared memory at the end.
 // The scores' fragments become the weights' fragments in place, as two bf16 terms (hi + lo: 16 bits of mantissa).
 // The splits of the context are a cluster: its CTAs read each other's sums through distributed shared memory, combine the
 // maps, norm the heads and gate the output, a row at a time each.  Only a context that wants more CTAs than a cluster has

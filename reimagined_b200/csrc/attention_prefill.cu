@@ -350,8 +350,7 @@ bool attention_flash_supported(const tbl_attention_mixer& m) {
 
 bool attention_flash_whole(const tbl_attention_mixer& m) { return m.vdim <= kChunk; }
 
-int launch_attention_flash(const AttnParams& p, int n_seq, int context, cudaStream_t st) {
-    (void)context;
+int launch_attention_flash(const AttnParams& p, int n_seq, cudaStream_t st) {
     const long long rows = static_cast<long long>(n_seq) * p.n_tok, cached = static_cast<long long>(p.n_slots) * p.G * p.capacity;
     if (n_seq > 65535 || rows > 2147483647LL || cached > 2147483647LL) return TBL_ERR_SHAPE;
     const Rings rings = pick_rings(p.maps, p.dp, p.vp);
